@@ -38,7 +38,9 @@ class PagedKVNeed:
     the engine was given.  A mixer that wants something else says so: ``page_size`` and ``pool_tokens`` (tokens
     the group's pool holds; a windowed group can do with fewer), ``dtype`` (a torch dtype name) and
     ``page_shape`` (what one page is, as a tuple in which the string "page" stands for the page size, for
-    instance ``("page", 96)`` for one compressed vector per token)."""
+    instance ``("page", 96)`` for one compressed vector per token).  ``tokens_per_entry`` above 1: a page's entries
+    stand for that many consecutive tokens each (means of blocks of tokens, say), so a page of page_size entries covers
+    page_size * tokens_per_entry positions; the group's slots and block tables go on counting tokens."""
     num_kv_heads: int
     head_dim: int
     window: int = 0            # 0: all keys are kept
@@ -47,6 +49,7 @@ class PagedKVNeed:
     pool_tokens: int = 0       # 0: the engine's
     dtype: str | None = None   # None: the model's
     page_shape: tuple | None = None
+    tokens_per_entry: int = 1
 
     def shape_of_page(self, page_size: int) -> tuple:
         if self.page_shape is None:
@@ -368,7 +371,12 @@ class CacheManager:
             ps = int(need.page_size or page_size)
             if ps < 1:
                 raise CacheError(f"a page must hold at least one token, not {ps}")
-            self.groups.append(GroupInfo(need, ps, (int(need.pool_tokens or max_tokens) + ps - 1) // ps, cids))
+            pool, spare = int(need.pool_tokens or max_tokens), 0
+            if need.tokens_per_entry > 1:
+                # pages that cover more tokens than a page of the engine: every live request may leave most of its
+                # last one empty
+                ps, spare = ps * int(need.tokens_per_entry), int(max_requests)
+            self.groups.append(GroupInfo(need, ps, (pool + ps - 1) // ps + spare, cids))
         self.alloc = PageAllocator([g.page_size for g in self.groups], [g.num_pages for g in self.groups],
                                    [g.need.window for g in self.groups], max_requests,
                                    keep_first=[g.need.keep_first for g in self.groups])
@@ -379,8 +387,8 @@ class CacheManager:
         for g in self.groups:
             page_dtype = getattr(torch, g.need.dtype) if g.need.dtype else dtype
             for cid in g.cache_ids:
-                self.kv[cid] = torch.zeros((g.num_pages, *g.need.shape_of_page(g.page_size)), dtype=page_dtype,
-                                           device=device)
+                self.kv[cid] = torch.zeros((g.num_pages, *g.need.shape_of_page(g.page_size // g.need.tokens_per_entry)),
+                                           dtype=page_dtype, device=device)
         self.state: dict = {}
         for cid, need in self.state_needs.items():
             self.state[cid] = torch.zeros((self.max_requests, *need.shape), dtype=getattr(torch, need.dtype),

@@ -80,3 +80,5 @@ def _ensure_builtin():
         from ..models import mepatar  # noqa: F401
     if "Kasarax" not in _ARCHITECTURES:
         from ..models import kasarax  # noqa: F401
+    if "Sagizen" not in _ARCHITECTURES:
+        from ..models import sagizen  # noqa: F401

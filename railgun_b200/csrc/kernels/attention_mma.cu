@@ -21,6 +21,13 @@
 // Optional in both: `sink` [nh] (one more term exp(sink[h]) in head h's denominator, with neither key nor
 // value, unscaled, counted once: in the split kernel where the splits are added up) and `gate` (rows gate_ld
 // apart: head h's output at token t is multiplied by sigmoid(gate[t, h]) where it is divided by the denominator).
+// Output rows may be further apart than their width (out_ld), and the output may be multiplied by a constant
+// (out_scale) before its one rounding.
+//
+// With a window, and with `pool` > 0, tokens that have left the window are seen in blocks of `pool` instead: entry b
+// of a second set of pages (pool_kv, its own block table; pages of as many entries as the others have tokens) stands
+// for the positions b pool .. (b + 1) pool - 1, and the query at position p sees it once the block lies wholly before
+// the window, (b + 1) pool - 1 <= p - window.  Tokens and entries share one softmax.
 //
 // Head sizes: any multiple of 16 up to 256, compiled in three register-size
 // classes (<= 64, <= 128, <= 256).  Any page size.  K/V tiles are gathered
@@ -74,6 +81,10 @@ __device__ __forceinline__ float join_sink(float sink, float M, float& L) {
 }
 __device__ __forceinline__ float gate_of(const bf16* __restrict__ gate, int gate_ld, int t, int h) {
     return gate ? 1.f / (1.f + __expf(-__bfloat162float(gate[(size_t)t * gate_ld + h]))) : 1.f;
+}
+// How many pooled entries the query at position p sees: those whose last token is at least `window` back.
+__device__ __forceinline__ int pooled_seen(int p, int window, int pool) {
+    return p - window + 1 >= pool ? (p - window + 1) / pool : 0;
 }
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -134,13 +145,16 @@ struct TileGather {
 // ---------------------------------------------------------------------------------------------------
 // EXACT: the head size is DMAX itself, known at compile time (loops unroll without guards and shared-memory
 // addresses fold into the instructions); otherwise any multiple of 16 up to DMAX, passed at run time.
-template <int DMAX, bool EXACT>
+// POOL: the pooled entries' tiles come first, like the kept first tokens' tiles (`keep` is 0 then).
+template <int DMAX, bool EXACT, bool POOL>
 __global__ void __launch_bounds__(NTHREADS, DMAX <= 64 ? 4 : (DMAX <= 128 ? 2 : 1))
 prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out,
                          const bf16* __restrict__ kv_cache, const int* __restrict__ block_table, int max_blocks,
                          const int* __restrict__ tiles, const int* __restrict__ positions, int nh, int nkv, int d_arg,
                          int page_size, int page_shift, int window, int keep, float scale_log2,
-                         const float* __restrict__ sink, const bf16* __restrict__ gate, int gate_ld) {
+                         const float* __restrict__ sink, const bf16* __restrict__ gate, int gate_ld,
+                         const bf16* __restrict__ pool_kv, const int* __restrict__ pool_table, int pool_blocks, int pool,
+                         int out_ld, float out_scale) {
     const int d = EXACT ? DMAX : d_arg;
     constexpr int KD = DMAX / 16;          // k-steps over the head dimension
     constexpr int ND = DMAX / 8;           // n-tiles of the output
@@ -168,7 +182,11 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     // window's: the loop runs over tile numbers vt = kt0 - nk .. kt1, of which those below kt0 stand for tiles
     // 0 .. nk - 1.  Where the window's first tile touches the kept ones it is one run from tile 0.
     int nk = (window > 0 && keep > 0) ? (keep + BN - 1) / BN : 0;
-    if (kt0 <= nk) { kt0 = 0; nk = 0; }
+    if (!POOL && kt0 <= nk) { kt0 = 0; nk = 0; }
+    const int* pbt = POOL ? pool_table + (size_t)r * pool_blocks : nullptr;
+    const int n_pool = POOL ? pooled_seen(hi, window, pool) : 0;   // entries that the tile's last row sees
+    if (POOL) nk = (n_pool + BN - 1) / BN;                         // v0 = kt0 - nk may be negative: only differences count
+    auto pooled = [&](int vt) { return POOL && vt < kt0; };
     const int gap = kt0 - nk, v0 = kt0 - nk;
     auto phys = [&](int vt) { return vt >= kt0 ? vt : vt - gap; };
     const int d16 = d >> 4, d8 = d >> 3;
@@ -189,10 +207,13 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const size_t page_elems = (size_t)2 * nkv * page_size * d;
     const int v_off = nkv * page_size * d;
     int page_next[KD];
-    tg.pages(bt, phys(v0) * BN, hi + 1, page_next);
-    tg.issue(sKV, sKV + BN * stride, kv_cache, page_next, phys(v0) * BN, page_elems, v_off);
+    auto pages_of = [&](int vt) {
+        tg.pages(pooled(vt) ? pbt : bt, phys(vt) * BN, pooled(vt) ? n_pool : hi + 1, page_next);
+    };
+    pages_of(v0);
+    tg.issue(sKV, sKV + BN * stride, pooled(v0) ? pool_kv : kv_cache, page_next, phys(v0) * BN, page_elems, v_off);
     cp_async_commit();
-    tg.pages(bt, phys(v0 + 1) * BN, hi + 1, page_next);            // beyond the last key: all -1
+    pages_of(v0 + 1);                                              // beyond the last key: all -1
 
     uint32_t qf[Q_IN_REGS ? KD : 1][4];
     float o[ND][4];
@@ -213,9 +234,10 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         bf16* sV = sK + BN * stride;
         if (vt + 1 <= kt1) {
             bf16* nK = sKV + (stage ^ 1) * stage_elems;
-            tg.issue(nK, nK + BN * stride, kv_cache, page_next, phys(vt + 1) * BN, page_elems, v_off);
+            tg.issue(nK, nK + BN * stride, pooled(vt + 1) ? pool_kv : kv_cache, page_next, phys(vt + 1) * BN, page_elems,
+                     v_off);
             cp_async_commit();
-            tg.pages(bt, phys(vt + 2) * BN, hi + 1, page_next);
+            pages_of(vt + 2);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
@@ -229,7 +251,9 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         // this warp's rows attend nothing in this tile?  (all keys after its last row, or before its first row's window)
         const int key_base = kt * BN;
         const int wfirst = p0 + warp * 16, wlast = wfirst + 15;      // warp-uniform: every lane takes the same branch
-        const bool skip = key_base > wlast || (window > 0 && key_base + BN - 1 < wfirst - window + 1 && key_base >= keep);
+        const bool pool_tile = pooled(vt);
+        const bool skip = pool_tile ? key_base >= pooled_seen(wlast, window, pool)
+                                    : key_base > wlast || (window > 0 && key_base + BN - 1 < wfirst - window + 1 && key_base >= keep);
         if (!skip) {
             float s[BN / 8][4];
 #pragma unroll
@@ -250,7 +274,9 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
                 }
             }
             // scale into the log2 domain; mask by absolute position where the tile is not wholly attended
-            const bool edge = key_base + BN - 1 > wfirst || (window > 0 && key_base < wlast - window + 1);
+            const bool edge = pool_tile ? key_base + BN > pooled_seen(wfirst, window, pool)
+                                        : key_base + BN - 1 > wfirst || (window > 0 && key_base < wlast - window + 1);
+            const int see0 = pool_tile ? pooled_seen(prow0, window, pool) : 0, see1 = pool_tile ? pooled_seen(prow1, window, pool) : 0;
             float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
             for (int j = 0; j < BN / 8; ++j) {
@@ -260,7 +286,9 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
                     if (edge) {
                         const int key = key_base + j * 8 + tq * 2 + (e & 1);
                         const int prow = (e < 2) ? prow0 : prow1;
-                        if (!(key <= prow && (window <= 0 || key > prow - window || key < keep))) v = -INFINITY;
+                        const bool ok = pool_tile ? key < (e < 2 ? see0 : see1)
+                                                  : key <= prow && (window <= 0 || key > prow - window || key < keep);
+                        if (!ok) v = -INFINITY;
                     }
                     s[j][e] = v;
                     if (e < 2) mx0 = fmaxf(mx0, v); else mx1 = fmaxf(mx1, v);
@@ -313,6 +341,8 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     float f0 = 1.f, f1 = 1.f;
     if (sink) { f0 = join_sink(sink[h], m0, l0); f1 = join_sink(sink[h], m1, l1); }
+    f0 *= out_scale;
+    f1 *= out_scale;
     const int lr0 = warp * 16 + g, lr1 = lr0 + 8;
     if (gate) {
         if (lr0 < nrows) f0 *= gate_of(gate, gate_ld, row0 + lr0, h);
@@ -324,10 +354,10 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         if (i < d8) {
             const int col = i * 8 + tq * 2;
             if (lr0 < nrows)
-                *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + lr0) * nh + h) * d + col) =
+                *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + lr0) * out_ld + h * d + col) =
                     pack_bf16(o[i][0] * inv0, o[i][1] * inv0);
             if (lr1 < nrows)
-                *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + lr1) * nh + h) * d + col) =
+                *reinterpret_cast<uint32_t*>(out + (size_t)(row0 + lr1) * out_ld + h * d + col) =
                     pack_bf16(o[i][2] * inv1, o[i][3] * inv1);
         }
     }
@@ -348,7 +378,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
 #endif
 #define DEC_HEADS 8        // query heads per CTA
 
-template <int DMAX, bool EXACT>
+template <int DMAX, bool EXACT, bool POOL>
 __global__ void __launch_bounds__(NTHREADS)
 decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __restrict__ kv_cache,
                         const int* __restrict__ block_table, int max_blocks, const int* __restrict__ rows,
@@ -357,7 +387,9 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
                         int* __restrict__ counters, int nh, int nkv, int d_arg,
                         int page_size, int page_shift, int window, int keep, float scale_log2, int num_splits,
                         int head_tiles, int cluster_merge, const float* __restrict__ sink,
-                        const bf16* __restrict__ gate, int gate_ld) {
+                        const bf16* __restrict__ gate, int gate_ld,
+                        const bf16* __restrict__ pool_kv, const int* __restrict__ pool_table, int pool_blocks, int pool,
+                        int out_ld, float out_scale) {
     const int d = EXACT ? DMAX : d_arg;
     __shared__ int is_last;
     constexpr int KD = DMAX / 16;
@@ -391,7 +423,12 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
     // in the splits' key numbers, directly before the window's first tile: a key number below lo_al stands for
     // the key `shift` places earlier.  Where the window's first tile touches the kept ones it is one run from 0.
     int kept_al = (window > 0 && keep > 0) ? (keep + BN - 1) / BN * BN : 0;
-    if (lo_al <= kept_al) { lo_al = 0; kept_al = 0; }
+    if (!POOL && lo_al <= kept_al) { lo_al = 0; kept_al = 0; }
+    // The pooled entries are numbered like kept tokens: a key number below lo_al stands for entry number - shift.  They
+    // were written in earlier steps (an entry that this step completes is not seen by the step's own token).
+    const int* pbt = POOL ? pool_table + (size_t)r * pool_blocks : nullptr;
+    const int n_pool = POOL ? pooled_seen(pos, window, pool) : 0;
+    if (POOL) kept_al = (n_pool + BN - 1) / BN * BN;                // shift may be negative
     const int shift = lo_al - kept_al;
     const int n_keys = pos + 1 - shift;
     const int per_split = ((n_keys + num_splits - 1) / num_splits + BN - 1) / BN * BN;
@@ -429,8 +466,8 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
                 if (w > 0.f) acc += w * __ldcg(part_o + (base + s2) * d + col);
             }
             if (sink) acc *= join_sink(sink[h0 + row], M, L);
-            const float inv = L > 0.f ? gate_of(gate, gate_ld, t, h0 + row) / L : 0.f;
-            out[((size_t)t * nh + h0 + row) * d + col] = __float2bfloat16_rn(acc * inv);
+            const float inv = L > 0.f ? out_scale * gate_of(gate, gate_ld, t, h0 + row) / L : 0.f;
+            out[(size_t)t * out_ld + (h0 + row) * d + col] = __float2bfloat16_rn(acc * inv);
         }
     };
     // The splits' partial results in a cluster: fin_o [8 heads][d] unnormalised, fin_ml [8][2] = max (log2 domain) and
@@ -453,8 +490,8 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
                 L += w * ml[row * 2 + 1];
                 if (w > 0.f) acc += w * cluster.map_shared_rank(fin_o, s2)[row * d + col];
             }
-            const float inv = L > 0.f ? 1.f / L : 0.f;
-            out[((size_t)t * nh + h0 + row) * d + col] = __float2bfloat16_rn(acc * inv);
+            const float inv = L > 0.f ? out_scale / L : 0.f;
+            out[(size_t)t * out_ld + (h0 + row) * d + col] = __float2bfloat16_rn(acc * inv);
         }
         cluster.sync();                                             // nobody leaves while its results are being read
     };
@@ -495,6 +532,19 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
     for (int j = 0; j < KD; ++j) g_dst[j] = g_row[j] * stride + g_col[j];
     auto pages_of = [&](int key0, int (&pg)[KD]) {                 // page of every piece's row (-1: no such key)
         const int back = key0 < lo_al ? shift : 0;                  // a tile of the kept first tokens
+        if (POOL && key0 < lo_al) {                                 // or of pooled entries
+            const int entry = key0 - shift + warp * 16;
+            if (one_page) {
+                pg[0] = key0 < k_end && entry < n_pool ? pbt[entry >> page_shift] : -1;
+                return;
+            }
+#pragma unroll
+            for (int j = 0; j < KD; ++j) {
+                const int pe = entry + g_row[j];
+                pg[j] = (g_row[j] >= 0 && key0 < k_end && pe < n_pool) ? pbt[page_shift >= 0 ? pe >> page_shift : pe / page_size] : -1;
+            }
+            return;
+        }
         if (one_page) {
             const int key = key0 + warp * 16;                      // the same page for the whole warp
             pg[0] = key < k_end ? bt[(key - back) >> page_shift] : -1;
@@ -511,19 +561,21 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
         bf16* sK = sKV + stage * stage_elems + warp * 16 * stride;
         bf16* sV = sK + BN * stride;
         const int back = key0 < lo_al ? shift : 0;
+        const bf16* pages = POOL && key0 < lo_al ? pool_kv : kv_cache;
         if (one_page) {
             const int key = key0 + warp * 16;
             const bool page_ok = pg[0] >= 0;
-            const bf16* base = kv_cache;
+            const bf16* base = pages;
             if (page_ok)
-                base = kv_cache + (size_t)pg[0] * page_elems +
+                base = pages + (size_t)pg[0] * page_elems +
                        ((size_t)kvh * page_size + ((key - back) & (page_size - 1))) * d;
-            const int rows_ok = k_end - key;                        // rows at or beyond it are zero-filled
+            // rows at or beyond it are zero-filled
+            const int rows_ok = POOL && key0 < lo_al ? n_pool - (key - shift) : k_end - key;
 #pragma unroll
             for (int j = 0; j < KD; ++j) {
                 if (g_row[j] >= 0) {
                     const bool valid = page_ok && g_row[j] < rows_ok;
-                    const bf16* ksrc = valid ? base + (lane + 32 * j) * 8 : kv_cache;
+                    const bf16* ksrc = valid ? base + (lane + 32 * j) * 8 : pages;
                     cp_async16(sK + g_dst[j], ksrc, valid);
                     cp_async16(sV + g_dst[j], ksrc + (valid ? v_off : 0), valid);
                 }
@@ -534,11 +586,11 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
         for (int j = 0; j < KD; ++j) {
             if (g_row[j] >= 0) {
                 const bool valid = pg[j] >= 0;
-                const bf16* ksrc = kv_cache;
+                const bf16* ksrc = pages;
                 if (valid) {
                     const int key = key0 + warp * 16 + g_row[j] - back;
                     const int off = page_shift >= 0 ? key & (page_size - 1) : key % page_size;
-                    ksrc = kv_cache + (size_t)pg[j] * page_elems + ((size_t)kvh * page_size + off) * d + g_col[j];
+                    ksrc = pages + (size_t)pg[j] * page_elems + ((size_t)kvh * page_size + off) * d + g_col[j];
                 }
                 cp_async16(sK + g_dst[j], ksrc, valid);
                 cp_async16(sV + g_dst[j], ksrc + (valid ? v_off : 0), valid);
@@ -607,7 +659,8 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
         __syncwarp();
         const int key_base = k_begin + it * BN + warp * 16;          // this warp's 16 keys (as the splits number them)
         const int pkb = key_base < lo_al ? key_base - shift : key_base;   // and where they are in the request
-        if (key_base < k_end && (pkb + 15 >= lo || pkb < keep)) {
+        const bool pool_tile = POOL && key_base < lo_al;
+        if (key_base < k_end && (pool_tile ? pkb < n_pool : (pkb + 15 >= lo || pkb < keep))) {
             float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
             for (int kd = 0; kd < KD; ++kd) {
@@ -622,7 +675,15 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
             }
             // head g, keys key_base + 2 tq + {0, 1} (s0) and + 8 (s1); rows 8..15 of the tile are padding
             float v00 = s0[0] * scale_log2, v01 = s0[1] * scale_log2, v10 = s1[0] * scale_log2, v11 = s1[1] * scale_log2;
-            if (key_base + 16 > k_end || pkb < lo) {                 // an edge tile: some of its keys are not attended
+            if (pool_tile) {
+                if (pkb + 16 > n_pool) {
+                    const int p0 = pkb + tq * 2;
+                    if (p0 >= n_pool) v00 = -INFINITY;
+                    if (p0 + 1 >= n_pool) v01 = -INFINITY;
+                    if (p0 + 8 >= n_pool) v10 = -INFINITY;
+                    if (p0 + 9 >= n_pool) v11 = -INFINITY;
+                }
+            } else if (key_base + 16 > k_end || pkb < lo) {          // an edge tile: some of its keys are not attended
                 const int k0 = key_base + tq * 2, p0 = pkb + tq * 2;
                 if (!(k0 < k_end && (p0 >= lo || p0 < keep))) v00 = -INFINITY;
                 if (!(k0 + 1 < k_end && (p0 + 1 >= lo || p0 + 1 < keep))) v01 = -INFINITY;
@@ -695,8 +756,8 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
         }
         if (num_splits == 1 && counters != nullptr) {               // the only split: this is the result
             if (sink) acc *= join_sink(sink[h0 + row], M, L);
-            const float inv = L > 0.f ? gate_of(gate, gate_ld, t, h0 + row) / L : 0.f;
-            out[((size_t)t * nh + h0 + row) * d + col] = __float2bfloat16_rn(acc * inv);
+            const float inv = L > 0.f ? out_scale * gate_of(gate, gate_ld, t, h0 + row) / L : 0.f;
+            out[(size_t)t * out_ld + (h0 + row) * d + col] = __float2bfloat16_rn(acc * inv);
         } else if (cluster_merge) {
             fin_o[row * d + col] = acc;
             if (col == 0) { fin_ml[row * 2] = M; fin_ml[row * 2 + 1] = L; }
@@ -714,7 +775,7 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
 __global__ void decode_reduce_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                      bf16* __restrict__ out, const int* __restrict__ rows, int nh, int d,
                                      int num_splits, const float* __restrict__ sink, const bf16* __restrict__ gate,
-                                     int gate_ld) {
+                                     int gate_ld, int out_ld, float out_scale) {
     pdl_wait();
     pdl_trigger();
     const int ti = blockIdx.x, h = blockIdx.y;
@@ -726,14 +787,14 @@ __global__ void decode_reduce_kernel(const float* __restrict__ part_o, const flo
     float L = 0.f;
     for (int s = 0; s < num_splits; ++s) L += exp2f(part_ml[(base + s) * 2] - Ms) * part_ml[(base + s) * 2 + 1];
     const float fs = sink ? join_sink(sink[h], M, L) : 1.f;
-    const float inv = L > 0.f ? fs * gate_of(gate, gate_ld, t, h) / L : 0.f;
+    const float inv = L > 0.f ? out_scale * fs * gate_of(gate, gate_ld, t, h) / L : 0.f;
     for (int c = threadIdx.x; c < d; c += blockDim.x) {
         float acc = 0.f;
         for (int s = 0; s < num_splits; ++s) {
             const float w = exp2f(part_ml[(base + s) * 2] - Ms);
             if (w > 0.f) acc += w * part_o[(base + s) * d + c];
         }
-        out[((size_t)t * nh + h) * d + c] = __float2bfloat16_rn(acc * inv);
+        out[(size_t)t * out_ld + h * d + c] = __float2bfloat16_rn(acc * inv);
     }
 }
 
@@ -750,15 +811,23 @@ template <typename K> static int allow_smem(K kernel, size_t bytes) {
     return (int)cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
 }
 
+// The pooled entries' pages: what the kernels take beside the tokens' pages (pool 0: none).
+static bool pool_ok(const void* pool_kv, const int* pool_table, int pool, int window, int keep_first) {
+    return pool == 0 || (pool > 0 && pool_kv && pool_table && window > 0 && keep_first == 0);
+}
+
 // keep_first: with a window, the first positions of a request that every later query still sees; sink [nh] and
-// gate (rows gate_ld apart) may be null
+// gate (rows gate_ld apart) may be null; pool_kv, pool_table [R, pool_blocks], pool: the pooled entries (pool 0: none);
+// out rows out_ld apart (an even number), the output times out_scale
 extern "C" int rg_prefill_attention_sink(const void* q, int q_stride, void* out, const void* kv_cache,
                                          const int* block_table, int max_blocks, const int* tiles, int n_tiles,
                                          const int* positions, int nh, int nkv, int d, int page_size, int window,
                                          int keep_first, float scale, const float* sink, const void* gate, int gate_ld,
-                                         void* stream) {
+                                         const void* pool_kv, const int* pool_table, int pool_blocks, int pool,
+                                         int out_ld, float out_scale, void* stream) {
     if (n_tiles <= 0) return 0;
-    if (keep_first < 0) return RG_ERR_UNSUPPORTED;
+    if (keep_first < 0 || !pool_ok(pool_kv, pool_table, pool, window, keep_first) || out_ld < nh * d || out_ld % 2)
+        return RG_ERR_UNSUPPORTED;
     if (d % 16 || d < 16 || d > 256 || nkv < 1 || nh < nkv || nh % nkv || (long long)n_tiles * nh > 0x7fffffffll)
         return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
@@ -767,12 +836,15 @@ extern "C" int rg_prefill_attention_sink(const void* q, int q_stride, void* out,
     int page_shift = -1;                                            // log2 of the page size when it is a power of two
     for (int b = 0; b < 31; ++b) if (page_size == (1 << b)) page_shift = b;
     dim3 grid(n_tiles * nh);
-#define RG_PREFILL(DM, EX) { int e = allow_smem(prefill_attention_kernel<DM, EX>, smem); if (e) return e; \
-    return rg_launch(prefill_attention_kernel<DM, EX>, grid, dim3(NTHREADS), smem, s, 1, (const bf16*)q, q_stride, \
+#define RG_PREFILL(DM, EX) { if (pool > 0) RG_PREFILL_(DM, EX, true) else RG_PREFILL_(DM, EX, false) }
+#define RG_PREFILL_(DM, EX, PO) { int e = allow_smem(prefill_attention_kernel<DM, EX, PO>, smem); if (e) return e; \
+    return rg_launch(prefill_attention_kernel<DM, EX, PO>, grid, dim3(NTHREADS), smem, s, 1, (const bf16*)q, q_stride, \
         (bf16*)out, (const bf16*)kv_cache, block_table, max_blocks, tiles, positions, nh, nkv, d, page_size, page_shift, \
-        window, window > 0 ? keep_first : 0, scale_log2, sink, (const bf16*)gate, gate_ld); }
+        window, window > 0 ? keep_first : 0, scale_log2, sink, (const bf16*)gate, gate_ld, (const bf16*)pool_kv, \
+        pool_table, pool_blocks, pool, out_ld, out_scale); }
     if (d == 64) RG_PREFILL(64, true) else if (d == 128) RG_PREFILL(128, true)
     else if (d < 64) RG_PREFILL(64, false) else if (d < 128) RG_PREFILL(128, false) else RG_PREFILL(256, false)
+#undef RG_PREFILL_
 #undef RG_PREFILL
 }
 
@@ -781,7 +853,8 @@ extern "C" int rg_prefill_attention_keep(const void* q, int q_stride, void* out,
                                          const int* positions, int nh, int nkv, int d, int page_size, int window,
                                          int keep_first, float scale, void* stream) {
     return rg_prefill_attention_sink(q, q_stride, out, kv_cache, block_table, max_blocks, tiles, n_tiles, positions, nh,
-                                     nkv, d, page_size, window, keep_first, scale, nullptr, nullptr, 0, stream);
+                                     nkv, d, page_size, window, keep_first, scale, nullptr, nullptr, 0, nullptr, nullptr, 0, 0,
+                                     nh * d, 1.f, stream);
 }
 
 extern "C" int rg_prefill_attention(const void* q, int q_stride, void* out, const void* kv_cache,
@@ -797,7 +870,9 @@ static int rg_decode_attention_any(const void* q, int q_stride, void* out, const
                                    const int* req_of_token, const int* positions, float* part_o, float* part_ml,
                                    int* counters, int nh, int nkv, int d, int page_size, int window, float scale,
                                    int num_splits, int cluster_merge, void* stream, int keep_first = 0,
-                                   const float* sink = nullptr, const void* gate = nullptr, int gate_ld = 0);
+                                   const float* sink = nullptr, const void* gate = nullptr, int gate_ld = 0,
+                                   const void* pool_kv = nullptr, const int* pool_table = nullptr, int pool_blocks = 0,
+                                   int pool = 0, int out_ld = 0, float out_scale = 1.f);
 
 // Scratch the caller provides: part_o floats = n_tokens * nh * num_splits * d; part_ml = n_tokens * nh * num_splits * 2.
 // counters: NULL (a second kernel reduces the splits), or n_tokens * nkv * ceil(group / 8) ints that are zero on
@@ -824,17 +899,19 @@ extern "C" int rg_decode_attention_keep(const void* q, int q_stride, void* out, 
                                    0, stream, keep_first);
 }
 
-// sink [nh] and gate (rows gate_ld apart) may be null
+// sink [nh] and gate (rows gate_ld apart) may be null; pooled entries, out_ld and out_scale as for prompts
 extern "C" int rg_decode_attention_sink(const void* q, int q_stride, void* out, const void* kv_cache,
                                         const int* block_table, int max_blocks, const int* rows, int n_tokens,
                                         const int* req_of_token, const int* positions, float* part_o, float* part_ml,
                                         int* counters, int nh, int nkv, int d, int page_size, int window,
                                         int keep_first, float scale, int num_splits, const float* sink, const void* gate,
-                                        int gate_ld, void* stream) {
-    if (keep_first < 0) return RG_ERR_UNSUPPORTED;
+                                        int gate_ld, const void* pool_kv, const int* pool_table, int pool_blocks, int pool,
+                                        int out_ld, float out_scale, void* stream) {
+    if (keep_first < 0 || !pool_ok(pool_kv, pool_table, pool, window, keep_first) || out_ld < nh * d) return RG_ERR_UNSUPPORTED;
     return rg_decode_attention_any(q, q_stride, out, kv_cache, block_table, max_blocks, rows, n_tokens, req_of_token,
                                    positions, part_o, part_ml, counters, nh, nkv, d, page_size, window, scale, num_splits,
-                                   0, stream, keep_first, sink, gate, gate_ld);
+                                   0, stream, keep_first, sink, gate, gate_ld, pool_kv, pool_table, pool_blocks, pool,
+                                   out_ld, out_scale);
 }
 
 // The same with the splits of every (token, head tile) as one thread-block cluster (2 to 8 splits): no scratch, no
@@ -858,9 +935,11 @@ static int rg_decode_attention_any(const void* q, int q_stride, void* out, const
                                    const int* req_of_token, const int* positions, float* part_o, float* part_ml,
                                    int* counters, int nh, int nkv, int d, int page_size, int window, float scale,
                                    int num_splits, int cluster_merge, void* stream, int keep_first, const float* sink,
-                                   const void* gate, int gate_ld) {
+                                   const void* gate, int gate_ld, const void* pool_kv, const int* pool_table,
+                                   int pool_blocks, int pool, int out_ld, float out_scale) {
     if (n_tokens <= 0) return 0;
-    if (cluster_merge && (sink || gate)) return RG_ERR_UNSUPPORTED;
+    if (out_ld == 0) out_ld = nh * d;
+    if (cluster_merge && (sink || gate || pool)) return RG_ERR_UNSUPPORTED;
     if (d % 16 || d < 16 || d > 256 || nkv < 1 || nh < nkv || nh % nkv || num_splits < 1) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const float scale_log2 = scale * 1.4426950408889634f;
@@ -873,20 +952,23 @@ static int rg_decode_attention_any(const void* q, int q_stride, void* out, const
     dim3 grid(n_tokens, nkv * head_tiles, num_splits);
     if (cluster_merge) grid = dim3(num_splits, nkv * head_tiles, n_tokens);
     int e = 0;
-#define RG_DECODE(DM, EX) { e = allow_smem(decode_attention_kernel<DM, EX>, smem); if (e) return e; \
-    e = rg_launch(decode_attention_kernel<DM, EX>, grid, dim3(NTHREADS), smem, s, cluster_merge ? num_splits : 1, \
+#define RG_DECODE(DM, EX) { if (pool > 0) RG_DECODE_(DM, EX, true) else RG_DECODE_(DM, EX, false) }
+#define RG_DECODE_(DM, EX, PO) { e = allow_smem(decode_attention_kernel<DM, EX, PO>, smem); if (e) return e; \
+    e = rg_launch(decode_attention_kernel<DM, EX, PO>, grid, dim3(NTHREADS), smem, s, cluster_merge ? num_splits : 1, \
         (const bf16*)q, q_stride, \
         (const bf16*)kv_cache, block_table, max_blocks, rows, req_of_token, positions, part_o, part_ml, (bf16*)out, \
         counters, nh, nkv, d, page_size, page_shift, window, window > 0 ? keep_first : 0, scale_log2, num_splits, \
-        head_tiles, cluster_merge, sink, (const bf16*)gate, gate_ld); }
+        head_tiles, cluster_merge, sink, (const bf16*)gate, gate_ld, (const bf16*)pool_kv, pool_table, pool_blocks, pool, \
+        out_ld, out_scale); }
     if (d == 64) RG_DECODE(64, true) else if (d == 128) RG_DECODE(128, true)
     else if (d < 64) RG_DECODE(64, false) else if (d < 128) RG_DECODE(128, false) else RG_DECODE(256, false)
+#undef RG_DECODE_
 #undef RG_DECODE
     if (e || counters != nullptr || cluster_merge) return e;
     dim3 rgrid(n_tokens, nh);
     RgStreamOrder in_order(true);       // measured: the merge starting early, beside the splits, costs a batch-8 step 4 %
     return rg_launch(decode_reduce_kernel, rgrid, dim3(d >= 128 ? 128 : 64), 0, s, 1, (const float*)part_o,
-                     (const float*)part_ml, (bf16*)out, rows, nh, d, num_splits, sink, (const bf16*)gate, gate_ld);
+                     (const float*)part_ml, (bf16*)out, rows, nh, d, num_splits, sink, (const bf16*)gate, gate_ld, out_ld, out_scale);
 }
 
 // ---------------------------------------------------------------------------------------------------

@@ -1,15 +1,20 @@
 // Mixers whose memory is a matrix per head instead of a growing cache, and the short causal convolutions
 // that sit in front of them.
 //
-//   causal_conv        y_t = [x_t +] act(sum_j w[:, j] x_(t - K + 1 + j)) per channel, K taps, the last column of w the
+//   causal_conv        y_t = [x_t +] act(bias + sum_j w[:, j] x_(t - K + 1 + j)) per channel, K taps, the last column of w the
 //                      current token's; continued from the K - 1 inputs a request keeps in its state slot
 //   conv_state_update  leaves the step's last K - 1 inputs in the slot
 //   retention_prepare  rotation of q and k in pairs (i, i + dims / 2), k times a constant, into 32-bit rows
 //   delta_prepare      q and k to unit length per head (q times a constant), beta = sigmoid(b),
 //                      g = exp(-exp(A) softplus(a + bias)) per head
 //   state_scan         per head, token by token, S [d, dv] in 32-bit:
-//                        retention:  S <- decay_h S + k v^T;                         o = S^T q
-//                        delta rule: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
+//                        scalar decay:  S <- g S + beta k v^T;  o = S^T q + skip_h v
+//                                       (retention: g fixed per head, beta 1, skip 0; the state-space duality form of
+//                                       Mamba-2: g and beta per token)
+//                        delta rule:    S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q
+//                        channel decay: o = (S + diag(bonus_h) k v^T)^T q;  S <- diag(w_t) S + k v^T
+//                                       (RWKV-style: a decay per token and key channel, the current token through the
+//                                       bonus instead)
 //                      (Sun et al., "Retentive Network: A Successor to Transformer for Large Language Models";
 //                      Yang et al., "Gated Delta Networks: Improving Mamba2 with Delta Rule")
 //   head_norm_gate     o / rms(o) per head [times a weight], times silu(gate), rounded once for the output product
@@ -28,7 +33,8 @@ __device__ __forceinline__ float sm_softplus(float z) { return log1pf(expf(-fabs
 // out: rows out_ld apart (type O).  residual: out = x + conv(x); act 1: silu of the convolution.
 template <typename A, typename O>
 __global__ void causal_conv_kernel(const A* __restrict__ x, int ld, int x_off, const float* __restrict__ taps,
-                                   const float* __restrict__ state, const int* __restrict__ cu_seqlens,
+                                   const float* __restrict__ bias, const float* __restrict__ state,
+                                   const int* __restrict__ cu_seqlens,
                                    const int* __restrict__ req_of_token, const int* __restrict__ start_pos,
                                    const int* __restrict__ slots, O* __restrict__ out, int out_ld, int C, int K,
                                    int residual, int act) {
@@ -41,7 +47,7 @@ __global__ void causal_conv_kernel(const A* __restrict__ x, int ld, int x_off, c
     const int i = t - cu_seqlens[r];
     const int slot = slots[r];
     const bool has_past = slot >= 0 && start_pos[r] > 0;
-    float acc = 0.f;
+    float acc = bias ? bias[c] : 0.f;
     for (int j = 0; j < K; ++j) {
         const int idx = i - (K - 1) + j;                     // the step's token this tap reads; negative: before the step
         float v;
@@ -57,7 +63,8 @@ __global__ void causal_conv_kernel(const A* __restrict__ x, int ld, int x_off, c
 // The same for bfloat16 inputs with eight channels per thread (16-byte loads), where rows and offsets allow it.
 template <typename O>
 __global__ void causal_conv8_kernel(const bf16* __restrict__ x, int ld, int x_off, const float* __restrict__ taps,
-                                    const float* __restrict__ state, const int* __restrict__ cu_seqlens,
+                                    const float* __restrict__ bias, const float* __restrict__ state,
+                                    const int* __restrict__ cu_seqlens,
                                     const int* __restrict__ req_of_token, const int* __restrict__ start_pos,
                                     const int* __restrict__ slots, O* __restrict__ out, int out_ld, int C, int K,
                                     int residual, int act) {
@@ -70,7 +77,9 @@ __global__ void causal_conv8_kernel(const bf16* __restrict__ x, int ld, int x_of
     const int i = t - cu_seqlens[r];
     const int slot = slots[r];
     const bool has_past = slot >= 0 && start_pos[r] > 0;
-    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    float acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = bias ? bias[c + e] : 0.f;
     float cur[8];
     for (int j = 0; j < K; ++j) {
         const int idx = i - (K - 1) + j;
@@ -142,8 +151,9 @@ __global__ void conv_state_update_kernel(const A* __restrict__ x, int ld, int x_
 }
 
 
-extern "C" int rg_causal_conv(const void* x, int x_dtype, int ld, int x_off, const float* taps, const float* state,
-                              const int* cu_seqlens, const int* req_of_token, const int* start_pos, const int* slots,
+// bias [C] or null
+extern "C" int rg_causal_conv(const void* x, int x_dtype, int ld, int x_off, const float* taps, const float* bias,
+                              const float* state, const int* cu_seqlens, const int* req_of_token, const int* start_pos, const int* slots,
                               void* out, int out_dtype, int out_ld, int T, int C, int K, int residual, int act,
                               void* stream) {
     if (T <= 0 || C <= 0) return 0;
@@ -157,17 +167,17 @@ extern "C" int rg_causal_conv(const void* x, int x_dtype, int ld, int x_off, con
         dim3 g8(T, (C / 8 + th - 1) / th);
         if (g8.y > 65535) return RG_ERR_UNSUPPORTED;
         if (out_dtype == RG_DTYPE_BF16)
-            return rg_launch(causal_conv8_kernel<bf16>, g8, dim3(th), 0, s, 1, (const bf16*)x, ld, x_off, taps, state,
+            return rg_launch(causal_conv8_kernel<bf16>, g8, dim3(th), 0, s, 1, (const bf16*)x, ld, x_off, taps, bias, state,
                              cu_seqlens, req_of_token, start_pos, slots, (bf16*)out, out_ld, C, K, residual, act);
         if (out_dtype == RG_DTYPE_F32)
-            return rg_launch(causal_conv8_kernel<float>, g8, dim3(th), 0, s, 1, (const bf16*)x, ld, x_off, taps, state,
+            return rg_launch(causal_conv8_kernel<float>, g8, dim3(th), 0, s, 1, (const bf16*)x, ld, x_off, taps, bias, state,
                              cu_seqlens, req_of_token, start_pos, slots, (float*)out, out_ld, C, K, residual, act);
     }
     const int threads = C >= 256 ? 256 : 128;
     dim3 grid(T, (C + threads - 1) / threads);
     if (grid.y > 65535) return RG_ERR_UNSUPPORTED;
 #define SM_CONV(A, O) return rg_launch(causal_conv_kernel<A, O>, grid, dim3(threads), 0, s, 1, (const A*)x, ld, x_off, taps, \
-        state, cu_seqlens, req_of_token, start_pos, slots, (O*)out, out_ld, C, K, residual, act)
+        bias, state, cu_seqlens, req_of_token, start_pos, slots, (O*)out, out_ld, C, K, residual, act)
     if (x_dtype == RG_DTYPE_BF16 && out_dtype == RG_DTYPE_BF16) SM_CONV(bf16, bf16);
     if (x_dtype == RG_DTYPE_BF16 && out_dtype == RG_DTYPE_F32) SM_CONV(bf16, float);
     if (x_dtype == RG_DTYPE_F32 && out_dtype == RG_DTYPE_F32) SM_CONV(float, float);
@@ -297,18 +307,23 @@ extern "C" int rg_delta_prepare(float* qk, int ld, int G, int d, float q_scale, 
 // are neighbouring lanes and add their shares with shuffles, read neighbouring 16 bytes of a k or q row (no bank
 // conflicts) and of the column's state.  The
 // columns of S never meet (S^T k and S^T q are sums down a column), so a head's columns are spread over blocks.
-// Tokens are staged in shared memory `chunk` at a time, the next chunk on its way (cp.async for q and k, registers
+// Tokens are staged in shared memory `chunk` at a time, the next chunk on its way (cp.async for q, k and w, registers
 // for v, g and beta) while this one is worked on; q and k rows are padded with zeros to parts * DPER numbers (rows
 // of S beyond d then stay zero without a test in the loop).  q, k: [T, Hqk, d] float rows q_ld / k_ld apart; head h
-// reads q/k head h / (H / Hqk).  v: rows v_ld apart (float or bfloat16), head h at column h dv.  decay [H]
-// (retention) or g, beta [T, H] (delta rule; beta null: retention).  state [slots, H, dv, d]: S transposed, a
+// reads q/k head h / (H / Hqk).  v: rows v_ld apart (float or bfloat16), head h at column h dv.  decay [H] or g [T, H];
+// beta [T, H] or null (1); skip [H] or null (0); channel decay: w like k (rows w_ld apart, its own head h), bonus
+// [H, d].  state [slots, H, dv, d]: S transposed, a
 // thread's rows side by side.  o [T, H, dv] float.
 //
 // The delta rule per token, with a = S_old^T k, b = S_old^T q (one pass over S, reduced together) and c = k . q:
 //   u = beta (v - g a);  o = g b + u c;  S <- g S + k u^T
 // (c once per token and block, when its chunk has arrived) which is S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q with one reduction in the chain from token
-// to token instead of two.  Retention: o = decay b + v c;  S <- decay S + k v^T.
+// to token instead of two.  Scalar decay: o = g b + v (beta c + skip);  S <- g S + k (beta v)^T.  Channel decay:
+// o = b + v c with c = sum_i bonus_i k_i q_i;  S <- diag(w) S + k v^T.
 #define SCAN_THREADS 128
+#define SCAN_SCALAR 0
+#define SCAN_DELTA 1
+#define SCAN_CHANNEL 2
 #define SCAN_MAX_PREFETCH 4       // v numbers of the next chunk a thread holds: chunk * CB <= 4 * threads of the block
 
 __device__ __forceinline__ void scan_cp_async4(float* dst, const float* src) {
@@ -320,18 +335,22 @@ __device__ __forceinline__ void scan_cp_async16(float* dst, const float* src) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(d), "l"(src));
 }
 
-template <int DPER, int PARTS, bool DELTA, typename V>
+template <int DPER, int PARTS, int RULE, typename V>
 __global__ void __launch_bounds__(SCAN_THREADS)
 state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict__ k, int k_ld,
                   const V* __restrict__ v, int v_ld, const float* __restrict__ decay,
-                  const float* __restrict__ g, const float* __restrict__ beta,
+                  const float* __restrict__ g, const float* __restrict__ beta, const float* __restrict__ skip,
+                  const float* __restrict__ w, int w_ld, const float* __restrict__ bonus,
                   float* __restrict__ state, const int* __restrict__ cu_seqlens,
                   const int* __restrict__ start_pos, const int* __restrict__ slots,
                   float* __restrict__ o, int H, int Hqk, int d, int dv, int CB, int chunk, int vec) {
     extern __shared__ __align__(16) float sm[];
     constexpr int parts = PARTS;
     constexpr int DP = PARTS * DPER;                 // padded length of a q or k row
-    const int stage = chunk * (2 * DP + CB + 4);     // floats of one stage: q, k [chunk][DP], v [chunk][CB], (g, beta, c, -) [chunk]
+    constexpr bool DELTA = RULE == SCAN_DELTA, CHANNEL = RULE == SCAN_CHANNEL;
+    constexpr int ROWS = CHANNEL ? 3 : 2;            // staged rows of a token: q, k (, w)
+    // floats of one stage: q, k (, w) [chunk][DP], v [chunk][CB], (g, beta, c, -) [chunk]; behind both stages the bonus [DP]
+    const int stage = chunk * (ROWS * DP + CB + 4);
     pdl_wait();
     pdl_trigger();
     const int r = blockIdx.x, h = blockIdx.y, j0 = blockIdx.z * CB;
@@ -365,8 +384,13 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
             const int tt = rem / (DP - d), i = d + rem - tt * (DP - d);
             sm[stg * stage + tt * DP + i] = 0.f;
             sm[stg * stage + chunk * DP + tt * DP + i] = 0.f;
+            if (CHANNEL) sm[stg * stage + 2 * chunk * DP + tt * DP + i] = 0.f;
         }
     }
+    float* sbonus = sm + 2 * stage;
+    if (CHANNEL)
+        for (int i = threadIdx.x; i < DP; i += blockDim.x) sbonus[i] = i < d ? bonus[(size_t)h * d + i] : 0.f;
+    const float own_skip = skip ? skip[h] : 0.f;
     float pv[SCAN_MAX_PREFETCH], pg = 0.f, pb = 0.f;
     // this thread's places in a chunk's tile of v (the same in every chunk), and in the rows of q and k
     int v_tt[SCAN_MAX_PREFETCH], v_i[SCAN_MAX_PREFETCH];
@@ -379,11 +403,12 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
     const V* vh = v + (size_t)h * dv + j0;
     const float* qh = q + (size_t)hq * d;
     const float* kh = k + (size_t)hq * d;
+    const float* wh = CHANNEL ? w + (size_t)h * d : nullptr;
     const int d4 = d >> 2;
     const bool by_rows = vec && d4 <= (int)blockDim.x;               // whole rows per pass: no division in the loop
     const int rpp = by_rows ? blockDim.x / d4 : 1, row_t = threadIdx.x / (by_rows ? d4 : 1),
               row_i = by_rows ? (threadIdx.x - row_t * d4) * 4 : 0;
-    // q and k of `n` tokens from `base` on into stage `stg`, asynchronously
+    // q and k (and w) of `n` tokens from `base` on into stage `stg`, asynchronously
     auto issue = [&](int stg, int base, int n) {
         float* sq = sm + stg * stage;
         float* sk = sq + chunk * DP;
@@ -392,18 +417,21 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
                 for (int tt = row_t; tt < n; tt += rpp) {
                     scan_cp_async16(sq + tt * DP + row_i, qh + (size_t)(base + tt) * q_ld + row_i);
                     scan_cp_async16(sk + tt * DP + row_i, kh + (size_t)(base + tt) * k_ld + row_i);
+                    if (CHANNEL) scan_cp_async16(sk + (chunk + tt) * DP + row_i, wh + (size_t)(base + tt) * w_ld + row_i);
                 }
         } else if (vec) {
             for (int e = threadIdx.x; e < n * d4; e += blockDim.x) {
                 const int tt = e / d4, i = (e - tt * d4) * 4;
                 scan_cp_async16(sq + tt * DP + i, q + (size_t)(base + tt) * q_ld + (size_t)hq * d + i);
                 scan_cp_async16(sk + tt * DP + i, k + (size_t)(base + tt) * k_ld + (size_t)hq * d + i);
+                if (CHANNEL) scan_cp_async16(sk + (chunk + tt) * DP + i, wh + (size_t)(base + tt) * w_ld + i);
             }
         } else {
             for (int e = threadIdx.x; e < n * d; e += blockDim.x) {
                 const int tt = e / d, i = e - tt * d;
                 scan_cp_async4(sq + tt * DP + i, q + (size_t)(base + tt) * q_ld + (size_t)hq * d + i);
                 scan_cp_async4(sk + tt * DP + i, k + (size_t)(base + tt) * k_ld + (size_t)hq * d + i);
+                if (CHANNEL) scan_cp_async4(sk + (chunk + tt) * DP + i, wh + (size_t)(base + tt) * w_ld + i);
             }
         }
         asm volatile("cp.async.commit_group;\n" ::);
@@ -415,11 +443,11 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
             if (v_tt[x] < n) pv[x] = to_f32(vh[(size_t)(base + v_tt[x]) * v_ld + v_i[x]]);
         if ((int)threadIdx.x < n) {
             pg = g ? g[(size_t)(base + threadIdx.x) * H + h] : fixed;
-            pb = beta ? beta[(size_t)(base + threadIdx.x) * H + h] : 0.f;
+            pb = beta ? beta[(size_t)(base + threadIdx.x) * H + h] : 1.f;
         }
     };
     auto park = [&](int stg, int n) {
-        float* sv = sm + stg * stage + 2 * chunk * DP;
+        float* sv = sm + stg * stage + ROWS * chunk * DP;
 #pragma unroll
         for (int x = 0; x < SCAN_MAX_PREFETCH; ++x)
             if (v_tt[x] < n) sv[v_tt[x] * CB + v_i[x]] = pv[x];
@@ -448,9 +476,10 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
         __syncthreads();                                            // this stage is complete for everybody
         const float* sq = sm + stg * stage;
         const float* sk = sq + chunk * DP;
-        const float* sv = sk + chunk * DP;
-        float* sgbc = sm + stg * stage + chunk * (2 * DP + CB);      // (g, beta, c, -) of every token
-        // c = k . q of the chunk's tokens, eight lanes a token
+        const float* sv = sk + (ROWS - 1) * chunk * DP;
+        float* sgbc = sm + stg * stage + chunk * (ROWS * DP + CB);   // (g, beta, c, -) of every token
+        // c = k . q of the chunk's tokens (scalar decay: beta c + skip; channel decay: with the bonus in the sum), eight
+        // lanes a token
         // (every lane runs every round of the loop, so that the shuffles meet whole warps)
         for (int t0 = 0; t0 < n; t0 += blockDim.x >> 3) {
             const int tt = t0 + (threadIdx.x >> 3);
@@ -459,14 +488,22 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
                 const float4* k4 = reinterpret_cast<const float4*>(sk + tt * DP);
                 const float4* q4 = reinterpret_cast<const float4*>(sq + tt * DP);
                 for (int i = threadIdx.x & 7; i < DP / 4; i += 8) {
-                    const float4 a = k4[i], b = q4[i];
+                    float4 a = k4[i];
+                    const float4 b = q4[i];
+                    if (CHANNEL) {
+                        const float4 u = reinterpret_cast<const float4*>(sbonus)[i];
+                        a.x *= u.x; a.y *= u.y; a.z *= u.z; a.w *= u.w;
+                    }
                     c += a.x * b.x + a.y * b.y + a.z * b.z + a.w * b.w;
                 }
             }
             c += __shfl_xor_sync(0xffffffffu, c, 1);
             c += __shfl_xor_sync(0xffffffffu, c, 2);
             c += __shfl_xor_sync(0xffffffffu, c, 4);
-            if (tt < n && (threadIdx.x & 7) == 0) sgbc[4 * tt + 2] = c;
+            if (tt < n && (threadIdx.x & 7) == 0) {
+                if (RULE == SCAN_SCALAR) c = sgbc[4 * tt + 1] * c + own_skip;
+                sgbc[4 * tt + 2] = c;
+            }
         }
         __syncthreads();
 #pragma unroll 2
@@ -495,11 +532,24 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
                 if (DELTA) a += __shfl_xor_sync(0xffffffffu, a, off);
                 b += __shfl_xor_sync(0xffffffffu, b, off);
             }
-            float u = live ? sv[tt * CB + jl] : 0.f;
-            if (DELTA) u = gbc.y * (u - gt * a);
+            const float vt = live ? sv[tt * CB + jl] : 0.f;
+            if (CHANNEL) {
+                const float4* wt = kt + chunk * (DP / 4);
 #pragma unroll
-            for (int i = 0; i < DPER; ++i) S[i] = S[i] * gt + kk[i] * u;
-            if (live && part == 0) *op = gt * b + u * c;
+                for (int i4 = 0; i4 < DPER / 4; ++i4) {
+                    const float4 w4 = wt[i4 * PARTS];
+                    S[4 * i4] = S[4 * i4] * w4.x + kk[4 * i4] * vt;
+                    S[4 * i4 + 1] = S[4 * i4 + 1] * w4.y + kk[4 * i4 + 1] * vt;
+                    S[4 * i4 + 2] = S[4 * i4 + 2] * w4.z + kk[4 * i4 + 2] * vt;
+                    S[4 * i4 + 3] = S[4 * i4 + 3] * w4.w + kk[4 * i4 + 3] * vt;
+                }
+                if (live && part == 0) *op = b + vt * c;
+            } else {
+                const float u = DELTA ? gbc.y * (vt - gt * a) : gbc.y * vt;
+#pragma unroll
+                for (int i = 0; i < DPER; ++i) S[i] = S[i] * gt + kk[i] * u;
+                if (live && part == 0) *op = gt * b + (DELTA ? u : vt) * c;
+            }
             op += ostep;
         }
     }
@@ -523,12 +573,16 @@ static int rg_scan_rows_override = 0;
 extern "C" void rg_state_scan_rows(int rows) { rg_scan_rows_override = rows; }
 
 extern "C" int rg_state_scan(const float* q, int q_ld, const float* k, int k_ld, const void* v, int v_dtype, int v_ld,
-                             const float* decay, const float* g, const float* beta, float* state,
+                             const float* decay, const float* g, const float* beta, const float* skip,
+                             const float* w, int w_ld, const float* bonus, int rule, float* state,
                              const int* cu_seqlens, const int* start_pos, const int* slots, float* o, int R, int H,
                              int Hqk, int d, int dv, void* stream) {
     if (R <= 0) return 0;
-    if (H < 1 || Hqk < 1 || H % Hqk || d < 1 || dv < 1 || d > 256 || (!decay && !g) || (beta && !g))
+    if (H < 1 || Hqk < 1 || H % Hqk || d < 1 || dv < 1 || d > 256 || rule < SCAN_SCALAR || rule > SCAN_CHANNEL)
         return RG_ERR_UNSUPPORTED;
+    if (rule == SCAN_CHANNEL ? (!w || !bonus || decay || g || beta || skip) : (w || bonus || (!decay && !g) || (beta && !g)))
+        return RG_ERR_UNSUPPORTED;
+    if (rule == SCAN_DELTA && (!beta || skip)) return RG_ERR_UNSUPPORTED;
     // Rows of S per thread: 8 up to d = 64, then 16, then 32; `parts` (a power of two) threads share a column, and a
     // block of at most SCAN_THREADS threads takes CB columns.  While that gives fewer blocks than SMs (a long prompt
     // alone), threads take half as many rows each, down to 8 (measured, one prompt of 4,096 tokens, 16 heads of
@@ -560,17 +614,23 @@ extern "C" int rg_state_scan(const float* q, int q_ld, const float* k, int k_ld,
     int chunk = DP > 128 ? 8 : 16;
     if (chunk > 4 * parts) chunk = 4 * parts;                      // what a thread prefetches of v stays in 4 registers
     if (chunk * CB > SCAN_MAX_PREFETCH * threads) return RG_ERR_UNSUPPORTED;
-    const size_t smem = (size_t)2 * chunk * (2 * DP + CB + 4) * sizeof(float);
+    const bool channel = rule == SCAN_CHANNEL;
+    auto smem_of = [&](int c) {
+        return ((size_t)2 * c * ((channel ? 3 : 2) * DP + CB + 4) + (channel ? DP : 0)) * sizeof(float);
+    };
+    while (chunk > 1 && smem_of(chunk) > 48 * 1024) chunk >>= 1;
+    const size_t smem = smem_of(chunk);
     if (smem > 48 * 1024 || H > 65535 || col_blocks > 65535) return RG_ERR_UNSUPPORTED;
     // 16-byte copies and state accesses where every row starts on a 16-byte boundary
     const int vec = d % 4 == 0 && q_ld % 4 == 0 && k_ld % 4 == 0 && ((uintptr_t)q & 15) == 0 && ((uintptr_t)k & 15) == 0 &&
-                    ((uintptr_t)state & 15) == 0;
+                    ((uintptr_t)state & 15) == 0 && (!w || (w_ld % 4 == 0 && ((uintptr_t)w & 15) == 0));
     cudaStream_t s = (cudaStream_t)stream;
     dim3 grid(R, H, col_blocks);
 #define SM_SCAN(DP_, PA_, DE_, V) return rg_launch(state_scan_kernel<DP_, PA_, DE_, V>, grid, dim3(threads), smem, s, 1, \
-        q, q_ld, k, k_ld, (const V*)v, v_ld, decay, g, beta, state, cu_seqlens, start_pos, slots, o, H, Hqk, d, dv, CB, \
+        q, q_ld, k, k_ld, (const V*)v, v_ld, decay, g, beta, skip, w, w_ld, bonus, state, cu_seqlens, start_pos, slots, o, H, Hqk, d, dv, CB, \
         chunk, vec)
-#define SM_SCAN_RULE(DP_, PA_, V) { if (beta) SM_SCAN(DP_, PA_, true, V); SM_SCAN(DP_, PA_, false, V); }
+#define SM_SCAN_RULE(DP_, PA_, V) { if (rule == SCAN_DELTA) SM_SCAN(DP_, PA_, SCAN_DELTA, V); \
+        if (rule == SCAN_CHANNEL) SM_SCAN(DP_, PA_, SCAN_CHANNEL, V); SM_SCAN(DP_, PA_, SCAN_SCALAR, V); }
 #define SM_SCAN_PARTS(DP_, V) switch (parts) { \
         case 1: SM_SCAN_RULE(DP_, 1, V) case 2: SM_SCAN_RULE(DP_, 2, V) case 4: SM_SCAN_RULE(DP_, 4, V) \
         case 8: SM_SCAN_RULE(DP_, 8, V) case 16: if (DP_ <= 16) SM_SCAN_RULE(DP_ <= 16 ? DP_ : 16, 16, V) break; \
@@ -588,12 +648,12 @@ extern "C" int rg_state_scan(const float* q, int q_ld, const float* k, int k_ld,
 }
 
 // o [T, H, dv] float; gate: rows gate_ld apart (type A), head h at column gate_off + h dv; weight [dv] or null.
-// out [T, H dv] (type A) = o / sqrt(mean(o^2) + eps) * weight * silu(gate) (gate_kind 1: sigmoid(gate)).  One warp
-// per (token, head).
+// out (rows out_ld apart) = o / sqrt(mean(o^2) + eps) * weight * silu(gate) (gate_kind 1: sigmoid(gate)) * out_scale.
+// weight_step: 0 for one weight [dv] for all heads, dv for a weight per head [H, dv].  One warp per (token, head).
 template <typename A, typename O>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, const A* __restrict__ gate, int gate_ld, int gate_off,
-                                      const float* __restrict__ weight, float eps, O* __restrict__ out, int T, int H,
-                                      int dv, int gate_kind) {
+                                      const float* __restrict__ weight, int weight_step, float eps, O* __restrict__ out,
+                                      int out_ld, float out_scale, int T, int H, int dv, int gate_kind) {
     pdl_wait();
     pdl_trigger();
     const int lane = threadIdx.x & 31;
@@ -606,18 +666,20 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const A* __re
     ss = warp_sum(ss);
     const float inv = rsqrtf(ss / (float)dv + eps);
     const A* grow = gate + (size_t)t * gate_ld + gate_off + (size_t)h * dv;
+    const float* wrow = weight ? weight + (size_t)h * weight_step : nullptr;
+    O* dst = out + (size_t)t * out_ld + (size_t)h * dv;
     for (int i = lane; i < dv; i += 32) {
         const float z = to_f32(grow[i]);
-        out[(size_t)idx * dv + i] = from_f32<O>(src[i] * inv * (weight ? weight[i] : 1.f) *
-                                                (gate_kind ? sm_sigmoid(z) : z * sm_sigmoid(z)));
+        dst[i] = from_f32<O>(src[i] * inv * (wrow ? wrow[i] : 1.f) *
+                             (gate_kind ? sm_sigmoid(z) : z * sm_sigmoid(z)) * out_scale);
     }
 }
 
 // The same with ONE root mean square over all H dv numbers of a token and a weight of that size: one block per token.
 template <typename A, typename O>
 __global__ void row_norm_gate_kernel(const float* __restrict__ o, const A* __restrict__ gate, int gate_ld, int gate_off,
-                                     const float* __restrict__ weight, float eps, O* __restrict__ out, int n,
-                                     int gate_kind) {
+                                     const float* __restrict__ weight, float eps, O* __restrict__ out, int out_ld,
+                                     float out_scale, int n, int gate_kind) {
     __shared__ float scratch[33];
     pdl_wait();
     pdl_trigger();
@@ -630,17 +692,19 @@ __global__ void row_norm_gate_kernel(const float* __restrict__ o, const A* __res
     const A* grow = gate + (size_t)t * gate_ld + gate_off;
     for (int i = threadIdx.x; i < n; i += blockDim.x) {
         const float z = to_f32(grow[i]);
-        out[(size_t)t * n + i] = from_f32<O>(src[i] * inv * (weight ? weight[i] : 1.f) *
-                                             (gate_kind ? sm_sigmoid(z) : z * sm_sigmoid(z)));
+        out[(size_t)t * out_ld + i] = from_f32<O>(src[i] * inv * (weight ? weight[i] : 1.f) *
+                                                  (gate_kind ? sm_sigmoid(z) : z * sm_sigmoid(z)) * out_scale);
     }
 }
 
-// whole 0: every head normed on its own (weight [dv]); 1: all heads of a token together (weight [H dv]).
+// whole 0: every head normed on its own (weight [dv]; with weight_step dv: [H, dv]); 1: all heads of a token together
+// (weight [H dv]).
 // gate_kind 0: silu(gate); 1: sigmoid(gate).
 extern "C" int rg_head_norm_gate(const float* o, const void* gate, int gate_dtype, int gate_ld, int gate_off,
-                                 const float* weight, float eps, void* out, int out_dtype, int T, int H, int dv,
-                                 int whole, int gate_kind, void* stream) {
+                                 const float* weight, int weight_step, float eps, void* out, int out_dtype, int out_ld,
+                                 float out_scale, int T, int H, int dv, int whole, int gate_kind, void* stream) {
     if (T <= 0) return 0;
+    if ((weight_step != 0 && weight_step != dv) || out_ld < H * dv) return RG_ERR_UNSUPPORTED;
     if (gate_kind < 0 || gate_kind > 1) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const long long n = (long long)T * H;
@@ -648,9 +712,9 @@ extern "C" int rg_head_norm_gate(const float* o, const void* gate, int gate_dtyp
     const int row = H * dv;
     const int threads = row >= 1024 ? 256 : 128;
 #define SM_HNG(A, O) { if (whole) return rg_launch(row_norm_gate_kernel<A, O>, dim3(T), dim3(threads), 0, s, 1, o, \
-        (const A*)gate, gate_ld, gate_off, weight, eps, (O*)out, row, gate_kind); \
+        (const A*)gate, gate_ld, gate_off, weight, eps, (O*)out, out_ld, out_scale, row, gate_kind); \
         return rg_launch(head_norm_gate_kernel<A, O>, grid, dim3(128), 0, s, 1, o, (const A*)gate, gate_ld, \
-        gate_off, weight, eps, (O*)out, T, H, dv, gate_kind); }
+        gate_off, weight, weight_step, eps, (O*)out, out_ld, out_scale, T, H, dv, gate_kind); }
     if (gate_dtype == RG_DTYPE_BF16 && out_dtype == RG_DTYPE_BF16) SM_HNG(bf16, bf16)
     if (gate_dtype == RG_DTYPE_F32 && out_dtype == RG_DTYPE_F32) SM_HNG(float, float)
     if (gate_dtype == RG_DTYPE_F32 && out_dtype == RG_DTYPE_BF16) SM_HNG(float, bf16)

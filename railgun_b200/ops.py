@@ -875,12 +875,12 @@ def recurrent_scan(proj: torch.Tensor, y_off: int, x_off: int, yb, xb, u: torch.
 # ---- short convolutions with state, matrix-state mixers (retention, delta rule), attention's per-token work -------
 
 def causal_conv(x: torch.Tensor, x_off: int, taps: torch.Tensor, state, batch, out_dtype, residual: bool = False,
-                silu: bool = False, out: torch.Tensor | None = None) -> torch.Tensor:
+                silu: bool = False, out: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> torch.Tensor:
     """[T, C]: per channel the causal convolution of x[:, x_off:x_off + C] with ``taps`` [K, C] (tap-major: what the
     tensor files hold as [C, K], transposed once at load; last row: the
     current token's) along each request's tokens, continued from the K - 1 inputs in the request's state slot
     (``state`` [slots, K - 1, C] float32; None when K = 1) unless the request starts at position 0.  ``silu``:
-    the activation on the convolution; ``residual``: x is added.  32-bit arithmetic, one rounding into
+    the activation on the convolution (and its ``bias`` [C], if there is one); ``residual``: x is added.  32-bit arithmetic, one rounding into
     ``out_dtype``.  The state is not changed (``conv_state_update`` does that, afterwards)."""
     _check_rows(x, "x")
     _check(taps, "taps", torch.float32)
@@ -892,12 +892,16 @@ def causal_conv(x: torch.Tensor, x_off: int, taps: torch.Tensor, state, batch, o
         _check(state, "state", torch.float32)
         if tuple(state.shape[1:]) != (K - 1, C):
             raise KernelError(f"causal_conv: state {tuple(state.shape)} is not [slots, {K - 1}, {C}]")
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+        if bias.numel() != C:
+            raise KernelError(f"causal_conv: bias has {bias.numel()} elements, expected {C}")
     if out is None:
         out = torch.empty((T, C), dtype=out_dtype, device=x.device)
     _check_out_view(out, T, C, out_dtype, "causal_conv")
     _ok(_fn("state_mixers", "rg_causal_conv")(
-        _ptr(x), c_int(_dtype_code(x)), c_int(x.stride(0)), c_int(x_off), _ptr(taps), _ptr(state if K > 1 else None),
-        _ptr(batch.cu_seqlens), _ptr(batch.req_of_token), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(out),
+        _ptr(x), c_int(_dtype_code(x)), c_int(x.stride(0)), c_int(x_off), _ptr(taps), _ptr(bias),
+        _ptr(state if K > 1 else None), _ptr(batch.cu_seqlens), _ptr(batch.req_of_token), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(out),
         c_int(_dtype_code(out)), c_int(out.stride(0)), c_int(T), c_int(C), c_int(K), c_int(1 if residual else 0),
         c_int(1 if silu else 0), _stream()), "causal_conv")
     return out
@@ -965,15 +969,27 @@ def delta_prepare(qkv: torch.Tensor, G: int, d: int, q_scale: float, unit_eps: f
     return beta, g
 
 
+SCAN_RULES = {"scalar": 0, "delta": 1, "channel": 2}
+
+
 def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, batch, H: int, d: int, dv: int,
                decay: torch.Tensor | None = None, g: torch.Tensor | None = None,
-               beta: torch.Tensor | None = None) -> torch.Tensor:
+               beta: torch.Tensor | None = None, rule: str | None = None, skip: torch.Tensor | None = None,
+               w: torch.Tensor | None = None, bonus: torch.Tensor | None = None) -> torch.Tensor:
     """A matrix S [d, dv] per head carried along each request's tokens, 32-bit, from the request's slot of ``state``
-    [slots, H, dv, d] (S transposed; zeros at position 0) and left there.  With ``decay`` [H]: S <- decay_h S + k v^T; with ``g``
-    and ``beta`` [T, H]: S <- g S, u = beta (v - S^T k), S <- S + k u^T.  Either way o = S^T q after the update.
+    [slots, H, dv, d] (S transposed; zeros at position 0) and left there.  ``rule``:
+      "scalar"   S <- g S + beta k v^T, o = S^T q + skip_h v, with ``decay`` [H] or ``g`` [T, H], ``beta`` [T, H]
+                 (default 1) and ``skip`` [H] (default 0);
+      "delta"    S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q, with ``g`` and ``beta`` [T, H];
+      "channel"  o = (S + diag(bonus_h) k v^T)^T q, then S <- diag(w_t) S + k v^T, with ``w`` (float32 [T, H * d] view)
+                 and ``bonus`` [H, d].
+    By default "delta" when ``beta`` is given, else "scalar".
     ``q``, ``k``: float32 [T, Hqk * d] views (head h reads head h / (H / Hqk)); ``v``: [T, H * dv] view, float32 or
     bfloat16.
     Returns o [T, H, dv] float32."""
+    rule = rule or ("delta" if beta is not None else "scalar")
+    if rule not in SCAN_RULES:
+        raise KernelError(f"state_scan: rule {rule!r} is not known; known: {sorted(SCAN_RULES)}")
     for t, name in ((q, "q"), (k, "k")):
         _check_rows(t, name, torch.float32)
     _check_rows(v, "v")
@@ -984,19 +1000,28 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
             or tuple(state.shape[1:]) != (H, dv, d):
         raise KernelError(f"state_scan: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)}, state "
                           f"{tuple(state.shape)} do not match {H} heads of {d} x {dv}")
-    for t, name, n in ((decay, "decay", H), (g, "g", T * H), (beta, "beta", T * H)):
+    for t, name, n in ((decay, "decay", H), (g, "g", T * H), (beta, "beta", T * H), (skip, "skip", H),
+                       (bonus, "bonus", H * d)):
         if t is not None:
             _check(t, name, torch.float32)
             if t.numel() != n:
                 raise KernelError(f"state_scan: {name} has {t.numel()} elements, expected {n}")
-    if (decay is None) == (g is None) or (beta is not None and g is None):
-        raise KernelError("state_scan: a fixed decay per head, or g and beta per token")
+    if rule == "channel":
+        if w is None or bonus is None or any(t is not None for t in (decay, g, beta, skip)):
+            raise KernelError("state_scan: the channel rule takes w and bonus, and nothing of the other rules")
+        _check_rows(w, "w", torch.float32)
+        if w.shape != (T, H * d):
+            raise KernelError(f"state_scan: w {tuple(w.shape)} is not [{T}, {H * d}]")
+    elif (decay is None) == (g is None) or (beta is not None and g is None) or w is not None or bonus is not None \
+            or (rule == "delta" and (beta is None or skip is not None)):
+        raise KernelError("state_scan: a fixed decay per head, or g (and beta) per token")
     o = torch.empty((T, H, dv), dtype=torch.float32, device=q.device)
     _ok(_fn("state_mixers", "rg_state_scan")(
         _ptr(q), c_int(q.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(_dtype_code(v)), c_int(v.stride(0)),
         _ptr(decay), _ptr(g),
-        _ptr(beta), _ptr(state), _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(o),
-        c_int(batch.num_requests), c_int(H), c_int(Hqk), c_int(d), c_int(dv), _stream()), "state_scan")
+        _ptr(beta), _ptr(skip), _ptr(w), c_int(w.stride(0) if w is not None else 0), _ptr(bonus),
+        c_int(SCAN_RULES[rule]), _ptr(state), _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots),
+        _ptr(o), c_int(batch.num_requests), c_int(H), c_int(Hqk), c_int(d), c_int(dv), _stream()), "state_scan")
     return o
 
 
@@ -1010,11 +1035,11 @@ HEAD_GATES = {"silu": 0, "sigmoid": 1}
 
 
 def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight, eps: float, out_dtype, whole: bool = False,
-                   gate_kind: str = "silu") -> torch.Tensor:
+                   gate_kind: str = "silu", out: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
     """[T, H dv] in ``out_dtype``: every head of ``o`` [T, H, dv] (float32) divided by its root mean square (``eps``
-    inside the root), times ``weight`` [dv] (None: no weight), times silu(``gate``) ([T, H dv] view) or, with
+    inside the root), times ``weight`` ([dv] for all heads or [H dv]; None: no weight), times silu(``gate``) ([T, H dv] view) or, with
     ``gate_kind`` "sigmoid", sigmoid(``gate``).  ``whole``: one root mean square over all H dv numbers of a token
-    and a weight of that size."""
+    and a weight of that size.  Everything times ``out_scale``; ``out``: a view to write into."""
     _check(o, "o", torch.float32)
     _check_rows(gate, "gate")
     T, H, dv = o.shape
@@ -1024,15 +1049,191 @@ def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight, eps: float, out_
         raise KernelError(f"head_norm_gate: gate {gate_kind!r} is not known; known: {sorted(HEAD_GATES)}")
     if weight is not None:
         _check(weight, "weight", torch.float32)
-        if weight.numel() != (H * dv if whole else dv):
+        if weight.numel() != H * dv and (whole or weight.numel() != dv):
             raise KernelError(f"head_norm_gate: weight has {weight.numel()} elements, expected "
                               f"{H * dv if whole else dv}")
-    out = torch.empty((T, H * dv), dtype=out_dtype, device=o.device)
+    if out is None:
+        out = torch.empty((T, H * dv), dtype=out_dtype, device=o.device)
+    _check_out_view(out, T, H * dv, out_dtype, "head_norm_gate")
+    step = dv if weight is not None and not whole and weight.numel() == H * dv and H > 1 else 0
     _ok(_fn("state_mixers", "rg_head_norm_gate")(
-        _ptr(o), _ptr(gate), c_int(_dtype_code(gate)), c_int(gate.stride(0)), c_int(0), _ptr(weight), c_float(eps),
-        _ptr(out), c_int(_dtype_code(out)), c_int(T), c_int(H), c_int(dv), c_int(1 if whole else 0),
+        _ptr(o), _ptr(gate), c_int(_dtype_code(gate)), c_int(gate.stride(0)), c_int(0), _ptr(weight), c_int(step),
+        c_float(eps), _ptr(out), c_int(_dtype_code(out)), c_int(out.stride(0)), c_float(out_scale), c_int(T), c_int(H), c_int(dv), c_int(1 if whole else 0),
         c_int(HEAD_GATES[gate_kind]), _stream()), "head_norm_gate")
     return out
+
+
+# ---- token shift, Mamba-2 around its scan, RWKV-style time mixing around its scan -----------------------------------
+
+def postnorm_shift(resid: torch.Tensor, pending, shift, state, batch, out_dtype):
+    """(new stream, h): the stream rows x = resid + what is pending (a ``PendingNormed``: its output normed; a tensor:
+    as it is; None), in 32-bit, and h = x + (x' - x) ``shift`` in ``out_dtype``, x' the row of the request's previous
+    token: the row before in the step, at the step's first row the one kept in the request's slot of ``state``
+    [slots, 1, H] float32 (zeros at position 0), where the step's last row is left.  The new stream is another tensor
+    (``resid`` stays as it was).  With ``shift`` None h is x itself, the stream is changed in place and ``state`` and
+    ``batch`` are not used."""
+    _check(resid, "resid", torch.float32)
+    T, H = resid.shape
+    post_w, post_eps, y = None, 0.0, pending
+    if isinstance(pending, PendingNormed):
+        post_w, post_eps, y = pending.weight, pending.eps, pending.y
+        _check(post_w, "post-norm weight", torch.float32)
+        if post_w.numel() != H:
+            raise KernelError(f"post-norm weight has {post_w.numel()} elements, rows have {H}")
+    if y is not None:
+        _check(y, "pending")
+        if y.shape != resid.shape:
+            raise KernelError(f"pending {tuple(y.shape)} vs residual {tuple(resid.shape)}")
+    out = torch.empty((T, H), dtype=out_dtype, device=resid.device)
+    new, rows = resid, 1
+    if shift is not None:
+        _check(shift, "shift", torch.float32)
+        _check(state, "state", torch.float32)
+        if shift.numel() != H or state[0].numel() != H:
+            raise KernelError(f"postnorm_shift: shift {tuple(shift.shape)} or state {tuple(state.shape)} vs rows of {H}")
+        new = torch.empty_like(resid)
+        # every block works out the row before its first one again: several rows per block once there are plenty
+        rows = SHIFT_ROWS_PER_BLOCK if T >= 148 * 4 * SHIFT_ROWS_PER_BLOCK else 1
+    none = lambda t: _ptr(t if shift is not None else None)
+    _ok(_fn("token_shift", "rg_postnorm_shift")(
+        _ptr(resid), _ptr(y), c_int(_dtype_code(y) if y is not None else 0), _ptr(post_w), c_float(post_eps),
+        _ptr(shift), none(state), none(batch.cu_seqlens if shift is not None else None),
+        none(batch.req_of_token if shift is not None else None), none(batch.start_pos if shift is not None else None),
+        none(batch.state_slots if shift is not None else None), _ptr(new), _ptr(out), c_int(_dtype_code(out)), c_int(T),
+        c_int(H), c_int(rows), _stream()), "postnorm_shift")
+    return new, out
+
+
+SHIFT_ROWS_PER_BLOCK = 4
+
+
+def shift_mixes(h: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, batch):
+    """Five mixes h + (h' - h) mu[s] of every row with the row of the request's previous token (``mu`` [5, H] float32;
+    ``state`` [slots, 1, H] float32 keeps the last row of ``h`` between steps).  Returns (mixes [4, T, H] of mu[0..3] in
+    h's type, last: mu[4] in 32-bit, [T, H] float32 for float32 rows, else [T, 2 H] bfloat16 as hi | lo, the two halves
+    of the 32-bit number)."""
+    _check(h, "h")
+    _check(mu, "mu", torch.float32)
+    _check(state, "state", torch.float32)
+    T, H = h.shape
+    if tuple(mu.shape) != (5, H) or state[0].numel() != H:
+        raise KernelError(f"shift_mixes: mu {tuple(mu.shape)} or state {tuple(state.shape)} does not match rows of {H}")
+    mixes = torch.empty((4, T, H), dtype=h.dtype, device=h.device)
+    last = torch.empty((T, H if h.dtype == torch.float32 else 2 * H), dtype=h.dtype, device=h.device)
+    _ok(_fn("token_shift", "rg_shift_mixes")(
+        _ptr(h), c_int(_dtype_code(h)), _ptr(mu), _ptr(state), _ptr(batch.cu_seqlens), _ptr(batch.req_of_token),
+        _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(mixes), _ptr(last), c_int(T), c_int(H), _stream()),
+        "shift_mixes")
+    return mixes, last
+
+
+def lowrank_decay(a: torch.Tensor, w: torch.Tensor, w0: torch.Tensor) -> torch.Tensor:
+    """float32 [T, N] = exp(-exp(tanh(a) w^T + w0)), ``a`` float32 [T, rank], ``w`` [N, rank], all in 32-bit."""
+    _check(a, "a", torch.float32)
+    _check(w, "w")
+    _check(w0, "w0", torch.float32)
+    (T, rank), N = a.shape, w.shape[0]
+    if w.shape[1] != rank or w0.numel() != N:
+        raise KernelError(f"lowrank_decay: a {tuple(a.shape)}, w {tuple(w.shape)}, w0 {tuple(w0.shape)} do not match")
+    out = torch.empty((T, N), dtype=torch.float32, device=a.device)
+    _ok(_fn("token_shift", "rg_lowrank_decay")(_ptr(a), _ptr(w), c_int(_dtype_code(w)), _ptr(w0), _ptr(out), c_int(T),
+                                               c_int(N), c_int(rank), _stream()), "lowrank_decay")
+    return out
+
+
+def ssd_prepare(raw: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor):
+    """(dt, g), both float32 [T, H]: dt = softplus(raw + dt_bias), g = exp(-exp(A_log) dt); ``raw``: float32 [T, H] view."""
+    _check_rows(raw, "raw", torch.float32)
+    T, H = raw.shape
+    for t, name in ((dt_bias, "dt_bias"), (A_log, "A_log")):
+        _check(t, name, torch.float32)
+        if t.numel() != H:
+            raise KernelError(f"ssd_prepare: {name} has {t.numel()} elements, expected {H}")
+    dt = torch.empty((T, H), dtype=torch.float32, device=raw.device)
+    g = torch.empty((T, H), dtype=torch.float32, device=raw.device)
+    _ok(_fn("ssd", "rg_ssd_prepare")(_ptr(raw), c_int(raw.stride(0)), _ptr(dt_bias), _ptr(A_log), _ptr(dt), _ptr(g),
+                                     c_int(T), c_int(H), _stream()), "ssd_prepare")
+    return dt, g
+
+
+def ssd_step(proj: torch.Tensor, x_off: int, dt_off: int, taps: torch.Tensor, bias, conv_state, dt_bias: torch.Tensor,
+             A_log: torch.Tensor, D: torch.Tensor, state: torch.Tensor, batch, H: int, G: int, N: int, dv: int):
+    """One token per request (rows of ``proj``, float32: x | B | C from column ``x_off``, the raw step sizes at
+    ``dt_off``): the causal convolution (``taps`` [K, C], ``bias`` [C]) with silu on x, B and C continued from
+    ``conv_state`` [slots, K - 1, C], and one step S <- g S + dt B x^T, o = S^T C + D x of every head from and into
+    ``state`` [slots, H, dv, N] (S transposed).  Returns o [T, H, dv] float32.  The convolution's state is left as it
+    is: ``gate_group_norm`` moves it on."""
+    _check_rows(proj, "proj", torch.float32)
+    K, C = taps.shape
+    T = proj.shape[0]
+    for t, name in ((taps, "taps"), (dt_bias, "dt_bias"), (A_log, "A_log"), (D, "D"), (state, "state")):
+        _check(t, name, torch.float32)
+    if bias is not None:
+        _check(bias, "bias", torch.float32)
+    if K > 1:
+        _check(conv_state, "conv_state", torch.float32)
+    if C != H * dv + 2 * G * N or proj.shape[1] < max(x_off + C, dt_off + H) or tuple(state.shape[1:]) != (H, dv, N) \
+            or (K > 1 and tuple(conv_state.shape[1:]) != (K - 1, C)) or (bias is not None and bias.numel() != C) \
+            or any(t.numel() != H for t in (dt_bias, A_log, D)) or batch.num_requests != T:
+        raise KernelError("ssd_step: sizes do not match, or a request brings more than one token")
+    o = torch.empty((T, H, dv), dtype=torch.float32, device=proj.device)
+    _ok(_fn("ssd", "rg_ssd_step")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(x_off), c_int(dt_off), _ptr(taps), _ptr(bias),
+        _ptr(conv_state if K > 1 else None), _ptr(dt_bias), _ptr(A_log), _ptr(D), _ptr(state), _ptr(batch.req_of_token),
+        _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(o), c_int(T), c_int(H), c_int(G), c_int(N), c_int(dv),
+        c_int(K), _stream()), "ssd_step")
+    return o
+
+
+def gate_group_norm(o: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, out_dtype,
+                    conv=None, batch=None) -> torch.Tensor:
+    """[T, n] in ``out_dtype``: o silu(z) cut into ``groups`` equal parts, each divided by its own root mean square
+    (``eps`` inside the root), times ``weight`` [n].  ``o`` float32 (n numbers per token), ``z`` a [T, n] view.
+    ``conv`` = (rows [T, C] float32 view, state [slots, K - 1, C]): also moves the convolution state of every request on
+    by its one token of the step."""
+    _check(o, "o", torch.float32)
+    _check_rows(z, "z")
+    _check(weight, "weight", torch.float32)
+    T, n = z.shape
+    if o.numel() != T * n or weight.numel() != n or groups < 1 or n % groups:
+        raise KernelError(f"gate_group_norm: o {tuple(o.shape)}, z {tuple(z.shape)}, {groups} groups do not match")
+    raw, state = conv if conv is not None else (None, None)
+    C, K = 0, 1
+    if raw is not None and state is not None:
+        _check_rows(raw, "rows", torch.float32)
+        _check(state, "state", torch.float32)
+        C, K = state.shape[2], state.shape[1] + 1
+        if raw.shape != (T, C) or batch.num_requests != T:
+            raise KernelError("gate_group_norm: the convolution's rows do not match its state")
+    else:
+        raw = None
+    out = torch.empty((T, n), dtype=out_dtype, device=o.device)
+    who = lambda t: _ptr(t if raw is not None else None)
+    _ok(_fn("ssd", "rg_gate_group_norm")(
+        _ptr(o), _ptr(z), c_int(_dtype_code(z)), c_int(z.stride(0)), _ptr(weight), c_float(eps), _ptr(out),
+        c_int(_dtype_code(out)), c_int(T), c_int(n), c_int(groups), _ptr(raw), c_int(raw.stride(0) if raw is not None else 0),
+        who(state), who(batch.req_of_token if raw is not None else None), who(batch.start_pos if raw is not None else None),
+        who(batch.state_slots if raw is not None else None), c_int(C), c_int(K), _stream()), "gate_group_norm")
+    return out
+
+
+def pool_blocks(kv_cache: torch.Tensor, block_table: torch.Tensor, batch, slots: torch.Tensor, entries: torch.Tensor,
+                pool: int) -> None:
+    """For every token of the step that ends a block of ``pool`` tokens of its request (positions b pool ..
+    (b + 1) pool - 1): the mean of the block's keys and of its values, as ``kv_cache`` [pages, 2, G, page, D] holds
+    them, into the block's entry of ``entries`` (pages of the same shape, an entry for a token).  ``slots``: the
+    entries' group's slot of each token, which counts tokens (the entry is slot / pool; negative: no write)."""
+    _check(kv_cache, "kv_cache")
+    _check(entries, "entries", kv_cache.dtype)
+    _check(block_table, "block_table", torch.int32)
+    _check(slots, "slots", torch.int32)
+    if entries.shape[1:] != kv_cache.shape[1:] or pool < 1:
+        raise KernelError(f"pool_blocks: entries {tuple(entries.shape)} vs tokens {tuple(kv_cache.shape)}")
+    _, _, G, page, D = kv_cache.shape
+    _ok(_fn("attention_pool", "rg_pool_blocks")(
+        _ptr(kv_cache), c_int(_dtype_code(kv_cache)), _ptr(block_table), c_int(block_table.shape[1]),
+        _ptr(batch.req_of_token), _ptr(batch.positions), _ptr(slots), _ptr(entries), c_int(slots.numel()), c_int(G),
+        c_int(page), c_int(D), c_int(pool), _stream()), "pool_blocks")
 
 
 def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, freq: torch.Tensor, rot_dims: int,
@@ -1079,6 +1280,20 @@ def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, f
         c_int(temp_every), c_int(T), c_int(H), c_int(G), c_int(d), c_int(dv), c_int(D),
         c_int(page_size), _stream()), "attention_prepare")
     return q
+
+
+def _pooled(pooled, kv_cache, window, keep_first):
+    """Checks of the attention kernels' optional ``pooled`` = (entries, block table, pool): pages of the tokens' shape
+    whose entry b stands for the positions b pool .. (b + 1) pool - 1 of a request, seen, beside the window, by the
+    queries at positions p with (b + 1) pool - 1 <= p - window.  Returns the launcher's four arguments."""
+    if pooled is None:
+        return (_ptr(None), _ptr(None), c_int(0), c_int(0))
+    entries, table, pool = pooled
+    _check(entries, "entries", kv_cache.dtype)
+    _check(table, "entries' block table", torch.int32)
+    if entries.shape[1:] != kv_cache.shape[1:] or pool < 1 or not window or keep_first:
+        raise KernelError("pooled entries go with a window, with no kept first tokens, in pages of the tokens' shape")
+    return (_ptr(entries), _ptr(table), c_int(table.shape[1]), c_int(pool))
 
 
 def _sink_and_gate(sink, gate, nh: int, T: int, dtype):
@@ -1372,11 +1587,13 @@ def skinny_rope_ok(x, weight: torch.Tensor, d: int) -> bool:
 
 def paged_attention_general(q: torch.Tensor, q_stride: int, kv_cache: torch.Tensor, block_table: torch.Tensor,
                             req_of_token: torch.Tensor, positions: torch.Tensor, nh: int, nkv: int, d: int,
-                            window: int, scale: float, keep_first: int = 0, sink=None, gate=None) -> torch.Tensor:
+                            window: int, scale: float, keep_first: int = 0, sink=None, gate=None, pooled=None,
+                            out: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
     """The general attention kernel: out [T, nh*d].  ``q`` may be a view whose
     rows are ``q_stride`` elements apart (the q part of a fused qkv buffer).
     ``keep_first``: with a window, the first positions of a request that every
-    later query still sees.  ``sink``, ``gate``: see ``_sink_and_gate``."""
+    later query still sees.  ``sink``, ``gate``: see ``_sink_and_gate``; ``pooled``: see ``_pooled``; ``out``: a view
+    to write into; the output is multiplied by ``out_scale``."""
     if not q.is_cuda:
         raise KernelError("q must be a CUDA tensor (there is no CPU path)")
     _check(kv_cache, "kv_cache", q.dtype)
@@ -1389,13 +1606,16 @@ def paged_attention_general(q: torch.Tensor, q_stride: int, kv_cache: torch.Tens
         raise KernelError(f"kv cache shape {tuple(kv_cache.shape)} does not match heads {nkv} x {d}")
     if d > 256:
         raise KernelError(f"head size {d} is above the kernels' limit of 256")
-    out = torch.empty((T, nh * d), dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty((T, nh * d), dtype=q.dtype, device=q.device)
+    _check_out_view(out, T, nh * d, q.dtype, "paged_attention_general")
     gate_ld = _sink_and_gate(sink, gate, nh, T, q.dtype)
     _ok(_fn("attention_general", "rg_paged_attention_general")(
         _ptr(q), c_int(q_stride), _ptr(out), _ptr(kv_cache), c_int(_dtype_code(q)), _ptr(block_table),
         c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), c_int(T), c_int(nh), c_int(nkv),
         c_int(d), c_int(page_size), c_int(window or 0), c_float(scale), c_int(keep_first if window else 0),
-        _ptr(sink), _ptr(gate), c_int(gate_ld), _stream()),
+        _ptr(sink), _ptr(gate), c_int(gate_ld), *_pooled(pooled, kv_cache, window, keep_first), c_int(out.stride(0)),
+        c_float(out_scale), _stream()),
         "paged_attention_general")
     return out
 
@@ -1416,22 +1636,25 @@ def _check_paged(q, kv_cache, block_table, nkv, d):
 
 
 def prefill_attention(q, q_stride: int, out, kv_cache, block_table, tiles, positions, nh: int, nkv: int, d: int,
-                      window: int, scale: float, keep_first: int = 0, sink=None, gate=None) -> None:
+                      window: int, scale: float, keep_first: int = 0, sink=None, gate=None, pooled=None,
+                      out_scale: float = 1.0) -> None:
     """Flash-style attention for requests that bring several tokens: ``tiles``
     [n, 3] = (first row, rows <= 64, request index).  Writes the tiles' rows of
     ``out`` [T, nh*d].  ``keep_first``: with a window, the first positions of a
     request that every later query still sees.  ``sink``, ``gate``: see
-    ``_sink_and_gate``."""
+    ``_sink_and_gate``; ``pooled``: see ``_pooled``.  ``out`` may be a view
+    whose rows are further apart; the output is multiplied by ``out_scale``."""
     page_size = _check_paged(q, kv_cache, block_table, nkv, d)
     _check(tiles, "tiles", torch.int32)
     _check(positions, "positions", torch.int32)
-    _check(out, "out", q.dtype)
+    _check_out_view(out, out.shape[0], nh * d, q.dtype, "prefill_attention")
     gate_ld = _sink_and_gate(sink, gate, nh, out.shape[0], q.dtype)
     _ok(_fn("attention_mma", "rg_prefill_attention_sink")(
         _ptr(q), c_int(q_stride), _ptr(out), _ptr(kv_cache), _ptr(block_table), c_int(block_table.shape[1]),
         _ptr(tiles), c_int(tiles.shape[0]), _ptr(positions), c_int(nh), c_int(nkv), c_int(d), c_int(page_size),
         c_int(window or 0), c_int(keep_first if window else 0), c_float(scale), _ptr(sink), _ptr(gate), c_int(gate_ld),
-        _stream()), "prefill_attention")
+        *_pooled(pooled, kv_cache, window, keep_first), c_int(out.stride(0)), c_float(out_scale), _stream()),
+        "prefill_attention")
 
 
 def decode_splits(n_tokens: int, kv_tiles: int, max_context: int) -> int:
@@ -1450,7 +1673,7 @@ _decode_counters: dict = {}
 def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_tokens: int, req_of_token, positions,
                      nh: int, nkv: int, d: int, window: int, scale: float, num_splits: int,
                      scratch=None, fused_reduce=None, cluster: bool = False, keep_first: int = 0, sink=None,
-                     gate=None) -> None:
+                     gate=None, pooled=None, out_scale: float = 1.0) -> None:
     """Split attention for single tokens: token rows ``rows`` (None: rows
     0..n_tokens-1) each attend their request's context.  Partial results go
     through scratch memory (allocated here unless given) and are reduced into
@@ -1465,21 +1688,23 @@ def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_token
     ``keep_first``: with a window, the first positions of a request that every
     later query still sees (not with ``cluster``).  ``sink``, ``gate``: see
     ``_sink_and_gate``; they enter where the splits are added up (not with
-    ``cluster``)."""
+    ``cluster``).  ``pooled``: see ``_pooled`` (not with ``cluster``).  ``out``
+    may be a view whose rows are further apart; the output is multiplied by
+    ``out_scale`` (neither with ``cluster``)."""
     if fused_reduce is None:
         fused_reduce = num_splits == 1
     page_size = _check_paged(q, kv_cache, block_table, nkv, d)
     _check(req_of_token, "req_of_token", torch.int32)
     _check(positions, "positions", torch.int32)
-    _check(out, "out", q.dtype)
+    _check_out_view(out, out.shape[0], nh * d, q.dtype, "decode_attention")
     if rows is not None:
         _check(rows, "rows", torch.int32)
     gate_ld = _sink_and_gate(sink, gate, nh, out.shape[0], q.dtype)
     if cluster:
         if keep_first and window:
             raise KernelError("decode_attention: the cluster form does not keep first tokens")
-        if sink is not None or gate is not None:
-            raise KernelError("decode_attention: the cluster form has neither sink nor gate")
+        if sink is not None or gate is not None or pooled is not None or out_scale != 1.0 or not out.is_contiguous():
+            raise KernelError("decode_attention: the cluster form has neither sink, gate, pooled entries nor an output view")
         if not 2 <= num_splits <= 8:
             raise KernelError("decode_attention: a cluster takes 2 to 8 splits")
         _ok(_fn("attention_mma", "rg_decode_attention_cluster")(
@@ -1508,7 +1733,8 @@ def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_token
         _ptr(rows), c_int(n_tokens), _ptr(req_of_token), _ptr(positions), _ptr(part_o), _ptr(part_ml),
         _ptr(counters), c_int(nh), c_int(nkv), c_int(d), c_int(page_size), c_int(window or 0),
         c_int(keep_first if window else 0), c_float(scale), c_int(num_splits), _ptr(sink), _ptr(gate), c_int(gate_ld),
-        _stream()), "decode_attention")
+        *_pooled(pooled, kv_cache, window, keep_first), c_int(out.stride(0)), c_float(out_scale), _stream()),
+        "decode_attention")
 
 
 _tc_err: dict = {}

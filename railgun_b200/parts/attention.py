@@ -141,14 +141,18 @@ register_mixer("paged_attention", PagedAttention)
 
 class NormedAttention(Mixer):
     """Grouped-query softmax attention with the options that recent designs add to it, each a parameter:
-    biases on the four projections, an RMS norm on q and k before the rotation (per head, with one weight vector
-    for all q heads and one for all k heads, or over the whole of q and the whole of k with weights of that
-    size), a short causal convolution per channel on q, k and v directly behind the projections, rotation of
-    the first ``rot_dims`` numbers of a head in either layout, a learned number per head on the scores
+    biases on the four projections (or on q, k and v only), an RMS norm on q and k before the rotation (per head, with
+    one weight vector for all q heads and one for all k heads, or without weights, which is the same before and
+    after a rotation, or over the whole of q and the whole of k with weights of that size), a short causal convolution per channel on q, k and v directly behind the projections, rotation of
+    the first ``rot_dims`` numbers of a head in either layout, its frequencies divided by a constant (linear scaling),
+    a learned number per head on the scores
     (``head_temp``), a query factor that grows with the logarithm of the position (``q_temp``), a sink in the
     softmax's denominator (of score 0, or a learned score per head), a sigmoid gate per head on the heads'
     outputs, values of another size than keys, and a sliding window that keeps the request's first
-    ``keep_first`` tokens visible (at their true positions).
+    ``keep_first`` tokens visible (at their true positions) or, with ``pool``, sees what has left it as the means of
+    the keys and of the values of blocks of ``pool`` tokens that lie wholly before the window (in a second group of
+    pages, one entry per block, written by the step that completes the block; the tokens' pages are kept until their
+    block is complete).
 
     Keys, queries and values are padded with zeros to one size D (a multiple of 16 that holds both), so the
     key/value pages and the attention kernels are the ordinary ones; the output product's matrix gets zero
@@ -158,8 +162,10 @@ class NormedAttention(Mixer):
 
     params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``v_dim``, ``scale`` (None:
     head_dim^-1/2), ``rot_dims``, ``rot_base``, ``rot_layout`` ("interleaved": pairs (2i, 2i + 1), or "half":
-    pairs (i, i + rot_dims/2)), ``eps`` (of the q and k norms), ``window`` (0: none), ``keep_first``,
-    ``bias``, ``head_temp`` (booleans, default true), ``qk_norm`` (true, the default: per head; "whole"; false),
+    pairs (i, i + rot_dims/2)), ``rot_factor`` (what the frequencies are divided by, default 1), ``eps`` (of the q and
+    k norms), ``window`` (0: none), ``keep_first``, ``pool`` (0: none),
+    ``bias`` (true, the default; "qkv": not on the output; false), ``head_temp`` (default true), ``qk_norm`` (true, the
+    default: per head; "unit": per head without weights; "whole"; false),
     ``q_temp`` (None, or (coef, every): q at position p times 1 + coef ln(floor((p + 1) / every) + 1)),
     ``sink`` (None, "zero" or "learned"), ``out_gate`` (default false), ``conv`` (taps; 0: none; 1: a factor per
     channel),
@@ -188,11 +194,14 @@ class NormedAttention(Mixer):
         b = cls._base(p, prefix)
         out = {b + "q": TensorSpec((H * d, W)), b + "k": TensorSpec((G * d, W)), b + "v": TensorSpec((G * dv, W)),
                b + "o": TensorSpec((W, H * dv))}
-        if p.get("bias", True):
+        p = dict(p, bias=p.get("bias", True))
+        if p["bias"]:
             out.update({b + "q.b": TensorSpec((H * d,)), b + "k.b": TensorSpec((G * d,)),
-                        b + "v.b": TensorSpec((G * dv,)), b + "o.b": TensorSpec((W,))})
+                        b + "v.b": TensorSpec((G * dv,))})
+            if p["bias"] != "qkv":
+                out[b + "o.b"] = TensorSpec((W,))
         norm = p.get("qk_norm", True)
-        if norm:
+        if norm and norm != "unit":
             whole = norm == "whole"
             out[b + "q.norm"] = TensorSpec((H * d if whole else d,), init="norm")
             out[b + "k.norm"] = TensorSpec((G * d if whole else d,), init="norm")
@@ -211,13 +220,17 @@ class NormedAttention(Mixer):
     @classmethod
     def cache_need(cls, p):
         window = int(p.get("window") or 0)
-        pages = PagedKVNeed(int(p["num_kv_heads"]), cls._padded(p), window,
-                            keep_first=int(p.get("keep_first") or 0) if window else 0)
+        pool = int(p.get("pool") or 0) if window else 0
+        # pages: the tokens'; with pooled blocks a token stays until its block is complete, also behind the window
+        needs = [PagedKVNeed(int(p["num_kv_heads"]), cls._padded(p), max(window, pool),
+                             keep_first=int(p.get("keep_first") or 0) if window else 0)]
+        if pool:
+            needs.append(PagedKVNeed(int(p["num_kv_heads"]), cls._padded(p), tokens_per_entry=pool))
         K = cls._taps(p)
-        if K <= 1:
-            return pages
-        H, G, d, dv = int(p["num_heads"]), int(p["num_kv_heads"]), int(p["head_dim"]), int(p["v_dim"])
-        return (pages, StateNeed((K - 1, (H + G) * d + G * dv), "float32"))
+        if K > 1:
+            H, G, d, dv = int(p["num_heads"]), int(p["num_kv_heads"]), int(p["head_dim"]), int(p["v_dim"])
+            needs.append(StateNeed((K - 1, (H + G) * d + G * dv), "float32"))
+        return tuple(needs) if len(needs) > 1 else needs[0]
 
     def __init__(self, p, prefix, env, tensors):
         super().__init__(p, prefix, env, tensors)
@@ -238,6 +251,9 @@ class NormedAttention(Mixer):
         self.interleaved = layout == "interleaved"
         self.window = int(p.get("window") or 0)
         self.keep_first = int(p.get("keep_first") or 0) if self.window else 0
+        self.pool = int(p.get("pool") or 0) if self.window else 0
+        if self.pool and self.keep_first:
+            raise ValueError("a window keeps first tokens or sees pooled blocks, not both")
         self.eps = float(p.get("eps") or 0.0)
         scale = float(p["scale"]) if p.get("scale") is not None else float(self.d) ** -0.5
         b = self._base(p, prefix)
@@ -245,12 +261,16 @@ class NormedAttention(Mixer):
         self.out_gate = bool(p.get("out_gate"))
         self.w_qkv = torch.cat([tensors.get(b + n, env.dtype) for n in names], dim=0).contiguous()
         self.b_qkv = self.b_o = None
-        if p.get("bias", True):
+        bias = p.get("bias", True)
+        if bias not in (True, False, None, "qkv"):
+            raise ValueError(f"bias {bias!r} is not known; known: true, 'qkv', false")
+        if bias:
             biases = [tensors.get(b + n, env.dtype) for n in ("q.b", "k.b", "v.b")]
             if self.out_gate:                                        # the gate's rows of the product have no bias
                 biases.append(torch.zeros(self.H, dtype=env.dtype, device=biases[0].device))
             self.b_qkv = torch.cat(biases, dim=0).contiguous()
-            self.b_o = tensors.get(b + "o.b", env.dtype).contiguous()
+            if bias != "qkv":
+                self.b_o = tensors.get(b + "o.b", env.dtype).contiguous()
         tensors.drop(b + "q", b + "k", b + "v", b + "g", b + "q.b", b + "k.b", b + "v.b")
         w_o = tensors.get(b + "o", env.dtype)
         if self.D != self.dv:
@@ -261,11 +281,14 @@ class NormedAttention(Mixer):
             tensors.drop(b + "o")
         self.w_o = w_o.contiguous()
         norm = p.get("qk_norm", True)
-        if norm not in (True, False, None, "whole", "head"):
-            raise ValueError(f"qk_norm {norm!r} is not known; known: true (per head), 'whole', false")
+        if norm not in (True, False, None, "whole", "head", "unit"):
+            raise ValueError(f"qk_norm {norm!r} is not known; known: true (per head), 'unit', 'whole', false")
         self.norm_whole = norm == "whole"
-        self.q_norm = tensors.get(b + "q.norm", torch.float32).contiguous() if norm else None
-        self.k_norm = tensors.get(b + "k.norm", torch.float32).contiguous() if norm else None
+        if norm == "unit":
+            self.q_norm = self.k_norm = torch.ones(self.d, dtype=torch.float32, device=env.device)
+        else:
+            self.q_norm = tensors.get(b + "q.norm", torch.float32).contiguous() if norm else None
+            self.k_norm = tensors.get(b + "k.norm", torch.float32).contiguous() if norm else None
         # what every q head is multiplied by: the score's scale times the head's own number
         self.factor = torch.full((self.H,), scale, dtype=torch.float32, device=env.device)
         if p.get("head_temp", True):
@@ -288,8 +311,13 @@ class NormedAttention(Mixer):
             self.taps = torch.cat([tensors.get(b + n, torch.float32) for n in ("q.conv", "k.conv", "v.conv")],
                                   dim=0).t().contiguous()                                  # [taps, channels]
         base = float(p.get("rot_base") or 10000.0)
-        self.freq = tensors.shared_part(("rotary_frequencies", self.rot_dims, base),
-                                        lambda: rotary_frequencies(self.rot_dims, base).to(env.device))
+        factor = float(p["rot_factor"]) if p.get("rot_factor") is not None else 1.0
+        self.freq = tensors.shared_part(("rotary_frequencies", self.rot_dims, base, factor),
+                                        lambda: (rotary_frequencies(self.rot_dims, base) / factor).to(env.device))
+        self.out_features = self.H * self.D
+
+    # a branch of "parallel" whose outputs are not normed: it computes its first product itself (which may have a bias)
+    w_in = None
 
     def input_weight(self):
         """The matrix of this mixer's first product, for a wrapper that computes the first products of several
@@ -300,13 +328,18 @@ class NormedAttention(Mixer):
         self.w_qkv = view
 
     def forward(self, x, batch, cache, writes=True, proj=None):
+        return ops.linear(self.mix(x, batch, cache, writes, proj=proj), self.w_o, bias=self.b_o)
+
+    def mix(self, x, batch, cache, writes=True, out=None, out_scale: float = 1.0, proj=None):
+        """The heads' outputs side by side [T, heads * D] (into ``out`` if given), times ``out_scale``, before the
+        output product."""
         H, G, d, dv, D, C = self.H, self.G, self.d, self.dv, self.D, self.C
         if proj is None:
             proj = ops.linear(x, self.w_qkv, bias=self.b_qkv)                 # [T, q | k | v (| gate)]
-        pages = cache.parts[0] if self.K > 1 else cache
+        pages = cache.parts[0] if cache.parts else cache
         qkv = proj if proj.shape[1] == C else proj[:, :C]
         if self.K >= 1:
-            state = cache.parts[1].state if self.K > 1 else None
+            state = cache.parts[-1].state if self.K > 1 else None
             qkv = ops.causal_conv(qkv, 0, self.taps, state, batch, torch.float32)
             if writes and state is not None:
                 ops.conv_state_update(proj, 0, state, batch)
@@ -315,33 +348,40 @@ class NormedAttention(Mixer):
                                   self.interleaved, batch.positions, slots, self.factor, H, G, d, dv, D,
                                   norm_whole=self.norm_whole, temp_coef=self.temp_coef, temp_every=self.temp_every,
                                   out_dtype=self.env.dtype)
+        pooled = None
+        if self.pool:
+            blocks = cache.parts[1]
+            if writes:
+                ops.pool_blocks(pages.kv, batch.block_table[pages.group], batch, batch.slot_mapping[blocks.group],
+                                blocks.kv, self.pool)
+            pooled = (blocks.kv, batch.block_table[blocks.group], self.pool)
         gate = proj[:, C:] if self.out_gate else None
-        out = self.attend(q.view(-1, H * D), batch, pages, gate)
-        return ops.linear(out, self.w_o, bias=self.b_o)
+        return self.attend(q.view(-1, H * D), batch, pages, gate, pooled, out, out_scale)
 
-    def attend(self, q, batch, cache, gate=None):
+    def attend(self, q, batch, cache, gate=None, pooled=None, out=None, out_scale: float = 1.0):
         """bfloat16 runs on the tensor cores (requests with several tokens through the flash-style kernel, single
-        tokens through the split kernel; both know the window, the kept first tokens, the sink and the gate); the
-        32-bit path runs the general kernel."""
+        tokens through the split kernel; both know the window, the kept first tokens or the pooled blocks, the sink
+        and the gate); the 32-bit path runs the general kernel."""
         H, G, D = self.H, self.G, self.D
         table = batch.block_table[cache.group]
+        more = dict(sink=self.sink, gate=gate, pooled=pooled, out_scale=out_scale)
         if q.dtype != torch.bfloat16:
             return ops.paged_attention_general(q, q.shape[1], cache.kv, table, batch.req_of_token, batch.positions,
-                                               H, G, D, self.window, 1.0, self.keep_first, sink=self.sink, gate=gate)
-        out = torch.empty((q.shape[0], H * D), dtype=q.dtype, device=q.device)
+                                               H, G, D, self.window, 1.0, self.keep_first, out=out, **more)
+        if out is None:
+            out = torch.empty((q.shape[0], H * D), dtype=q.dtype, device=q.device)
         kv_tiles = G * (-(-(H // G) // 8))
         reach = batch.max_context_len
         if self.window:
-            reach = min(reach, self.window + self.keep_first)
+            reach = min(reach, self.window + self.keep_first + (reach // self.pool if self.pool else 0))
         if batch.num_prefill_tiles:
             ops.prefill_attention(q, q.shape[1], out, cache.kv, table, batch.prefill_tiles, batch.positions,
-                                  H, G, D, self.window, 1.0, self.keep_first, sink=self.sink, gate=gate)
+                                  H, G, D, self.window, 1.0, self.keep_first, **more)
         n = batch.num_tokens if batch.decode_only else batch.num_decode_rows
         if n:
             ops.decode_attention(q, q.shape[1], out, cache.kv, table, None if batch.decode_only else batch.decode_rows,
                                  n, batch.req_of_token, batch.positions, H, G, D, self.window, 1.0,
-                                 ops.decode_splits(n, kv_tiles, reach), keep_first=self.keep_first, sink=self.sink,
-                                 gate=gate)
+                                 ops.decode_splits(n, kv_tiles, reach), keep_first=self.keep_first, **more)
         return out
 
 

@@ -99,10 +99,14 @@ class Mixer(Part):
     says that ``x`` may be an ``ops.NormedRows`` (which ``ops.linear`` takes in
     place of a tensor); ``defers_output`` = True says that ``forward`` has a
     keyword ``defer`` and, when it is True, may return its last product as an
-    ``ops.PendingLinear``."""
+    ``ops.PendingLinear``.  A mixer with ``takes_stream`` = True has
+    ``forward_stream(stream, batch, cache, writes)``, which adds what is pending
+    to the stream and reads it in one kernel, for arrangements without a norm
+    before the part."""
 
     takes_normed_rows = False
     defers_output = False
+    takes_stream = False
 
     @classmethod
     def cache_need(cls, params: dict):

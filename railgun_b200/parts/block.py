@@ -13,6 +13,12 @@ multiplier, a per-feature layer scale) are part of the post-norm's weight.
 The post-norm, the 32-bit addition and the next branch's norm are one kernel
 (ops.PendingNormed).
 
+"postnorm": a norm on each part's output only, x = x + post_norm(part(x)); the
+part reads the stream itself (norm kind "identity").  Norm, addition and the
+rounding for the next part are one kernel; a part that does more with the
+stream before it reads it (``takes_stream``, the token shift) gets the stream
+and what is pending and does all of it in one kernel of its own.
+
 "hyper": S copies of the residual stream instead of one (hyper-connections).
 A branch reads u = sum_s a[s] x_s through its norm, and its output y changes
 every copy at once: x_t <- sum_s M[s, t] x_s + b[t] y, with a [S], M [S, S]
@@ -62,6 +68,19 @@ class Sandwich(Arrangement):
                 raise ValueError("the 'sandwich' arrangement needs a post_norm on every branch")
             h = normed_input(b.norm, b.part, stream)
             y = b.part.forward(h, batch, cache, writes) if b.role == "mixer" else b.part.forward(h, batch)
+            stream.pending = ops.PendingNormed(y, b.post_norm.weight, b.post_norm.eps)
+
+
+class PostNorm(Arrangement):
+    def run(self, layer, stream, batch, cache, writes):
+        for b in layer.branches:
+            if b.post_norm is None:
+                raise ValueError("the 'postnorm' arrangement needs a post_norm on every branch")
+            if b.role == "mixer" and getattr(b.part, "takes_stream", False):
+                y = b.part.forward_stream(stream, batch, cache, writes)
+            else:
+                h = normed_input(b.norm, b.part, stream)
+                y = b.part.forward(h, batch, cache, writes) if b.role == "mixer" else b.part.forward(h, batch)
             stream.pending = ops.PendingNormed(y, b.post_norm.weight, b.post_norm.eps)
 
 
@@ -183,6 +202,7 @@ class Reinject(StreamOp):
 
 register_arrangement("prenorm", PreNorm)
 register_arrangement("sandwich", Sandwich)
+register_arrangement("postnorm", PostNorm)
 register_arrangement("hyper", Hyper)
 register_arrangement("parallel_residual", ParallelResidual)
 register_stream_op("reinject", Reinject)

@@ -68,4 +68,16 @@ class RMSNorm(Norm):
         return ops.add_rmsnorm(resid, pending, self.weight, self.eps, self.env.dtype, rows)
 
 
+class Identity(Norm):
+    """No norm: the part behind it reads the stream itself, in the activation type.  No parameters."""
+
+    fuses_post_norm = True
+
+    def add_norm(self, resid, pending, rows=None):
+        if rows is not None:
+            return ops.add_postnorm_rmsnorm(resid, pending, None, 0.0, self.env.dtype, rows)
+        return ops.postnorm_shift(resid, pending, None, None, None, self.env.dtype)[1]
+
+
 register_norm("rmsnorm", RMSNorm)
+register_norm("identity", Identity)

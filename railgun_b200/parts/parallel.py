@@ -3,9 +3,11 @@ the sum of the branches' outputs, each times a constant.
 
 A branch is any mixer that can hand out what goes into its output product
 (``mix(x, batch, cache, writes, out, out_scale, proj)`` -> [T, out_features],
-``w_o`` [hidden, out_features]) and takes its first product from outside
-(``w_in`` [in_features, hidden]; ``proj`` = x w_in^T).  ONE product with the
-branches' input matrices stacked feeds them all; they write side by side
+``w_o`` [hidden, out_features]).  A branch may take its first product from
+outside (``w_in`` [in_features, hidden]; ``proj`` = x w_in^T): ONE product with
+those branches' input matrices stacked feeds them; a branch whose ``w_in`` is
+None (its first product has a bias, or it does more to x first) computes its
+own.  They write side by side
 into one buffer, already multiplied by their constants in 32-bit before the
 one rounding, and ONE product with the output matrices side by side gives
 sum_b c_b W_o,b z_b.  What the branches keep between steps is asked for as a
@@ -92,15 +94,27 @@ class Parallel(Mixer):
         for part in self.parts:
             if not all(hasattr(part, a) for a in ("mix", "w_o", "w_in")):
                 raise ValueError(f"{type(part).__name__} cannot be a branch of 'parallel': it has no mix(), w_in and w_o")
-        self.w_in = torch.cat([part.w_in for part in self.parts], dim=0).contiguous()
-        self.w_o = torch.cat([part.w_o for part in self.parts], dim=1).contiguous()
+        takers = [part for part in self.parts if part.w_in is not None]
+        for part in self.parts:
+            if getattr(part, "b_o", None) is not None:
+                raise ValueError("a branch of 'parallel' cannot have a bias on its output")
+        self.w_in = torch.cat([part.w_in for part in takers], dim=0).contiguous() if takers else None
         self.widths = [int(part.out_features) for part in self.parts]
-        self.in_widths = [int(part.w_in.shape[0]) for part in self.parts]
+        # zero columns up to a multiple of 8, so that the products take the rows with 16-byte loads
+        self.padding = -sum(self.widths) % 8
+        w_os = [part.w_o for part in self.parts]
+        if self.padding:
+            w_os.append(torch.zeros((w_os[0].shape[0], self.padding), dtype=w_os[0].dtype, device=w_os[0].device))
+        self.w_o = torch.cat(w_os, dim=1).contiguous()
+        self.in_widths = [int(part.w_in.shape[0]) if part.w_in is not None else 0 for part in self.parts]
         # the stacked matrices are the ones that are kept: the branches see their share of them
         at = off = 0
         for part, n_in, n in zip(self.parts, self.in_widths, self.widths):
-            part.w_in = self.w_in[at:at + n_in]
             part.w_o = self.w_o[:, off:off + n]
+            if not n_in:
+                off += n
+                continue
+            part.w_in = self.w_in[at:at + n_in]
             for name in ("w_qkv", "w_yx"):
                 if hasattr(part, name):
                     setattr(part, name, part.w_in)
@@ -118,11 +132,13 @@ class Parallel(Mixer):
                 ys = [part.forward(x, batch, view, writes) for part, view in zip(self.parts, self._views(cache))]
             return ops.norm_sum(ys, self.out_norms, self.scales, self.eps)
         T = x.shape[0]
-        proj = ops.linear(x, self.w_in)
-        z = torch.empty((T, sum(self.widths)), dtype=self.env.dtype, device=self.w_o.device)
+        proj = ops.linear(x, self.w_in) if self.w_in is not None else None
+        new = torch.zeros if self.padding else torch.empty
+        z = new((T, self.w_o.shape[1]), dtype=self.env.dtype, device=self.w_o.device)
         off = at = 0
         for part, c, n, n_in, view in zip(self.parts, self.scales, self.widths, self.in_widths, self._views(cache)):
-            part.mix(x, batch, view, writes, out=z[:, off:off + n], out_scale=c, proj=proj[:, at:at + n_in])
+            part.mix(x, batch, view, writes, out=z[:, off:off + n], out_scale=c,
+                     proj=proj[:, at:at + n_in] if n_in else None)
             off += n
             at += n_in
         return ops.linear(z, self.w_o)

@@ -27,11 +27,20 @@ class WeightError(ValueError):
         self.wrong_shape = list(wrong_shape)
 
 
+class AnySize(int):
+    """A size that only the files give (no key of config.json does): any number matches.  As a number it is what
+    random-weights mode makes."""
+
+
 @dataclass(frozen=True)
 class TensorSpec:
-    shape: tuple
+    shape: tuple                # an AnySize stands for whatever size the file has there
     init: str = "normal"        # how random-weights mode fills it: "normal" | "norm" | "eye" | "zeros"
     optional: bool = False
+
+
+def shapes_match(expected, got) -> bool:
+    return len(expected) == len(got) and all(isinstance(e, AnySize) or int(e) == int(g) for e, g in zip(expected, got))
 
 
 def stored_precision(t: torch.Tensor) -> torch.Tensor:
@@ -57,7 +66,7 @@ def load_weights(model_dir, expected: dict[str, TensorSpec], device="cpu",
     missing = [n for n, s in expected.items() if n not in entries and not s.optional]
     unexpected = [n for n in entries if n not in expected and n not in allow_unexpected]
     wrong = [(n, tuple(expected[n].shape), entries[n].shape)
-             for n in expected if n in entries and tuple(expected[n].shape) != entries[n].shape]
+             for n in expected if n in entries and not shapes_match(expected[n].shape, entries[n].shape)]
     if missing or unexpected or wrong:
         lines = [f"weights in {model_dir} do not match the model:"]
         if missing:
