@@ -901,6 +901,136 @@ def run_kasarax(args):
     return 0
 
 
+def sagizen_sizes(name):
+    """(Sagizen configuration, and the two closest designs at equal width, layers, feed-forward and vocabulary: Mepatar
+    with the gated delta rule where Sagizen has Mamba-2, Kasarax with its parallel mixer in every layer)."""
+    def all_of(width, heads, kv, d, ff, vocab):
+        half, dense = heads // 2, dict(kind="dense", ff=ff)
+        mamba = dict(type="mamba2", mixer=dict(heads=width // 64, vdim=64, state=128, groups=2, conv=4, norm_groups=2), mlp=dense)
+        left = dict(heads=half, kv_heads=kv, dim=d, vdim=d, scale=d ** -0.5, mask=dict(size=512, pool=8),
+                    rot=dict(base=10000.0, dims=d // 2, scaling=dict(factor=4.0)))
+        par = dict(type="parallel", mixer=dict(left=left, right=dict(heads=half, dim=d), left_scale=0.6, right_scale=0.7),
+                   mlp=dense)
+        sag = dict(architecture="Sagizen", width=width, vocab=vocab, norm=dict(eps=1e-6),
+                   layers=[mamba, mamba, par, mamba, mamba, par])
+        delta = dict(type="delta", mixer=dict(heads=heads, kv_heads=heads // 2, dim=d, vdim=d, conv=4), mlp=dense)
+        att = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv, dim=d, vdim=d, scale=d ** -0.5,
+                                                rot=dict(base=10000.0, dims=d // 2), mask=dict(size=512, keep_first=4)), mlp=dense)
+        mep = dict(architecture="Mepatar", width=width, vocab=vocab, norm=dict(eps=1e-6, groups=4),
+                   embedding=dict(scale=width ** 0.5), canon=dict(taps=4), layers=[delta, delta, att, delta, delta, att])
+        kleft = dict(heads=half, kv_heads=kv, dim=d, vdim=d, conv=4, scale=d ** -0.5, rot=dict(base=10000.0, dims=d // 2))
+        kright = dict(heads=half, dim=d, vdim=d, decay=[1.0 - 2.0 ** (-5 - 0.4 * i) for i in range(half)])
+        kpar = dict(type="parallel", mixer=dict(left=kleft, right=kright), mlp=dense)
+        kas = dict(architecture="Kasarax", width=width, vocab=vocab, norm=dict(eps=1e-6), logit_scale=0.5, layers=[kpar] * 6)
+        return dict(sagizen=sag, mepatar=mep, kasarax=kas)
+
+    if name == "w2048":      # 32 state heads of 128 x 64; halves of 8 heads of 128 (2 key/value heads, window 512, blocks of 8)
+        return all_of(2048, 16, 2, 128, 8192, 32768)
+    if name == "w1024":      # 16 state heads of 128 x 64; halves of 4 heads of 128
+        return all_of(1024, 8, 2, 128, 4096, 32768)
+    raise ValueError(name)
+
+
+SAGIZEN_RANK = 64            # of the decay's low-rank product, which random weights are made with
+
+
+def sagizen_decode_bytes(cfg, batch, context):
+    """Bytes a decode step has to read or write: the weights of every layer, the head, and what the live requests keep:
+    the matrix states in 32-bit (read and written), convolution tails and previous rows, and an attention half's cache
+    as far back as its window, with the pooled blocks before it."""
+    W, V = cfg["width"], cfg["vocab"]
+    total = V * W * 2
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        total += batch * W * 4 * 2
+        if L["type"] == "mamba2":
+            H, dv, N, G, K = m["heads"], m["vdim"], m["state"], m["groups"], m["conv"]
+            C = H * dv + 2 * G * N
+            total += (H * dv + C + H) * W * 2 + W * H * dv * 2 + batch * (H * dv * N + (K - 1) * C) * 4 * 2
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, dv, D = a["heads"], a["kv_heads"], a["dim"], a["vdim"], -(-max(a["dim"], a["vdim"]) // 16) * 16
+            win, pool = a["mask"]["size"], a["mask"]["pool"]
+            seen = min(context, win) + max(0, context - win) // pool
+            total += ((H + G) * d + G * dv) * W * 2 + W * H * dv * 2 + batch * seen * G * 2 * D * 2
+            H, d = r["heads"], r["dim"]
+            total += 5 * H * d * W * 2 + SAGIZEN_RANK * (W + H * d) * 2 + batch * (H * d * d + W) * 4 * 2
+        if L["mlp"]:
+            total += 3 * L["mlp"]["ff"] * W * 2
+    return total
+
+
+def sagizen_prefill_flops(cfg, T):
+    """FLOPs of one prompt of T tokens by the design's own arithmetic: products, attention over the tokens and blocks
+    a query sees, and the matrix states' updates and read-outs (4 d dv per head and token)."""
+    W, V = cfg["width"], cfg["vocab"]
+    total = 2 * V * W
+    for L in cfg["layers"]:
+        m = L["mixer"]
+        if L["type"] == "mamba2":
+            H, dv, N, G = m["heads"], m["vdim"], m["state"], m["groups"]
+            total += 2 * T * ((2 * H * dv + 2 * G * N + H) * W + W * H * dv) + T * H * 4 * N * dv
+        else:
+            a, r = m["left"], m["right"]
+            H, G, d, dv, win, pool = a["heads"], a["kv_heads"], a["dim"], a["vdim"], a["mask"]["size"], a["mask"]["pool"]
+            pairs = sum(min(t + 1, win) + max(0, t + 1 - win) // pool for t in range(T))
+            total += 2 * T * (((H + G) * d + G * dv) * W + W * H * dv) + H * 2 * (d + dv) * pairs
+            H, d = r["heads"], r["dim"]
+            total += 2 * T * (5 * H * d * W + SAGIZEN_RANK * (W + H * d)) + T * H * 4 * d * d
+        if L["mlp"]:
+            total += 2 * T * 3 * L["mlp"]["ff"] * W
+    return total
+
+
+def run_sagizen(args):
+    """Prefill and decode throughput of Sagizen at layer sizes of real models (random weights), beside the closest two
+    designs at equal width, number of layers, feed-forward and vocabulary.  One JSON line per model and size."""
+    import numpy as np
+    import torch
+    from railgun_b200.engine.batch import StepEntry
+    from railgun_b200.engine.engine import Engine
+    page, pool_tokens = 16, 64 * 4096
+    pk, pk_src = peaks()
+    counts = dict(sagizen=(sagizen_decode_bytes, sagizen_prefill_flops), mepatar=(mepatar_decode_bytes, mepatar_prefill_flops),
+                  kasarax=(kasarax_decode_bytes, kasarax_prefill_flops))
+    for size in (args.sizes.split(",") if args.sizes else ["w1024", "w2048"]):
+        for label, cfg in sagizen_sizes(size).items():
+            eng = Engine(model_folder(cfg), dtype="bfloat16", block_size=page, num_gpu_blocks=pool_tokens // page,
+                         max_num_seqs=64, max_num_batched_tokens=8192, max_model_len=4096)
+            runner, V, rng = eng.runner, cfg["vocab"], np.random.default_rng(0)
+            _, _, time_decode = decode_tools(runner, V, rng)
+            line = {"mode": "sagizen", "size": size, "model": label, "layer_runs": len(runner.model.order),
+                    "cache_bytes_per_token": runner.cache.bytes_per_token()}
+            for b in (8, 64):
+                tok_s, ms, n_launch, _ = time_decode(b, args.steps, args.warmup, 1000 * b, args.context)
+                line[f"decode_b{b}_tok_s"], line[f"decode_b{b}_ms"] = round(tok_s, 1), round(ms, 4)
+                line[f"decode_b{b}_launches_per_step"] = n_launch // args.steps
+                by = counts[label][0](cfg, b, args.context + args.warmup + args.steps // 2)
+                line[f"decode_b{b}_GB_per_step"] = round(by / 1e9, 3)
+                line[f"decode_b{b}_frac_hbm"] = round(by / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 3)
+            prompt = rng.integers(0, V, size=args.tokens).tolist()
+            times = []
+            for i in range(args.warmup + 7):
+                torch.cuda.synchronize()
+                t0, t1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                t0.record()
+                runner.step([StepEntry(7000 + i, prompt, [args.tokens - 1])])
+                t1.record()
+                torch.cuda.synchronize()
+                runner.end([7000 + i])
+                times.append(t0.elapsed_time(t1))
+            runner.check_device_errors()
+            ms = sorted(times[args.warmup:])[len(times[args.warmup:]) // 2]
+            fl = counts[label][1](cfg, args.tokens)
+            line.update(prefill_tokens=args.tokens, prefill_ms=round(ms, 3), prefill_tok_s=round(args.tokens / ms * 1e3, 1),
+                        prefill_TFLOP=round(fl / 1e12, 3), prefill_frac_flops=round(fl / (ms * 1e-3) / (pk["bf16_tflops"] * 1e12), 3),
+                        peaks=pk_src)
+            print(json.dumps(line), flush=True)
+            del eng, runner, time_decode
+            torch.cuda.empty_cache()
+    return 0
+
+
 def run_kernels(args):
     """Times the hot kernels one by one, each as a CUDA graph of 16 calls over 16 different operand sets (so
     that weights and caches come from HBM, not L2), with CUDA events around replays.  One JSON line per case."""
@@ -1380,6 +1510,175 @@ def run_kernels(args):
                     "without_frac_hbm": round(by / res[False] / 1e3 / pk["hbm_gbs"], 3)} if B > 1 else
                    {"frac_flops": round(fl / res[True] / 1e6 / pk["bf16_tflops"], 3),
                     "without_frac_flops": round(fl / res[False] / 1e6 / pk["bf16_tflops"], 3)}))
+    if on("sagizen_rows"):
+        # Sagizen's own kernels by the bytes they have to move, each beside the like kernel of another design: the
+        # residual addition with the norm behind a part and the token shift beside the one with the next part's norm, the
+        # mixes of a row with the row before beside the short convolution, the scans beside retention's and the delta
+        # rule's, the fused single-token step beside the delta rule's kernels, the gated norm in parts beside the heads'
+        # norm, attention over a window and pooled blocks beside a window that keeps first tokens
+        from types import SimpleNamespace
+        pk, _ = peaks()
+        W, K = 2048, 4
+        for T in (64, 4096):
+            R_ = 1 if T > 64 else T
+            per = T // R_
+            batch = SimpleNamespace(cu_seqlens=torch.arange(0, T + 1, per, dtype=torch.int32, device=dev),
+                                    num_requests=R_, req_of_token=(torch.arange(T, device=dev) // per).to(torch.int32),
+                                    start_pos=torch.full((R_,), 1000, dtype=torch.int32, device=dev),
+                                    state_slots=torch.arange(R_, dtype=torch.int32, device=dev), max_query_len=per,
+                                    positions=(1000 + torch.arange(T, device=dev) % per).to(torch.int32))
+            gbs = lambda by, us: round(by / us / 1e3 / pk["hbm_gbs"], 3)
+            ys = [torch.randn(T, W, device=dev).to(torch.bfloat16) for _ in range(L)]
+            rs = [torch.randn(T, W, device=dev) for _ in range(L)]
+            nw, share = torch.ones(W, device=dev), torch.rand(W, device=dev)
+            prev = [torch.randn(R_, 1, W, device=dev) for _ in range(L)]
+            us = timed(lambda: [ops.postnorm_shift(r, ops.PendingNormed(y, nw, 1e-6), share, p, batch, torch.bfloat16)
+                                for r, y, p in zip(rs, ys, prev)])
+            usn = timed(lambda: [ops.postnorm_shift(r, ops.PendingNormed(y, nw, 1e-6), None, None, None, torch.bfloat16)
+                                 for r, y in zip(rs, ys)])
+            us2 = timed(lambda: [ops.add_postnorm_rmsnorm(r, ops.PendingNormed(y, nw, 1e-6), nw, 1e-6, torch.bfloat16)
+                                 for r, y in zip(rs, ys)])
+            by, by2 = T * W * (4 + 2 + 4 + 2) + R_ * W * 8, T * W * (4 + 2 + 4 + 2)
+            out(f"addition, norm behind the part, token shift W{W} T{T}", us, frac=gbs(by, us), no_shift_us=round(usn, 2),
+                no_shift_frac=gbs(by2, usn), both_norms_us=round(us2, 2), both_norms_frac=gbs(by2, us2))
+            mu = torch.rand(5, W, device=dev)
+            us = timed(lambda: [ops.shift_mixes(y, mu, p, batch) for y, p in zip(ys, prev)])
+            taps1 = torch.randn(K, W, device=dev) * 0.3
+            cst = [torch.randn(R_, K - 1, W, device=dev) for _ in range(L)]
+            us2 = timed(lambda: [(ops.causal_conv(y, 0, taps1, c, batch, torch.bfloat16, residual=True),
+                                  ops.conv_state_update(y, 0, c, batch)) for y, c in zip(ys, cst)])
+            by, by2 = T * W * (2 + 6 * 2) + R_ * W * 8, T * W * (2 + 2) + R_ * (K - 1) * W * 8
+            out(f"five mixes with the row before W{W} T{T}", us, frac=gbs(by, us), conv_us=round(us2, 2), conv_frac=gbs(by2, us2))
+            # RWKV half: 8 heads of 128 x 128; decay from a low-rank product
+            Hr, dr, rank = 8, 128, SAGIZEN_RANK
+            n = Hr * dr
+            las = [torch.randn(T, rank, device=dev) for _ in range(L)]
+            w2 = (torch.randn(n, rank, device=dev) * 0.1).to(torch.bfloat16)
+            w0 = torch.randn(n, device=dev) - 3
+            us = timed(lambda: [ops.lowrank_decay(a, w2, w0) for a in las])
+            by, fl = T * (rank + n) * 4 + n * rank * 2, 2 * T * n * rank
+            out(f"low-rank decay rank{rank} N{n} T{T}", us, frac=gbs(by, us), TFLOPs=round(fl / us / 1e6, 2))
+            rk = [[torch.randn(T, n, device=dev) * 0.2 for _ in range(3)] for _ in range(L)]
+            ws_ = [torch.rand(T, n, device=dev) * 0.1 + 0.9 for _ in range(L)]
+            sts = [torch.randn(R_, Hr, dr, dr, device=dev) * 0.1 for _ in range(L)]
+            bonus, decay = torch.randn(Hr, dr, device=dev), torch.full((Hr,), 0.99, device=dev)
+            us = timed(lambda: [ops.state_scan(r, k, v, st, batch, Hr, dr, dr, rule="channel", w=w, bonus=bonus)
+                                for (r, k, v), w, st in zip(rk, ws_, sts)])
+            us2 = timed(lambda: [ops.state_scan(r, k, v, st, batch, Hr, dr, dr, decay=decay) for (r, k, v), st in zip(rk, sts)])
+            by, by2 = T * n * 5 * 4 + R_ * n * dr * 8, T * n * 4 * 4 + R_ * n * dr * 8
+            out(f"scan with a decay per channel H{Hr} d{dr} T{T} ({R_} requests)", us, frac=gbs(by, us), retention_us=round(us2, 2),
+                retention_frac=gbs(by2, us2))
+            os_ = [torch.randn(T, Hr, dr, device=dev) for _ in range(L)]
+            nwr = torch.ones(n, device=dev)
+            us = timed(lambda: [ops.head_norm_gate(o, x[0], nwr, 1e-6, torch.bfloat16, out_scale=0.7) for o, x in zip(os_, rk)])
+            out(f"heads' norm, weight and gate H{Hr} dv{dr} T{T}", us, frac=gbs(T * n * 10, us))
+            # Mamba-2: 32 heads of 128 x 64 beside the delta rule with 16 heads of 128 x 128
+            H, N, dv, G = 32, 128, 64, 2
+            inner = H * dv
+            C = inner + 2 * G * N
+            projs = [torch.randn(T, inner + C + H, device=dev) for _ in range(L)]
+            taps, cb = torch.randn(K, C, device=dev) * 0.3, torch.zeros(C, device=dev)
+            cstate = [torch.randn(R_, K - 1, C, device=dev) for _ in range(L)]
+            A, dtb, D = torch.zeros(H, device=dev), torch.full((H,), -2.0, device=dev), torch.ones(H, device=dev)
+            sts = [torch.randn(R_, H, dv, N, device=dev) * 0.1 for _ in range(L)]
+            nwm = torch.ones(inner, device=dev)
+            Hd, Hq, dd = 16, 8, 128
+            Cd = 2 * Hq * dd + Hd * dd
+            pd = [torch.randn(T, Cd + Hd * dd, device=dev).to(torch.bfloat16) for _ in range(L)]
+            bad = [torch.randn(T, 2 * Hd, device=dev) for _ in range(L)]
+            tapd, cstd = torch.randn(K, Cd, device=dev) * 0.3, [torch.randn(R_, K - 1, Cd, device=dev) for _ in range(L)]
+            std = [torch.randn(R_, Hd, dd, dd, device=dev) * 0.1 for _ in range(L)]
+            Ad, nwd = torch.zeros(Hd, device=dev), torch.ones(dd, device=dev)
+
+            def delta(p, ba, c, st):
+                qkv = ops.causal_conv(p, 0, tapd, c, batch, torch.float32, silu=True)
+                ops.conv_state_update(p, 0, c, batch)
+                beta, g = ops.delta_prepare(qkv, Hq, dd, dd ** -0.5, 1e-6, ba, 0, Hd, Ad, Ad, Hd)
+                o = ops.state_scan(qkv[:, :Hq * dd], qkv[:, Hq * dd:2 * Hq * dd], qkv[:, 2 * Hq * dd:], st, batch, Hd, dd, dd,
+                                   g=g, beta=beta)
+                return ops.head_norm_gate(o, p[:, Cd:], nwd, 1e-6, torch.bfloat16)
+
+            usd = timed(lambda: [delta(p, ba, c, st) for p, ba, c, st in zip(pd, bad, cstd, std)])
+            byd = T * (Cd + Hd * dd) * 2 + R_ * ((K - 1) * Cd * 8 + Hd * dd * dd * 8) + T * Hd * dd * 2
+            if T == R_:
+                def step(p, c, st):
+                    o = ops.ssd_step(p, inner, inner + C, taps, cb, c, dtb, A, D, st, batch, H, G, N, dv)
+                    return ops.gate_group_norm(o, p[:, :inner], nwm, 1e-6, 2, torch.bfloat16,
+                                               conv=(p[:, inner:inner + C], c), batch=batch)
+                us = timed(lambda: [step(p, c, st) for p, c, st in zip(projs, cstate, sts)])
+                by = T * (inner + C + H) * 4 + R_ * ((K - 1) * C * 8 + H * dv * N * 8) + T * inner * 2
+                us1 = timed(lambda: [ops.ssd_step(p, inner, inner + C, taps, cb, c, dtb, A, D, st, batch, H, G, N, dv)
+                                     for p, c, st in zip(projs, cstate, sts)])
+                out(f"Mamba-2 between its products, single tokens, {T} requests", us, frac=gbs(by, us), step_us=round(us1, 2),
+                    delta_us=round(usd, 2), delta_frac=gbs(byd, usd))
+            else:
+                p16 = [p.to(torch.bfloat16) for p in projs]
+                xbc = [torch.randn(T, C, device=dev) * 0.3 for _ in range(L)]
+                us = timed(lambda: [(ops.causal_conv(p, inner, taps, c, batch, torch.float32, silu=True, bias=cb),
+                                     ops.conv_state_update(p, inner, c, batch)) for p, c in zip(p16, cstate)])
+                us2 = timed(lambda: [(ops.causal_conv(p, 0, tapd, c, batch, torch.float32, silu=True),
+                                      ops.conv_state_update(p, 0, c, batch)) for p, c in zip(pd, cstd)])
+                out(f"convolution with bias and silu C{C} T{T}", us, frac=gbs(T * C * 6, us), delta_us=round(us2, 2),
+                    delta_frac=gbs(T * Cd * 6, us2))
+                dt, g = ops.ssd_prepare(projs[0][:, inner + C:], dtb, A)
+                us = timed(lambda: [ops.state_scan(x[:, inner + G * N:], x[:, inner:inner + G * N], x[:, :inner], st, batch, H, N,
+                                                   dv, g=g, beta=dt, rule="scalar", skip=D) for x, st in zip(xbc, sts)])
+                qd = [torch.randn(T, Hq * dd, device=dev) * 0.1 for _ in range(L)]
+                vd = [torch.randn(T, Hd * dd, device=dev) for _ in range(L)]
+                gd = torch.rand(T, Hd, device=dev)
+                us2 = timed(lambda: [ops.state_scan(q, q, v, st, batch, Hd, dd, dd, g=gd, beta=gd) for q, v, st in zip(qd, vd, std)])
+                out(f"scan H{H} {N} x {dv} T{T}", us, frac=gbs(T * (C + inner) * 4, us), delta_us=round(us2, 2),
+                    delta_frac=gbs(T * (2 * Hq + 2 * Hd) * dd * 4, us2))
+                us = timed(lambda: [ops.ssd_prepare(p[:, inner + C:], dtb, A) for p in projs])
+                out(f"step sizes and decays H{H} T{T}", us, frac=gbs(T * H * 12, us))
+                om = [torch.randn(T, H, dv, device=dev) for _ in range(L)]
+                us = timed(lambda: [ops.gate_group_norm(o, p[:, :inner], nwm, 1e-6, 2, torch.bfloat16) for o, p in zip(om, p16)])
+                ohd = [torch.randn(T, Hd, dd, device=dev) for _ in range(L)]
+                us2 = timed(lambda: [ops.head_norm_gate(o, p[:, Cd:], nwd, 1e-6, torch.bfloat16) for o, p in zip(ohd, pd)])
+                out(f"gate, then a norm in 2 parts of {inner // 2} T{T}", us, frac=gbs(T * inner * 8, us), heads_us=round(us2, 2),
+                    heads_frac=gbs(T * Hd * dd * 8, us2))
+        # attention over a window of 512 and blocks of 8 beside the window alone and the window with 4 kept tokens
+        Hh, G, dd, win, pool = 8, 2, 128, 512, 8
+        for T, B in ((64, 64), (4096, 1)):
+            ctx = 4096
+            blocks, pblocks = -(-ctx // page), -(-ctx // (page * pool))
+            kvs = [torch.randn(B * blocks, 2, G, page, dd, device=dev).to(torch.bfloat16) for _ in range(L)]
+            pks = [torch.randn(B * pblocks, 2, G, page, dd, device=dev).to(torch.bfloat16) for _ in range(L)]
+            bt = torch.arange(B * blocks, dtype=torch.int32, device=dev).view(B, blocks).contiguous()
+            pt = torch.arange(B * pblocks, dtype=torch.int32, device=dev).view(B, pblocks).contiguous()
+            q = (torch.randn(T, Hh * dd, device=dev) * dd ** -0.5).to(torch.bfloat16)
+            req = (torch.arange(T, device=dev) // (T // B)).to(torch.int32)
+            pos = (torch.arange(T, device=dev) % (T // B) + (ctx - T // B)).to(torch.int32)
+            o = torch.empty(T, Hh * dd, dtype=torch.bfloat16, device=dev)
+            res = {}
+            for form in ("pool", "keep", "window"):
+                keep = 4 if form == "keep" else 0
+                def call(kv, pk_):
+                    more = dict(pooled=(pk_, pt, pool)) if form == "pool" else {}
+                    if B > 1:
+                        reach = win + keep + (ctx // pool if form == "pool" else 0)
+                        ops.decode_attention(q, Hh * dd, o, kv, bt, None, T, req, pos, Hh, G, dd, win, 1.0,
+                                             ops.decode_splits(T, G * (-(-(Hh // G) // 8)), reach), keep_first=keep, **more)
+                    else:
+                        ops.prefill_attention(q, Hh * dd, o, kv, bt, t64, pos, Hh, G, dd, win, 1.0, keep_first=keep, **more)
+                t64 = torch.tensor([(k, min(64, T - k), 0) for k in range(0, T, 64)], dtype=torch.int32, device=dev)
+                res[form] = timed(lambda: [call(kv, pk_) for kv, pk_ in zip(kvs, pks)])
+            see = lambda p, form: min(p + 1, win) + (max(0, p + 1 - win) // pool if form == "pool" else 4 if form == "keep" else 0)
+            seen = {f: sum(see(int(p), f) for p in pos.tolist()) for f in res}
+            info = {}
+            for f, us in res.items():
+                info[f + "_us"] = round(us, 2)
+                if B > 1:
+                    info[f + "_frac_hbm"] = round(seen[f] * G * 2 * dd * 2 / us / 1e3 / pk["hbm_gbs"], 3)
+                else:
+                    info[f + "_frac_flops"] = round(Hh * 4 * dd * seen[f] / us / 1e6 / pk["bf16_tflops"], 3)
+            out(f"attention window {win} and blocks of {pool}, H{Hh} G{G} d{dd}, {B} requests x {T // B} tokens", res["pool"], **info)
+            slots = torch.zeros(T, dtype=torch.int32, device=dev) if B > 1 else torch.arange(T, dtype=torch.int32, device=dev)
+            batch = SimpleNamespace(req_of_token=req, positions=pos)
+            us = timed(lambda: [ops.pool_blocks(kv, bt, batch, slots, pk_, pool) for kv, pk_ in zip(kvs, pks)])
+            ends = int(((pos + 1) % pool == 0).sum())
+            out(f"pooled entries of {T} tokens ({ends} blocks)", us,
+                frac=round(ends * (pool + 1) * 2 * G * dd * 2 / us / 1e3 / pk["hbm_gbs"], 3))
     if on("moe"):
         # the routed experts' two grouped products (32 experts of 1,024 at width 2,048, 4 choices) beside the dense
         # model's gate|up and down products of equal work: decode by bytes of weights read, prompts by FLOP/s
@@ -1427,15 +1726,17 @@ def main():
     ap.add_argument("--warmup", type=int, default=5)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the named configuration (0: all)")
-    ap.add_argument("--mode", default="all", choices=["all", "decode", "prefill", "kernels", "dizatar", "rupulix", "mepatar", "kasarax"],
+    ap.add_argument("--mode", default="all", choices=["all", "decode", "prefill", "kernels", "dizatar", "rupulix", "mepatar", "kasarax",
+                                                           "sagizen"],
                     help="all: the contract's line; decode / prefill: one short measurement (for profiling); "
                          "kernels: the hot kernels one by one; dizatar / rupulix: prefill and decode of the Dizatar / Rupulix design at "
                          "layer sizes of real models beside the dense model of equal width; mepatar: the same for "
-                         "the Mepatar design beside Rupulix; kasarax: the same for the Kasarax design beside Mepatar")
-    ap.add_argument("--sizes", default="", help="--mode dizatar / rupulix / mepatar / kasarax: comma-separated subset of w1024, w2048")
+                         "the Mepatar design beside Rupulix; kasarax: the same for the Kasarax design beside Mepatar; "
+                         "sagizen: the same for the Sagizen design beside Mepatar and Kasarax")
+    ap.add_argument("--sizes", default="", help="--mode dizatar / rupulix / mepatar / kasarax / sagizen: comma-separated subset of w1024, w2048")
     ap.add_argument("--cases", default="", help="--mode kernels: comma-separated subset of sampling, decode_gemm, "
                     "decode_gemm_mid, decode_attention, prefill_gemm, prefill_attention, primitives, latent_attention, moe, "
-                    "talking_attention, rupulix_rows, mepatar_rows, kasarax_rows")
+                    "talking_attention, rupulix_rows, mepatar_rows, kasarax_rows, sagizen_rows")
     ap.add_argument("--batch", type=int, default=8, help="--mode decode: requests in the batch")
     ap.add_argument("--tokens", type=int, default=PREFILL_TOKENS, help="--mode prefill: prompt length")
     ap.add_argument("--context", type=int, default=CONTEXT, help="--mode decode: tokens each request holds")
@@ -1460,6 +1761,8 @@ def main():
         return run_mepatar(args)
     if args.mode == "kasarax":
         return run_kasarax(args)
+    if args.mode == "sagizen":
+        return run_sagizen(args)
     return run_ours(args)
 
 

@@ -1239,8 +1239,9 @@ def pool_blocks(kv_cache: torch.Tensor, block_table: torch.Tensor, batch, slots:
 def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, freq: torch.Tensor, rot_dims: int,
                       interleaved: bool, positions: torch.Tensor, slots, factor, H: int, G: int, d: int, dv: int,
                       D: int, norm_whole: bool = False, temp_coef: float = 0.0, temp_every: int = 0,
-                      out_dtype=None) -> torch.Tensor:
-    """Per token of ``qkv`` [T, H d + G d + G dv] (a view whose rows may be further apart): q and k RMS-normed,
+                      out_dtype=None, bias: torch.Tensor | None = None, pooled=None) -> torch.Tensor:
+    """Per token of ``qkv`` [T, H d + G d + G dv] (a view whose rows may be further apart), ``bias`` (float32, that many
+    numbers) added if given: q and k RMS-normed,
     per head over d (``q_norm`` / ``k_norm`` [d] float32) or, with ``norm_whole``, all q heads together and all k
     heads together (weights [H d] and [G d]); None: no norm.  Then their first ``rot_dims`` numbers rotated in
     pairs (2i, 2i + 1) (``interleaved``) or (i, i + rot_dims / 2) by position * ``freq[i]`` (float64), q head h
@@ -1248,7 +1249,9 @@ def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, f
     1 + ``temp_coef`` ln(floor((position + 1) / ``temp_every``) + 1).
     Returns q [T, H, D] in ``out_dtype`` (default: qkv's; 32-bit rows may be rounded to bfloat16 here, once); k and
     v go to place ``slots[t]`` of ``kv_cache`` [pages, 2, G, page, D] of that type (negative slot or None: no
-    write).  D >= max(d, dv): the rest of every row is zeros."""
+    write).  D >= max(d, dv): the rest of every row is zeros.
+    ``pooled`` = (entries, slots, pool, block table, batch), for steps in which every request brings one token: a token
+    that ends a block of ``pool`` tokens also leaves the block's entry, as ``pool_blocks`` does."""
     _check_rows(qkv, "qkv")
     _check(freq, "freq", torch.float64)
     _check(positions, "positions", torch.int32)
@@ -1259,7 +1262,7 @@ def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, f
     if out_dtype != qkv.dtype and qkv.dtype != torch.float32:
         raise KernelError("attention_prepare: only 32-bit rows can be written in another type")
     for w, name, n in ((q_norm, "q_norm", H * d if norm_whole else d), (k_norm, "k_norm", G * d if norm_whole else d),
-                       (factor, "factor", H)):
+                       (factor, "factor", H), (bias, "bias", qkv.shape[1])):
         if w is not None:
             _check(w, name, torch.float32)
             if w.numel() != n:
@@ -1271,14 +1274,26 @@ def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, f
         page_size = kv_cache.shape[3]
         if tuple(kv_cache.shape[1:]) != (2, G, page_size, D):
             raise KernelError(f"kv cache shape {tuple(kv_cache.shape)} does not match {G} heads of {D}")
+    entries = pslots = table = req = None
+    pool = 0
+    if pooled is not None:
+        entries, pslots, pool, table, batch = pooled
+        _check(entries, "entries", out_dtype)
+        _check(table, "block table", torch.int32)
+        _check(pslots, "entries' slots", torch.int32)
+        if not batch.decode_only or slots is None or entries.shape[1:] != kv_cache.shape[1:] or pool < 1:
+            raise KernelError("attention_prepare: pooled entries are written here in single-token steps only, in pages of "
+                              "the tokens' shape")
+        req = batch.req_of_token
     q = torch.empty((T, H, D), dtype=out_dtype, device=qkv.device)
     _ok(_fn("attention_prepare", "rg_attention_prepare")(
-        _ptr(qkv), c_int(_dtype_code(qkv)), c_int(qkv.stride(0)), _ptr(q), c_int(_dtype_code(q)),
+        _ptr(qkv), c_int(_dtype_code(qkv)), c_int(qkv.stride(0)), _ptr(bias), _ptr(q), c_int(_dtype_code(q)),
         _ptr(kv_cache if slots is not None else None),
         _ptr(q_norm), _ptr(k_norm), c_int(1 if norm_whole else 0), c_float(eps), _ptr(freq), c_int(rot_dims),
         c_int(1 if interleaved else 0), _ptr(positions), _ptr(slots), _ptr(factor), c_float(temp_coef),
         c_int(temp_every), c_int(T), c_int(H), c_int(G), c_int(d), c_int(dv), c_int(D),
-        c_int(page_size), _stream()), "attention_prepare")
+        c_int(page_size), c_int(pool), _ptr(table), c_int(table.shape[1] if table is not None else 0), _ptr(req),
+        _ptr(pslots), _ptr(entries), _stream()), "attention_prepare")
     return q
 
 

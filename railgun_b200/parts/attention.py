@@ -260,7 +260,7 @@ class NormedAttention(Mixer):
         names = ["q", "k", "v"] + (["g"] if p.get("out_gate") else [])
         self.out_gate = bool(p.get("out_gate"))
         self.w_qkv = torch.cat([tensors.get(b + n, env.dtype) for n in names], dim=0).contiguous()
-        self.b_qkv = self.b_o = None
+        self.b_qkv = self.b_o = self.prepare_bias = None
         bias = p.get("bias", True)
         if bias not in (True, False, None, "qkv"):
             raise ValueError(f"bias {bias!r} is not known; known: true, 'qkv', false")
@@ -307,6 +307,10 @@ class NormedAttention(Mixer):
             self.sink = tensors.get(b + "sink", torch.float32).contiguous()
         self.K = self._taps(p)
         self.taps = None
+        if self.b_qkv is not None and self.K == 0:
+            # nothing stands between the product and the per-token kernel: the bias is added there, in 32-bit, and
+            # the product is free to run on the kernels that have no bias
+            self.prepare_bias, self.b_qkv = self.b_qkv[:self.C].float().contiguous(), None
         if self.K >= 1:
             self.taps = torch.cat([tensors.get(b + n, torch.float32) for n in ("q.conv", "k.conv", "v.conv")],
                                   dim=0).t().contiguous()                                  # [taps, channels]
@@ -321,7 +325,7 @@ class NormedAttention(Mixer):
 
     def input_weight(self):
         """The matrix of this mixer's first product, for a wrapper that computes the first products of several
-        mixers that read the same rows as one (None: the product has a bias and stays here)."""
+        mixers that read the same rows as one (None: the product adds a bias itself and stays here)."""
         return self.w_qkv if self.b_qkv is None else None
 
     def adopt_input_weight(self, view):
@@ -344,16 +348,18 @@ class NormedAttention(Mixer):
             if writes and state is not None:
                 ops.conv_state_update(proj, 0, state, batch)
         slots = batch.slot_mapping[pages.group] if writes else None
+        table = batch.block_table[pages.group]
+        blocks = cache.parts[1] if self.pool else None
+        pooled = None
+        if self.pool and writes and batch.decode_only:
+            pooled = (blocks.kv, batch.slot_mapping[blocks.group], self.pool, table, batch)
         q = ops.attention_prepare(qkv, pages.kv, self.q_norm, self.k_norm, self.eps, self.freq, self.rot_dims,
                                   self.interleaved, batch.positions, slots, self.factor, H, G, d, dv, D,
                                   norm_whole=self.norm_whole, temp_coef=self.temp_coef, temp_every=self.temp_every,
-                                  out_dtype=self.env.dtype)
-        pooled = None
+                                  out_dtype=self.env.dtype, bias=self.prepare_bias, pooled=pooled)
         if self.pool:
-            blocks = cache.parts[1]
-            if writes:
-                ops.pool_blocks(pages.kv, batch.block_table[pages.group], batch, batch.slot_mapping[blocks.group],
-                                blocks.kv, self.pool)
+            if writes and not batch.decode_only:
+                ops.pool_blocks(pages.kv, table, batch, batch.slot_mapping[blocks.group], blocks.kv, self.pool)
             pooled = (blocks.kv, batch.block_table[blocks.group], self.pool)
         gate = proj[:, C:] if self.out_gate else None
         return self.attend(q.view(-1, H * D), batch, pages, gate, pooled, out, out_scale)
