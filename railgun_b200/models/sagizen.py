@@ -38,7 +38,7 @@ def _mixer_spec(c: SagizenConfig, L) -> PartSpec:
     left = PartSpec("gqa_attention", dict(
         hidden_size=W, num_heads=a.heads, num_kv_heads=a.kv_heads, head_dim=a.dim, v_dim=a.vdim, scale=a.scale,
         rot_dims=a.rot_dims, rot_base=a.rot_base, rot_factor=a.rot_factor, rot_layout="half", eps=c.norm_eps,
-        window=a.size, pool=a.pool, bias="qkv", qk_norm="unit", head_temp=False, base="mix.left."))
+        window=a.size, pool=a.pool, bias="qkv", bias_in="rows", qk_norm="unit", head_temp=False, base="mix.left."))
     right = PartSpec("rwkv", dict(hidden_size=W, num_heads=s.heads, head_dim=s.dim, eps=c.norm_eps, base="mix.right."))
     return PartSpec("parallel", dict(branches=((left, m.left_scale), (right, m.right_scale))))
 

@@ -143,16 +143,16 @@ class NormedAttention(Mixer):
     """Grouped-query softmax attention with the options that recent designs add to it, each a parameter:
     biases on the four projections (or on q, k and v only), an RMS norm on q and k before the rotation (per head, with
     one weight vector for all q heads and one for all k heads, or without weights, which is the same before and
-    after a rotation, or over the whole of q and the whole of k with weights of that size), a short causal convolution per channel on q, k and v directly behind the projections, rotation of
-    the first ``rot_dims`` numbers of a head in either layout, its frequencies divided by a constant (linear scaling),
-    a learned number per head on the scores
-    (``head_temp``), a query factor that grows with the logarithm of the position (``q_temp``), a sink in the
-    softmax's denominator (of score 0, or a learned score per head), a sigmoid gate per head on the heads'
-    outputs, values of another size than keys, and a sliding window that keeps the request's first
-    ``keep_first`` tokens visible (at their true positions) or, with ``pool``, sees what has left it as the means of
-    the keys and of the values of blocks of ``pool`` tokens that lie wholly before the window (in a second group of
-    pages, one entry per block, written by the step that completes the block; the tokens' pages are kept until their
-    block is complete).
+    after a rotation, or over the whole of q and the whole of k with weights of that size), a short causal
+    convolution per channel on q, k and v directly behind the projections, rotation of the first ``rot_dims``
+    numbers of a head in either layout, its frequencies divided by a constant (linear scaling), a learned number
+    per head on the scores (``head_temp``), a query factor that grows with the logarithm of the position
+    (``q_temp``), a sink in the softmax's denominator (of score 0, or a learned score per head), a sigmoid gate per
+    head on the heads' outputs, values of another size than keys, and a sliding window that keeps the request's
+    first ``keep_first`` tokens visible (at their true positions) or, with ``pool``, sees what has left it as the
+    means of the keys and of the values of blocks of ``pool`` tokens that lie wholly before the window (in a second
+    group of pages, one entry per block, written by the step that completes the block; the tokens' pages are kept
+    until their block is complete).
 
     Keys, queries and values are padded with zeros to one size D (a multiple of 16 that holds both), so the
     key/value pages and the attention kernels are the ordinary ones; the output product's matrix gets zero
@@ -164,7 +164,9 @@ class NormedAttention(Mixer):
     head_dim^-1/2), ``rot_dims``, ``rot_base``, ``rot_layout`` ("interleaved": pairs (2i, 2i + 1), or "half":
     pairs (i, i + rot_dims/2)), ``rot_factor`` (what the frequencies are divided by, default 1), ``eps`` (of the q and
     k norms), ``window`` (0: none), ``keep_first``, ``pool`` (0: none),
-    ``bias`` (true, the default; "qkv": not on the output; false), ``head_temp`` (default true), ``qk_norm`` (true, the
+    ``bias`` (true, the default; "qkv": not on the output; false), ``bias_in`` (where the bias of q, k and v is added:
+    "product", the default, or "rows": by the per-token kernel behind it, in 32-bit, which leaves the product to the
+    kernels that have no bias; not with a convolution), ``head_temp`` (default true), ``qk_norm`` (true, the
     default: per head; "unit": per head without weights; "whole"; false),
     ``q_temp`` (None, or (coef, every): q at position p times 1 + coef ln(floor((p + 1) / every) + 1)),
     ``sink`` (None, "zero" or "learned"), ``out_gate`` (default false), ``conv`` (taps; 0: none; 1: a factor per
@@ -307,9 +309,9 @@ class NormedAttention(Mixer):
             self.sink = tensors.get(b + "sink", torch.float32).contiguous()
         self.K = self._taps(p)
         self.taps = None
-        if self.b_qkv is not None and self.K == 0:
-            # nothing stands between the product and the per-token kernel: the bias is added there, in 32-bit, and
-            # the product is free to run on the kernels that have no bias
+        if p.get("bias_in") == "rows" and self.b_qkv is not None:
+            if self.K:
+                raise ValueError("bias_in 'rows' needs the per-token kernel directly behind the product: no convolution")
             self.prepare_bias, self.b_qkv = self.b_qkv[:self.C].float().contiguous(), None
         if self.K >= 1:
             self.taps = torch.cat([tensors.get(b + n, torch.float32) for n in ("q.conv", "k.conv", "v.conv")],

@@ -309,7 +309,7 @@ def test_pooled_entries_alone(G, D, page, pool, dtype):
     kernel); a padding row writes nothing; entries of blocks that are not complete stay as they were."""
     from railgun_b200 import ops
     rng = np.random.default_rng(page + pool)
-    n = 3 * page * max(1, pool // page) + pool + 3
+    n = 3 * page * max(1, pool // page) + 3 * pool + 3
     k, v = (torch.tensor(rng.normal(size=(n, G, D)), dtype=TORCH[dtype]) for _ in range(2))
     pages = -(-n // page)
     order = rng.permutation(pages + 2)[:pages].tolist()
