@@ -1623,11 +1623,13 @@ def run_kernels(args):
                 dt, g = ops.ssd_prepare(projs[0][:, inner + C:], dtb, A)
                 us = timed(lambda: [ops.state_scan(x[:, inner + G * N:], x[:, inner:inner + G * N], x[:, :inner], st, batch, H, N,
                                                    dv, g=g, beta=dt, rule="scalar", skip=D) for x, st in zip(xbc, sts)])
+                usc = timed(lambda: [ops.ssd_chunk_scan(x, dt, A, D, st, batch, H, G, N, dv) for x, st in zip(xbc, sts)])
                 qd = [torch.randn(T, Hq * dd, device=dev) * 0.1 for _ in range(L)]
                 vd = [torch.randn(T, Hd * dd, device=dev) for _ in range(L)]
                 gd = torch.rand(T, Hd, device=dev)
                 us2 = timed(lambda: [ops.state_scan(q, q, v, st, batch, Hd, dd, dd, g=gd, beta=gd) for q, v, st in zip(qd, vd, std)])
-                out(f"scan H{H} {N} x {dv} T{T}", us, frac=gbs(T * (C + inner) * 4, us), delta_us=round(us2, 2),
+                out(f"scan H{H} {N} x {dv} T{T}", us, frac=gbs(T * (C + inner) * 4, us), chunked_us=round(usc, 2),
+                    chunked_frac=gbs(T * (C + inner) * 4, usc), delta_us=round(us2, 2),
                     delta_frac=gbs(T * (2 * Hq + 2 * Hd) * dd * 4, us2))
                 us = timed(lambda: [ops.ssd_prepare(p[:, inner + C:], dtb, A) for p in projs])
                 out(f"step sizes and decays H{H} T{T}", us, frac=gbs(T * H * 12, us))

@@ -127,19 +127,38 @@ extern "C" int rg_ssd_step(const float* proj, int ld, int x_off, int dt_off, con
 }
 
 // o [T, n] float; z: rows z_ld apart (type Z).  One block per (token, group of n / groups numbers); the gated numbers
-// wait in shared memory for the group's root mean square.  With `raw` (rows raw_ld apart, C numbers) the block of a
-// token's first group also moves the convolution state of the token's request on by that one token (single-token steps).
+// wait in shared memory for the group's root mean square.  With `raw` (rows raw_ld apart, C numbers) further blocks of
+// the same launch move the convolution state of the token's request on by that one token (single-token steps).
 template <typename Z, typename O>
 __global__ void gate_group_norm_kernel(const float* __restrict__ o, const Z* __restrict__ z, int z_ld,
                                        const float* __restrict__ weight, float eps, O* __restrict__ out, int n, int gs,
-                                       const float* __restrict__ raw, int raw_ld, float* __restrict__ conv_state,
-                                       const int* __restrict__ req_of_token, const int* __restrict__ start_pos,
-                                       const int* __restrict__ slots, int C, int K) {
+                                       int groups, const float* __restrict__ raw, int raw_ld,
+                                       float* __restrict__ conv_state, const int* __restrict__ req_of_token,
+                                       const int* __restrict__ start_pos, const int* __restrict__ slots, int C, int K) {
     extern __shared__ __align__(16) float y[];        // [gs]
     __shared__ float scratch[33];
     pdl_wait();
     pdl_trigger();
-    const int t = blockIdx.x, base = blockIdx.y * gs;
+    const int t = blockIdx.x;
+    if ((int)blockIdx.y >= groups) {
+        const int c = (blockIdx.y - groups) * blockDim.x + threadIdx.x;
+        const int r = req_of_token[t], slot = slots[r];
+        if (slot < 0 || c >= C) return;
+        const bool has_past = start_pos[r] > 0;
+        float* st = conv_state + (size_t)slot * (K - 1) * C + c;
+        const float now = raw[(size_t)t * raw_ld + c];
+        for (int j0 = 0; j0 < K - 2; j0 += 4) {       // four rows at a time, each read before the one above it is written
+            float v[4];
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[j] = has_past && j0 + j < K - 2 ? st[(size_t)(j0 + j + 1) * C] : 0.f;
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (j0 + j < K - 2) st[(size_t)(j0 + j) * C] = v[j];
+        }
+        st[(size_t)(K - 2) * C] = now;
+        return;
+    }
+    const int base = blockIdx.y * gs;
     const float* src = o + (size_t)t * n + base;
     const Z* zr = z + (size_t)t * z_ld + base;
     float ss = 0.f;
@@ -151,16 +170,6 @@ __global__ void gate_group_norm_kernel(const float* __restrict__ o, const Z* __r
     const float inv = rsqrtf(block_sum(ss, scratch) / (float)gs + eps);
     for (int i = threadIdx.x; i < gs; i += blockDim.x)
         out[(size_t)t * n + base + i] = from_f32<O>(y[i] * inv * weight[base + i]);
-    if (raw && K > 1) {
-        const int r = req_of_token[t], slot = slots[r];
-        if (slot < 0) return;
-        const bool has_past = start_pos[r] > 0;
-        float* st = conv_state + (size_t)slot * (K - 1) * C;
-        for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < C; c += gridDim.y * blockDim.x) {
-            for (int j = 0; j < K - 2; ++j) st[(size_t)j * C + c] = has_past ? st[(size_t)(j + 1) * C + c] : 0.f;
-            st[(size_t)(K - 2) * C + c] = raw[(size_t)t * raw_ld + c];
-        }
-    }
 }
 
 extern "C" int rg_gate_group_norm(const float* o, const void* z, int z_dtype, int z_ld, const float* weight, float eps,
@@ -174,13 +183,15 @@ extern "C" int rg_gate_group_norm(const float* o, const void* z, int z_dtype, in
     if (smem > 200 * 1024) return RG_ERR_UNSUPPORTED;
     int threads = 64;
     while (threads < 512 && threads * 4 < gs) threads <<= 1;
-    dim3 grid(T, groups);
+    const int conv_blocks = raw && K > 1 ? (C + threads - 1) / threads : 0;
+    if (groups + conv_blocks > 65535) return RG_ERR_UNSUPPORTED;
+    dim3 grid(T, groups + conv_blocks);
     cudaStream_t s = (cudaStream_t)stream;
 #define SSD_GGN(Z, O) { if (smem > 47 * 1024) { \
             const int e = (int)cudaFuncSetAttribute(gate_group_norm_kernel<Z, O>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e) return e; } \
         return rg_launch(gate_group_norm_kernel<Z, O>, grid, dim3(threads), smem, s, 1, o, (const Z*)z, z_ld, weight, eps, \
-                         (O*)out, n, gs, raw, raw_ld, conv_state, req_of_token, start_pos, slots, C, K); }
+                         (O*)out, n, gs, groups, raw, raw_ld, conv_state, req_of_token, start_pos, slots, C, K); }
     if (z_dtype == RG_DTYPE_BF16 && out_dtype == RG_DTYPE_BF16) SSD_GGN(bf16, bf16)
     if (z_dtype == RG_DTYPE_F32 && out_dtype == RG_DTYPE_BF16) SSD_GGN(float, bf16)
     if (z_dtype == RG_DTYPE_F32 && out_dtype == RG_DTYPE_F32) SSD_GGN(float, float)

@@ -1,0 +1,321 @@
+// The recurrence of Mamba-2 over portions of prompts, in chunks of 64 tokens side by side instead of token by token:
+//
+//   S <- g_t S + dt_t B_t x_t^T,  o_t = S^T C_t + D x_t,   g_t = exp(a_t),  a_t = -exp(A_log) dt_t
+//
+// With c_i = a_1 + .. + a_i inside a chunk of L tokens and S the state before it,
+//   o_i   = exp(c_i) S^T C_i + sum_(j <= i) exp(c_i - c_j) dt_j (B_j . C_i) x_j + D x_i
+//   S_end = exp(c_L) S + sum_j exp(c_L - c_j) dt_j B_j x_j^T
+// so that everything but the pass from chunk to chunk is products.  Three kernels:
+//   chunk_states   per (chunk, head): the sum in S_end, and exp(c_L); per (chunk, group): all B_j . C_i
+//   chunk_pass     per (request, head, number of S): S before every chunk, and the last one into the request's slot
+//   chunk_outputs  per (chunk, head): o
+// (the block decomposition of Dao and Gu, "Transformers are SSMs: Generalized Models and Efficient Algorithms Through
+// Structured State Space Duality").  The products are 32-bit fused multiply-adds; the exponents' sums are 64-bit, since
+// their differences are small beside them where a head forgets fast.
+//
+// The step's tokens are packed request by request (cu_seqlens); a request's chunks start at its first token of the step.
+#include "common.cuh"
+
+#define CH 64                 // tokens per chunk
+#define TILE 64               // rows and columns of a block's output (columns: 64 or 128)
+#define PITCH (TILE + 4)
+#define NTH 256
+
+// Chunk number c of the step: its request, first token and number of tokens; false beyond the last one.
+__device__ __forceinline__ bool find_chunk(const int* __restrict__ cu, int R, int c, int& r, int& lo, int& n) {
+    for (r = 0; r < R; ++r) {
+        const int len = cu[r + 1] - cu[r], k = (len + CH - 1) / CH;
+        if (c < k) {
+            lo = cu[r] + c * CH;
+            n = min(CH, len - c * CH);
+            return true;
+        }
+        c -= k;
+    }
+    return false;
+}
+
+// c_i of the chunk's tokens for head h (64-bit), by the block's first warp; dt of the tokens into sdt.
+__device__ __forceinline__ void chunk_sums(const float* __restrict__ dt, float A_log, int lo, int n, int H, int h,
+                                           double* __restrict__ cum, float* __restrict__ sdt) {
+    if (threadIdx.x < 32) {
+        const int i0 = 2 * threadIdx.x, i1 = i0 + 1;
+        const float d0 = i0 < n ? dt[(size_t)(lo + i0) * H + h] : 0.f, d1 = i1 < n ? dt[(size_t)(lo + i1) * H + h] : 0.f;
+        const float rate = -expf(A_log);
+        const double a0 = (double)(rate * d0), a1 = (double)(rate * d1);
+        double s = a0 + a1;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double up = __shfl_up_sync(0xffffffffu, s, o);
+            if ((int)threadIdx.x >= o) s += up;
+        }
+        cum[i0] = s - a1;
+        cum[i1] = s;
+        sdt[i0] = d0;
+        sdt[i1] = d1;
+    }
+}
+
+// dst[k][i] = src row i, number k0 + k (rows ld apart, n rows of N numbers; zeros elsewhere), for 64 x 64, times scale[i].
+// A warp reads 4 rows x 8 neighbouring numbers at a time and writes 32 different banks.
+__device__ __forceinline__ void load_transposed(float (*__restrict__ dst)[PITCH], const float* __restrict__ src, size_t ld,
+                                                int n, int N, int k0, const float* __restrict__ scale) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int kl = lane & 7, il = lane >> 3;
+#pragma unroll 4
+    for (int p = warp; p < (TILE / 8) * (TILE / 4); p += NTH / 32) {
+        const int k = (p & 7) * 8 + kl, i = (p >> 3) * 4 + il;
+        float v = i < n && k0 + k < N ? src[(size_t)i * ld + k0 + k] : 0.f;
+        if (scale) v *= scale[i];
+        dst[k][i] = v;
+    }
+}
+
+// acc[4][4 W] += A[k][4 rows]^T B[k][4 W columns] over kn values of k.  Thread (ty, tx): rows 4 ty .., columns 4 tx .. (+ 64)
+template <int W>
+__device__ __forceinline__ void multiply(float (&acc)[4][4 * W], const float (*__restrict__ A)[PITCH],
+                                         const float (*__restrict__ B)[TILE * W + 4], int kn, int ty, int tx) {
+#pragma unroll 4
+    for (int k = 0; k < kn; ++k) {
+        const float4 a = *reinterpret_cast<const float4*>(&A[k][4 * ty]);
+#pragma unroll
+        for (int w = 0; w < W; ++w) {
+            const float4 b = *reinterpret_cast<const float4*>(&B[k][TILE * w + 4 * tx]);
+            acc[0][4 * w] += a.x * b.x; acc[0][4 * w + 1] += a.x * b.y; acc[0][4 * w + 2] += a.x * b.z; acc[0][4 * w + 3] += a.x * b.w;
+            acc[1][4 * w] += a.y * b.x; acc[1][4 * w + 1] += a.y * b.y; acc[1][4 * w + 2] += a.y * b.z; acc[1][4 * w + 3] += a.y * b.w;
+            acc[2][4 * w] += a.z * b.x; acc[2][4 * w + 1] += a.z * b.y; acc[2][4 * w + 2] += a.z * b.z; acc[2][4 * w + 3] += a.z * b.w;
+            acc[3][4 * w] += a.w * b.x; acc[3][4 * w + 1] += a.w * b.y; acc[3][4 * w + 2] += a.w * b.z; acc[3][4 * w + 3] += a.w * b.w;
+        }
+    }
+}
+
+// x, B, C: rows ld apart (head h's x at column h dv, group g's B and C at column g N).  sums [chunks, H, dv, N], decays
+// [chunks, H], dots [chunks, G, 64, 64] = B_j . C_i at [j][i].  grid: chunks, H (tiles of S: z) and then G (z = 0).
+template <int W>
+__global__ void __launch_bounds__(NTH)
+chunk_states_kernel(const float* __restrict__ x, const float* __restrict__ B, const float* __restrict__ C, int ld,
+                    const float* __restrict__ dt, const float* __restrict__ A_log, const int* __restrict__ cu, int R,
+                    float* __restrict__ sums, float* __restrict__ decays, float* __restrict__ dots, int H, int G, int N,
+                    int dv, int ntiles) {
+    extern __shared__ __align__(16) float sm[];
+    float (*sA)[PITCH] = reinterpret_cast<float (*)[PITCH]>(sm);                            // [CH][PITCH]
+    float (*sB)[TILE * W + 4] = reinterpret_cast<float (*)[TILE * W + 4]>(sm + CH * PITCH);     // [CH][TILE W + 4]
+    __shared__ double cum[CH];
+    __shared__ float sdt[CH];
+    pdl_wait();
+    pdl_trigger();
+    int r, lo, n;
+    if (!find_chunk(cu, R, blockIdx.x, r, lo, n)) return;
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    float acc[4][4 * W];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4 * W; ++j) acc[i][j] = 0.f;
+    if ((int)blockIdx.y >= H) {
+        if (blockIdx.z > 0) return;
+        const int g = blockIdx.y - H;
+        float (*sC)[PITCH] = reinterpret_cast<float (*)[PITCH]>(sm + CH * PITCH);
+        float a1[4][4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) a1[i][j] = 0.f;
+        for (int k0 = 0; k0 < N; k0 += TILE) {
+            load_transposed(sA, B + (size_t)lo * ld + (size_t)g * N, ld, n, N, k0, nullptr);
+            load_transposed(sC, C + (size_t)lo * ld + (size_t)g * N, ld, n, N, k0, nullptr);
+            __syncthreads();
+            multiply<1>(a1, sA, sC, min(TILE, N - k0), ty, tx);
+            __syncthreads();
+        }
+        float* out = dots + ((size_t)blockIdx.x * G + g) * CH * CH;
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            *reinterpret_cast<float4*>(out + (4 * ty + i) * CH + 4 * tx) = make_float4(a1[i][0], a1[i][1], a1[i][2], a1[i][3]);
+        return;
+    }
+    const int h = blockIdx.y, grp = h / (H / G);
+    const int j0 = (blockIdx.z / ntiles) * TILE, n0 = (blockIdx.z % ntiles) * TILE * W;      // columns of S, rows of S
+    chunk_sums(dt, A_log[h], lo, n, H, h, cum, sdt);
+    __syncthreads();
+    const double end = cum[CH - 1];
+    for (int e = threadIdx.x; e < CH * TILE; e += NTH) {
+        const int t = e / TILE, j = e - t * TILE;
+        sA[t][j] = t < n && j0 + j < dv
+                       ? x[(size_t)(lo + t) * ld + (size_t)h * dv + j0 + j] * sdt[t] * expf((float)(end - cum[t])) : 0.f;
+    }
+    for (int e = threadIdx.x; e < CH * TILE * W; e += NTH) {
+        const int t = e / (TILE * W), k = e - t * TILE * W;
+        sB[t][k] = t < n && n0 + k < N ? B[(size_t)(lo + t) * ld + (size_t)grp * N + n0 + k] : 0.f;
+    }
+    __syncthreads();
+    multiply<W>(acc, sA, sB, n, ty, tx);
+    float* out = sums + ((size_t)blockIdx.x * H + h) * dv * N;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int j = j0 + 4 * ty + i;
+        if (j >= dv) continue;
+#pragma unroll
+        for (int w = 0; w < W; ++w) {
+            const int k = n0 + TILE * w + 4 * tx;
+            if (N % 4 == 0) {
+                if (k < N) *reinterpret_cast<float4*>(out + (size_t)j * N + k) =
+                    make_float4(acc[i][4 * w], acc[i][4 * w + 1], acc[i][4 * w + 2], acc[i][4 * w + 3]);
+            } else {
+#pragma unroll
+                for (int q = 0; q < 4; ++q)
+                    if (k + q < N) out[(size_t)j * N + k + q] = acc[i][4 * w + q];
+            }
+        }
+    }
+    if (blockIdx.z == 0 && threadIdx.x == 0) decays[(size_t)blockIdx.x * H + h] = expf((float)end);
+}
+
+// sums [chunks, H, dv N]: each chunk's sum becomes the state before the chunk.  V numbers per thread.
+template <int V>
+__global__ void chunk_pass_kernel(float* __restrict__ sums, const float* __restrict__ decays, float* __restrict__ state,
+                                  const int* __restrict__ cu, const int* __restrict__ start_pos,
+                                  const int* __restrict__ slots, int H, int M) {
+    pdl_wait();
+    pdl_trigger();
+    const int r = blockIdx.y;
+    const long long e = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (e >= (long long)H * M) return;
+    const int h = (int)(e / M);
+    int c0 = 0;
+    for (int q = 0; q < r; ++q) c0 += (cu[q + 1] - cu[q] + CH - 1) / CH;
+    const int nc = (cu[r + 1] - cu[r] + CH - 1) / CH;
+    const int slot = slots[r];
+    float S[V];
+#pragma unroll
+    for (int i = 0; i < V; ++i) S[i] = 0.f;
+    float* st = state + (size_t)(slot >= 0 ? slot : 0) * H * M + e;
+    if (slot >= 0 && start_pos[r] > 0) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) S[i] = st[i];
+    }
+    float* p = sums + (size_t)c0 * H * M + e;
+    const float* dec = decays + (size_t)c0 * H + h;
+    const size_t step = (size_t)H * M;
+    constexpr int U = 4;                              // chunks in flight
+    for (int c = 0; c < nc; c += U) {
+        float u[U][V], d[U];
+#pragma unroll
+        for (int k = 0; k < U; ++k) {
+            if (c + k < nc) {
+                d[k] = dec[(size_t)(c + k) * H];
+                if (V == 4) {
+                    const float4 q = *reinterpret_cast<const float4*>(p + (c + k) * step);
+                    u[k][0] = q.x; u[k][1 % V] = q.y; u[k][2 % V] = q.z; u[k][3 % V] = q.w;
+                } else {
+                    u[k][0] = p[(c + k) * step];
+                }
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < U; ++k) {
+            if (c + k < nc) {
+                if (V == 4) *reinterpret_cast<float4*>(p + (c + k) * step) = make_float4(S[0], S[1 % V], S[2 % V], S[3 % V]);
+                else p[(c + k) * step] = S[0];
+#pragma unroll
+                for (int i = 0; i < V; ++i) S[i] = S[i] * d[k] + u[k][i];
+            }
+        }
+    }
+    if (slot >= 0) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) st[i] = S[i];
+    }
+}
+
+// before [chunks, H, dv, N]: the state before every chunk.  o [T, H, dv].  grid: chunks, H, tiles of 64 columns.
+__global__ void __launch_bounds__(NTH)
+chunk_outputs_kernel(const float* __restrict__ x, const float* __restrict__ C, int ld, const float* __restrict__ dt,
+                     const float* __restrict__ A_log, const float* __restrict__ D, const int* __restrict__ cu, int R,
+                     const float* __restrict__ before, const float* __restrict__ dots, float* __restrict__ o, int H, int G,
+                     int N, int dv) {
+    __shared__ __align__(16) float sA[CH][PITCH];
+    __shared__ __align__(16) float sB[CH][PITCH];
+    __shared__ double cum[CH];
+    __shared__ float sdt[CH], grown[CH];
+    pdl_wait();
+    pdl_trigger();
+    int r, lo, n;
+    if (!find_chunk(cu, R, blockIdx.x, r, lo, n)) return;
+    const int h = blockIdx.y, grp = h / (H / G), j0 = blockIdx.z * TILE;
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    chunk_sums(dt, A_log[h], lo, n, H, h, cum, sdt);
+    __syncthreads();
+    if (threadIdx.x < CH) grown[threadIdx.x] = expf((float)cum[threadIdx.x]);
+    // within the chunk
+    const float* d = dots + ((size_t)blockIdx.x * G + grp) * CH * CH;
+    for (int e = threadIdx.x; e < CH * CH; e += NTH) {
+        const int j = e / CH, i = e - j * CH;
+        sA[j][i] = j <= i && i < n ? d[e] * sdt[j] * expf((float)(cum[i] - cum[j])) : 0.f;
+    }
+    for (int e = threadIdx.x; e < CH * TILE; e += NTH) {
+        const int t = e / TILE, j = e - t * TILE;
+        sB[t][j] = t < n && j0 + j < dv ? x[(size_t)(lo + t) * ld + (size_t)h * dv + j0 + j] : 0.f;
+    }
+    __syncthreads();
+    float acc[4][4];
+    const float skip = D[h];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = skip * sB[4 * ty + i][4 * tx + j];
+    multiply<1>(acc, sA, sB, min(n, 4 * (ty | 1) + 4), ty, tx);     // token j counts for the tokens from j on only
+    // from the state before it
+    const float* S = before + (((size_t)blockIdx.x * H + h) * dv + j0) * N;
+    for (int k0 = 0; k0 < N; k0 += TILE) {
+        __syncthreads();
+        load_transposed(sA, C + (size_t)lo * ld + (size_t)grp * N, ld, n, N, k0, grown);
+        load_transposed(sB, S, N, min(TILE, dv - j0), N, k0, nullptr);
+        __syncthreads();
+        multiply<1>(acc, sA, sB, min(TILE, N - k0), ty, tx);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int t = 4 * ty + i;
+        if (t >= n) continue;
+        float* out = o + ((size_t)(lo + t) * H + h) * dv + j0 + 4 * tx;
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            if (j0 + 4 * tx + j < dv) out[j] = acc[i][j];
+    }
+}
+
+// Scratch of the caller: sums [chunks, H, dv, N], decays [chunks, H], dots [chunks, G, 64, 64], with chunks at least
+// T / 64 + R (rounded down).
+extern "C" int rg_ssd_chunk_scan(const float* x, const float* B, const float* C, int ld, const float* dt, const float* A_log,
+                                 const float* D, float* state, const int* cu_seqlens, const int* start_pos, const int* slots,
+                                 float* sums, float* decays, float* dots, float* o, int T, int R, int H, int G, int N, int dv,
+                                 void* stream) {
+    if (T <= 0 || R <= 0) return 0;
+    if (H < 1 || G < 1 || H % G || N < 1 || dv < 1 || H + G > 65535 || R > 65535) return RG_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int chunks = T / CH + R;
+    const int wide = N > TILE ? 2 : 1;
+    const int jt = (dv + TILE - 1) / TILE, nt = (N + TILE * wide - 1) / (TILE * wide);
+    if (jt * nt > 65535) return RG_ERR_UNSUPPORTED;
+    dim3 g1(chunks, H + G, jt * nt);
+    const size_t smem = (size_t)CH * (PITCH + TILE * wide + 4) * sizeof(float);
+    int e = 0;
+#define SSD_STATES(W) { \
+        if (smem > 46 * 1024) e = (int)cudaFuncSetAttribute(chunk_states_kernel<W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (e == 0) e = rg_launch(chunk_states_kernel<W>, g1, dim3(NTH), smem, s, 1, x, B, C, ld, dt, A_log, cu_seqlens, R, \
+                                  sums, decays, dots, H, G, N, dv, nt); }
+    if (wide == 2) SSD_STATES(2) else SSD_STATES(1)
+#undef SSD_STATES
+    if (e) return e;
+    const int M = dv * N;
+    const bool vec = M % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    const long long work = vec ? (long long)H * M / 4 : (long long)H * M;
+    dim3 g2((unsigned)((work + 255) / 256), R);
+    e = vec ? rg_launch(chunk_pass_kernel<4>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M)
+            : rg_launch(chunk_pass_kernel<1>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M);
+    if (e) return e;
+    dim3 g3(chunks, H, jt);
+    return rg_launch(chunk_outputs_kernel, g3, dim3(NTH), 0, s, 1, x, C, ld, dt, A_log, D, cu_seqlens, R, (const float*)sums,
+                     (const float*)dots, o, H, G, N, dv);
+}

@@ -207,42 +207,50 @@ extern "C" int rg_shift_mixes(const void* h, int dtype, const float* mu, float* 
 }
 
 // a [T, rank] float; w [N, rank] (type A), w0 [N]; out [T, N] float = exp(-exp(w . tanh(a) + w0)).  A block takes TT
-// tokens and 64 channels, the rank in pieces of 64 through shared memory; a thread has TT / 16 tokens x 4 channels.
+// tokens and CC channels, the rank in pieces of 64 through shared memory; a thread has TT / 16 tokens x CC / 16 channels
+// (few tokens: 16 x 16, so that a step of single tokens has blocks enough; portions: 64 x 64).
 #define LD_RANK 64
-template <int TT, typename A>
+template <int TT, int CC, typename A>
 __global__ void __launch_bounds__(256)
 lowrank_decay_kernel(const float* __restrict__ a, const A* __restrict__ w, const float* __restrict__ w0,
                      float* __restrict__ out, int T, int N, int rank) {
-    constexpr int NT = TT / 16;
+    constexpr int NT = TT / 16, NC = CC / 16;
     __shared__ __align__(16) float sa[LD_RANK][TT + 4];
-    __shared__ __align__(16) float sw[LD_RANK][64 + 4];
+    __shared__ __align__(16) float sw[LD_RANK][CC + 4];
     pdl_wait();
     pdl_trigger();
-    const int t0 = blockIdx.x * TT, n0 = blockIdx.y * 64;
-    const int tc = threadIdx.x & 15, tr = threadIdx.x >> 4;     // channels 4 tc .. + 3, tokens tr NT .. + NT - 1
-    float acc[NT][4];
+    const int t0 = blockIdx.x * TT, n0 = blockIdx.y * CC;
+    const int tc = threadIdx.x & 15, tr = threadIdx.x >> 4;     // channels NC tc .. + NC - 1, tokens tr NT .. + NT - 1
+    float acc[NT][NC];
 #pragma unroll
     for (int x = 0; x < NT; ++x)
 #pragma unroll
-        for (int y = 0; y < 4; ++y) acc[x][y] = 0.f;
+        for (int y = 0; y < NC; ++y) acc[x][y] = 0.f;
     for (int k0 = 0; k0 < rank; k0 += LD_RANK) {
         const int n = min(LD_RANK, rank - k0);
+        // 8 neighbouring k of 4 rows at a time: whole sectors in, different banks out
+#pragma unroll 4
         for (int e = threadIdx.x; e < TT * LD_RANK; e += 256) {
-            const int t = e / LD_RANK, k = e - t * LD_RANK;
+            const int k = (e & 7) + ((e >> 5) & 7) * 8, t = ((e >> 3) & 3) + (e >> 8) * 4;
             sa[k][t] = (k < n && t0 + t < T) ? tanhf(a[(size_t)(t0 + t) * rank + k0 + k]) : 0.f;
         }
-        for (int e = threadIdx.x; e < 64 * LD_RANK; e += 256) {
-            const int c = e / LD_RANK, k = e - c * LD_RANK;
+#pragma unroll 4
+        for (int e = threadIdx.x; e < CC * LD_RANK; e += 256) {
+            const int k = (e & 7) + ((e >> 5) & 7) * 8, c = ((e >> 3) & 3) + (e >> 8) * 4;
             sw[k][c] = (k < n && n0 + c < N) ? to_f32(w[(size_t)(n0 + c) * rank + k0 + k]) : 0.f;
         }
         __syncthreads();
+#pragma unroll 4
         for (int k = 0; k < n; ++k) {
-            const float4 wv = *reinterpret_cast<const float4*>(&sw[k][4 * tc]);
+            float av[NT], wv[NC];
 #pragma unroll
-            for (int x = 0; x < NT; ++x) {
-                const float av = sa[k][tr * NT + x];
-                acc[x][0] += av * wv.x; acc[x][1] += av * wv.y; acc[x][2] += av * wv.z; acc[x][3] += av * wv.w;
-            }
+            for (int x = 0; x < NT; ++x) av[x] = sa[k][tr * NT + x];
+#pragma unroll
+            for (int y = 0; y < NC; ++y) wv[y] = sw[k][tc * NC + y];
+#pragma unroll
+            for (int x = 0; x < NT; ++x)
+#pragma unroll
+                for (int y = 0; y < NC; ++y) acc[x][y] += av[x] * wv[y];
         }
         __syncthreads();
     }
@@ -251,8 +259,8 @@ lowrank_decay_kernel(const float* __restrict__ a, const A* __restrict__ w, const
         const int t = t0 + tr * NT + x;
         if (t >= T) continue;
 #pragma unroll
-        for (int y = 0; y < 4; ++y) {
-            const int c = n0 + 4 * tc + y;
+        for (int y = 0; y < NC; ++y) {
+            const int c = n0 + NC * tc + y;
             if (c < N) out[(size_t)t * N + c] = expf(-expf(acc[x][y] + w0[c]));
         }
     }
@@ -264,9 +272,9 @@ extern "C" int rg_lowrank_decay(const float* a, const void* w, int dtype, const 
     if (rank < 1) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const int tt = T > 64 ? 64 : 16;
-    dim3 grid((T + tt - 1) / tt, (N + 63) / 64);
+    dim3 grid((T + tt - 1) / tt, (N + tt - 1) / tt);
     if (grid.y > 65535) return RG_ERR_UNSUPPORTED;
-#define TS_DECAY(TT, A) return rg_launch(lowrank_decay_kernel<TT, A>, grid, dim3(256), 0, s, 1, a, (const A*)w, w0, out, T, N, rank)
+#define TS_DECAY(TT, A) return rg_launch(lowrank_decay_kernel<TT, TT, A>, grid, dim3(256), 0, s, 1, a, (const A*)w, w0, out, T, N, rank)
     if (dtype == RG_DTYPE_BF16) { if (tt == 64) TS_DECAY(64, bf16); TS_DECAY(16, bf16); }
     if (dtype == RG_DTYPE_F32) { if (tt == 64) TS_DECAY(64, float); TS_DECAY(16, float); }
 #undef TS_DECAY

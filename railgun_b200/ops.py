@@ -1156,6 +1156,36 @@ def ssd_prepare(raw: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor):
     return dt, g
 
 
+SSD_CHUNK = 64
+# Steps whose longest portion has at least this many tokens run the recurrence in chunks side by side.
+SSD_CHUNKED_MIN_TOKENS = 128
+
+
+def ssd_chunk_scan(xbc: torch.Tensor, dt: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor, state: torch.Tensor, batch,
+                   H: int, G: int, N: int, dv: int) -> torch.Tensor:
+    """S <- exp(-exp(A_log_h) dt) S + dt B x^T, o = S^T C + D x per head along each request's tokens, as ``state_scan`` with
+    the scalar rule computes it token by token, in chunks of 64 tokens side by side.  ``xbc``: float32 [T, H dv + 2 G N]
+    (x | B | C), ``dt`` [T, H], ``state`` [slots, H, dv, N] (S transposed).  Returns o [T, H, dv] float32."""
+    _check_rows(xbc, "xbc", torch.float32)
+    for t, name in ((dt, "dt"), (A_log, "A_log"), (D, "D"), (state, "state")):
+        _check(t, name, torch.float32)
+    T, R, inner = xbc.shape[0], batch.num_requests, H * dv
+    if xbc.shape[1] != inner + 2 * G * N or tuple(dt.shape) != (T, H) or A_log.numel() != H or D.numel() != H \
+            or tuple(state.shape[1:]) != (H, dv, N) or H % G:
+        raise KernelError("ssd_chunk_scan: sizes do not match")
+    chunks = T // SSD_CHUNK + R
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=xbc.device)
+    sums, decays, dots = new(chunks, H, dv, N), new(chunks, H), new(chunks, G, SSD_CHUNK, SSD_CHUNK)
+    o = new(T, H, dv)
+    _COUNTER.value += 2                              # the launcher runs three kernels
+    at = lambda col: c_void_p(xbc.data_ptr() + 4 * col)
+    _ok(_fn("ssd_chunk", "rg_ssd_chunk_scan")(
+        at(0), at(inner), at(inner + G * N), c_int(xbc.stride(0)), _ptr(dt), _ptr(A_log), _ptr(D), _ptr(state),
+        _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(sums), _ptr(decays), _ptr(dots), _ptr(o),
+        c_int(T), c_int(R), c_int(H), c_int(G), c_int(N), c_int(dv), _stream()), "ssd_chunk_scan")
+    return o
+
+
 def ssd_step(proj: torch.Tensor, x_off: int, dt_off: int, taps: torch.Tensor, bias, conv_state, dt_bias: torch.Tensor,
              A_log: torch.Tensor, D: torch.Tensor, state: torch.Tensor, batch, H: int, G: int, N: int, dv: int):
     """One token per request (rows of ``proj``, float32: x | B | C from column ``x_off``, the raw step sizes at

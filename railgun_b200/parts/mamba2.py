@@ -11,10 +11,10 @@ where group_norm divides each of ``norm_groups`` equal parts by its own root
 mean square.
 
 Steps of single tokens run the convolution, the step sizes and the
-recurrence as one kernel from 32-bit rows; longer portions run the
-convolution, the step sizes and the state scan one after the other, the wide
-part of the product in the model's type and the step sizes' columns in
-32-bit.  Between steps a request keeps, in its state slot and in 32-bit, S of
+recurrence as one kernel from 32-bit rows; portions run the convolution, the
+step sizes and the recurrence one after the other (token by token, or in
+chunks of 64 tokens side by side once a portion is long), the wide part of
+the product in the model's type and the step sizes' columns in 32-bit.  Between steps a request keeps, in its state slot and in 32-bit, S of
 every head (transposed, [dv, N]) and the convolution's last taps - 1 inputs.
 """
 from __future__ import annotations
@@ -98,8 +98,11 @@ class Mamba2(Mixer):
         if writes and conv_state is not None:
             ops.conv_state_update(proj, inner, conv_state, batch)
         dt, g = ops.ssd_prepare(raw_dt, self.dt_bias, self.A_log)
-        o = ops.state_scan(xbc[:, inner + G * N:], xbc[:, inner:inner + G * N], xbc[:, :inner], state, batch, H, N, dv,
-                           g=g, beta=dt, rule="scalar", skip=self.D)
+        if batch.max_query_len >= ops.SSD_CHUNKED_MIN_TOKENS:
+            o = ops.ssd_chunk_scan(xbc, dt, self.A_log, self.D, state, batch, H, G, N, dv)
+        else:
+            o = ops.state_scan(xbc[:, inner + G * N:], xbc[:, inner:inner + G * N], xbc[:, :inner], state, batch, H, N, dv,
+                               g=g, beta=dt, rule="scalar", skip=self.D)
         y = ops.gate_group_norm(o, z, self.norm, self.eps, self.norm_groups, self.env.dtype)
         return ops.linear(y, self.w_o)
 

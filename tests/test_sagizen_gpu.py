@@ -168,34 +168,44 @@ def test_scan_with_a_decay_per_channel(H, d, dv):
 
 @pytest.mark.parametrize("H,G,N,dv", [(1, 1, 9, 6), (6, 3, 16, 8), (4, 2, 24, 16), (5, 5, 10, 6), (8, 2, 128, 64), (2, 1, 200, 40),
                                       (3, 1, 256, 256)])
-def test_scan_with_step_sizes(H, G, N, dv):
+@pytest.mark.parametrize("form", ["tokens", "chunks"])
+def test_scan_with_step_sizes(form, H, G, N, dv):
     """The state-space duality form: a decay and a step size per token and head, B and C shared by a group's heads,
-    D on the token's own x."""
+    D on the token's own x; token by token, and in chunks side by side (whole ones, ends of one token and more, requests
+    of less than one, heads that forget within a few tokens)."""
     from railgun_b200 import ops
     rng = np.random.default_rng(H + N)
-    lengths, starts, slots = [40, 75, 1], [0, 33, 9], [2, 0, 3]
+    lengths, starts, slots = ([40, 75, 1], [0, 33, 9], [2, 0, 3]) if form == "tokens" else (
+        [64, 129, 1, 200, 63], [5, 0, 9, 33, 0], [2, 0, 3, 4, -1])
     T = sum(lengths)
     xbc = torch.tensor(rng.normal(size=(T, H * dv + 2 * G * N)) * 0.5, dtype=torch.float32)
     raw = torch.tensor(rng.normal(size=(T, H)) * 2.0, dtype=torch.float32)
     bias, A, D = rng.uniform(-5, 1, size=H), rng.uniform(-3, 1, size=H), rng.normal(size=H)
+    A[0] = 2.5
     dt, g = ops.ssd_prepare(dev(raw), dev(bias, torch.float32), dev(A, torch.float32))
     dt_ref = P.softplus(raw.double().numpy() + bias)
     assert rel(dt, dt_ref) < 1e-6 and np.abs(g.double().cpu().numpy() - np.exp(-np.exp(A) * dt_ref)).max() < 1e-6
-    state0 = rng.normal(size=(4, H, dv, N)) * 0.3
+    state0 = rng.normal(size=(5, H, dv, N)) * 0.3
     state = dev(state0, torch.float32)
     x = dev(xbc)
     inner = H * dv
-    o = ops.state_scan(x[:, inner + G * N:], x[:, inner:inner + G * N], x[:, :inner], state, step_batch(lengths, starts, slots),
-                       H, N, dv, g=g, beta=dt, rule="scalar", skip=dev(D, torch.float32))
+    batch = step_batch(lengths, starts, slots)
+    if form == "tokens":
+        o = ops.state_scan(x[:, inner + G * N:], x[:, inner:inner + G * N], x[:, :inner], state, batch, H, N, dv, g=g, beta=dt,
+                           rule="scalar", skip=dev(D, torch.float32))
+    else:
+        o = ops.ssd_chunk_scan(x, dt, dev(A, torch.float32), dev(D, torch.float32), state, batch, H, G, N, dv)
     xr = xbc.double().numpy()
     X, B, Cc = xr[:, :inner].reshape(T, H, dv), xr[:, inner:inner + G * N].reshape(T, G, N), xr[:, inner + G * N:].reshape(T, G, N)
-    refs = []
     for sl, start, slot in zip(split(lengths), starts, slots):
-        S0 = None if start == 0 else np.transpose(state0[slot], (0, 2, 1))
+        S0 = None if start == 0 or slot < 0 else np.transpose(state0[slot], (0, 2, 1))
         ro, S = P.ssd_scan(X[sl], dt_ref[sl], A, B[sl], Cc[sl], S0)
-        refs.append(ro + D[None, :, None] * X[sl])
-        assert rel(state[slot], np.transpose(S, (0, 2, 1))) < 3e-5
-    assert rel(o, np.concatenate(refs)) < 3e-5 and rel(state[1], state0[1]) < 1e-7
+        ref = ro + D[None, :, None] * X[sl]
+        for h in range(H):                                                     # every head to its own size
+            assert rel(o[sl][:, h], ref[:, h]) < 3e-5
+            if slot >= 0:
+                assert rel(state[slot, h], S[h].T) < 3e-5
+    assert rel(state[1], state0[1]) < 1e-7
 
 
 def test_scans_of_the_other_designs_are_unchanged():
