@@ -1566,7 +1566,12 @@ def run_kernels(args):
                                 for (r, k, v), w, st in zip(rk, ws_, sts)])
             us2 = timed(lambda: [ops.state_scan(r, k, v, st, batch, Hr, dr, dr, decay=decay) for (r, k, v), st in zip(rk, sts)])
             by, by2 = T * n * 5 * 4 + R_ * n * dr * 8, T * n * 4 * 4 + R_ * n * dr * 8
-            out(f"scan with a decay per channel H{Hr} d{dr} T{T} ({R_} requests)", us, frac=gbs(by, us), retention_us=round(us2, 2),
+            more = {}
+            if R_ == 1:
+                usc = timed(lambda: [ops.channel_chunk_scan(r, k, v, w, bonus, st, batch, Hr, dr, dr)
+                                     for (r, k, v), w, st in zip(rk, ws_, sts)])
+                more = dict(chunked_us=round(usc, 2), chunked_frac=gbs(by, usc))
+            out(f"scan with a decay per channel H{Hr} d{dr} T{T} ({R_} requests)", us, frac=gbs(by, us), **more, retention_us=round(us2, 2),
                 retention_frac=gbs(by2, us2))
             os_ = [torch.randn(T, Hr, dr, device=dev) for _ in range(L)]
             nwr = torch.ones(n, device=dev)
@@ -1675,7 +1680,9 @@ def run_kernels(args):
                 else:
                     info[f + "_frac_flops"] = round(Hh * 4 * dd * seen[f] / us / 1e6 / pk["bf16_tflops"], 3)
             out(f"attention window {win} and blocks of {pool}, H{Hh} G{G} d{dd}, {B} requests x {T // B} tokens", res["pool"], **info)
-            slots = torch.zeros(T, dtype=torch.int32, device=dev) if B > 1 else torch.arange(T, dtype=torch.int32, device=dev)
+            if B > 1:
+                continue                                  # single tokens pool inside the per-token kernel
+            slots = torch.arange(T, dtype=torch.int32, device=dev)
             batch = SimpleNamespace(req_of_token=req, positions=pos)
             us = timed(lambda: [ops.pool_blocks(kv, bt, batch, slots, pk_, pool) for kv, pk_ in zip(kvs, pks)])
             ends = int(((pos + 1) % pool == 0).sum())

@@ -14,26 +14,7 @@
 // their differences are small beside them where a head forgets fast.
 //
 // The step's tokens are packed request by request (cu_seqlens); a request's chunks start at its first token of the step.
-#include "common.cuh"
-
-#define CH 64                 // tokens per chunk
-#define TILE 64               // rows and columns of a block's output (columns: 64 or 128)
-#define PITCH (TILE + 4)
-#define NTH 256
-
-// Chunk number c of the step: its request, first token and number of tokens; false beyond the last one.
-__device__ __forceinline__ bool find_chunk(const int* __restrict__ cu, int R, int c, int& r, int& lo, int& n) {
-    for (r = 0; r < R; ++r) {
-        const int len = cu[r + 1] - cu[r], k = (len + CH - 1) / CH;
-        if (c < k) {
-            lo = cu[r] + c * CH;
-            n = min(CH, len - c * CH);
-            return true;
-        }
-        c -= k;
-    }
-    return false;
-}
+#include "chunk_scan.cuh"
 
 // c_i of the chunk's tokens for head h (64-bit), by the block's first warp; dt of the tokens into sdt.
 __device__ __forceinline__ void chunk_sums(const float* __restrict__ dt, float A_log, int lo, int n, int H, int h,
@@ -53,39 +34,6 @@ __device__ __forceinline__ void chunk_sums(const float* __restrict__ dt, float A
         cum[i1] = s;
         sdt[i0] = d0;
         sdt[i1] = d1;
-    }
-}
-
-// dst[k][i] = src row i, number k0 + k (rows ld apart, n rows of N numbers; zeros elsewhere), for 64 x 64, times scale[i].
-// A warp reads 4 rows x 8 neighbouring numbers at a time and writes 32 different banks.
-__device__ __forceinline__ void load_transposed(float (*__restrict__ dst)[PITCH], const float* __restrict__ src, size_t ld,
-                                                int n, int N, int k0, const float* __restrict__ scale) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int kl = lane & 7, il = lane >> 3;
-#pragma unroll 4
-    for (int p = warp; p < (TILE / 8) * (TILE / 4); p += NTH / 32) {
-        const int k = (p & 7) * 8 + kl, i = (p >> 3) * 4 + il;
-        float v = i < n && k0 + k < N ? src[(size_t)i * ld + k0 + k] : 0.f;
-        if (scale) v *= scale[i];
-        dst[k][i] = v;
-    }
-}
-
-// acc[4][4 W] += A[k][4 rows]^T B[k][4 W columns] over kn values of k.  Thread (ty, tx): rows 4 ty .., columns 4 tx .. (+ 64)
-template <int W>
-__device__ __forceinline__ void multiply(float (&acc)[4][4 * W], const float (*__restrict__ A)[PITCH],
-                                         const float (*__restrict__ B)[TILE * W + 4], int kn, int ty, int tx) {
-#pragma unroll 4
-    for (int k = 0; k < kn; ++k) {
-        const float4 a = *reinterpret_cast<const float4*>(&A[k][4 * ty]);
-#pragma unroll
-        for (int w = 0; w < W; ++w) {
-            const float4 b = *reinterpret_cast<const float4*>(&B[k][TILE * w + 4 * tx]);
-            acc[0][4 * w] += a.x * b.x; acc[0][4 * w + 1] += a.x * b.y; acc[0][4 * w + 2] += a.x * b.z; acc[0][4 * w + 3] += a.x * b.w;
-            acc[1][4 * w] += a.y * b.x; acc[1][4 * w + 1] += a.y * b.y; acc[1][4 * w + 2] += a.y * b.z; acc[1][4 * w + 3] += a.y * b.w;
-            acc[2][4 * w] += a.z * b.x; acc[2][4 * w + 1] += a.z * b.y; acc[2][4 * w + 2] += a.z * b.z; acc[2][4 * w + 3] += a.z * b.w;
-            acc[3][4 * w] += a.w * b.x; acc[3][4 * w + 1] += a.w * b.y; acc[3][4 * w + 2] += a.w * b.z; acc[3][4 * w + 3] += a.w * b.w;
-        }
     }
 }
 
@@ -169,63 +117,6 @@ chunk_states_kernel(const float* __restrict__ x, const float* __restrict__ B, co
         }
     }
     if (blockIdx.z == 0 && threadIdx.x == 0) decays[(size_t)blockIdx.x * H + h] = expf((float)end);
-}
-
-// sums [chunks, H, dv N]: each chunk's sum becomes the state before the chunk.  V numbers per thread.
-template <int V>
-__global__ void chunk_pass_kernel(float* __restrict__ sums, const float* __restrict__ decays, float* __restrict__ state,
-                                  const int* __restrict__ cu, const int* __restrict__ start_pos,
-                                  const int* __restrict__ slots, int H, int M) {
-    pdl_wait();
-    pdl_trigger();
-    const int r = blockIdx.y;
-    const long long e = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
-    if (e >= (long long)H * M) return;
-    const int h = (int)(e / M);
-    int c0 = 0;
-    for (int q = 0; q < r; ++q) c0 += (cu[q + 1] - cu[q] + CH - 1) / CH;
-    const int nc = (cu[r + 1] - cu[r] + CH - 1) / CH;
-    const int slot = slots[r];
-    float S[V];
-#pragma unroll
-    for (int i = 0; i < V; ++i) S[i] = 0.f;
-    float* st = state + (size_t)(slot >= 0 ? slot : 0) * H * M + e;
-    if (slot >= 0 && start_pos[r] > 0) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) S[i] = st[i];
-    }
-    float* p = sums + (size_t)c0 * H * M + e;
-    const float* dec = decays + (size_t)c0 * H + h;
-    const size_t step = (size_t)H * M;
-    constexpr int U = 4;                              // chunks in flight
-    for (int c = 0; c < nc; c += U) {
-        float u[U][V], d[U];
-#pragma unroll
-        for (int k = 0; k < U; ++k) {
-            if (c + k < nc) {
-                d[k] = dec[(size_t)(c + k) * H];
-                if (V == 4) {
-                    const float4 q = *reinterpret_cast<const float4*>(p + (c + k) * step);
-                    u[k][0] = q.x; u[k][1 % V] = q.y; u[k][2 % V] = q.z; u[k][3 % V] = q.w;
-                } else {
-                    u[k][0] = p[(c + k) * step];
-                }
-            }
-        }
-#pragma unroll
-        for (int k = 0; k < U; ++k) {
-            if (c + k < nc) {
-                if (V == 4) *reinterpret_cast<float4*>(p + (c + k) * step) = make_float4(S[0], S[1 % V], S[2 % V], S[3 % V]);
-                else p[(c + k) * step] = S[0];
-#pragma unroll
-                for (int i = 0; i < V; ++i) S[i] = S[i] * d[k] + u[k][i];
-            }
-        }
-    }
-    if (slot >= 0) {
-#pragma unroll
-        for (int i = 0; i < V; ++i) st[i] = S[i];
-    }
 }
 
 // before [chunks, H, dv, N]: the state before every chunk.  o [T, H, dv].  grid: chunks, H, tiles of 64 columns.
@@ -312,8 +203,8 @@ extern "C" int rg_ssd_chunk_scan(const float* x, const float* B, const float* C,
     const bool vec = M % 4 == 0 && ((uintptr_t)state & 15) == 0;
     const long long work = vec ? (long long)H * M / 4 : (long long)H * M;
     dim3 g2((unsigned)((work + 255) / 256), R);
-    e = vec ? rg_launch(chunk_pass_kernel<4>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M)
-            : rg_launch(chunk_pass_kernel<1>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M);
+    e = vec ? rg_launch(chunk_pass_kernel<4, false>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M, N)
+            : rg_launch(chunk_pass_kernel<1, false>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M, N);
     if (e) return e;
     dim3 g3(chunks, H, jt);
     return rg_launch(chunk_outputs_kernel, g3, dim3(NTH), 0, s, 1, x, C, ld, dt, A_log, D, cu_seqlens, R, (const float*)sums,

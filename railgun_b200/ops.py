@@ -1156,9 +1156,9 @@ def ssd_prepare(raw: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor):
     return dt, g
 
 
-SSD_CHUNK = 64
-# Steps whose longest portion has at least this many tokens run the recurrence in chunks side by side.
-SSD_CHUNKED_MIN_TOKENS = 128
+SCAN_CHUNK = 64
+# Steps whose longest portion has at least this many tokens run these recurrences in chunks side by side.
+SCAN_CHUNKED_MIN_TOKENS = 128
 
 
 def ssd_chunk_scan(xbc: torch.Tensor, dt: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor, state: torch.Tensor, batch,
@@ -1173,9 +1173,9 @@ def ssd_chunk_scan(xbc: torch.Tensor, dt: torch.Tensor, A_log: torch.Tensor, D: 
     if xbc.shape[1] != inner + 2 * G * N or tuple(dt.shape) != (T, H) or A_log.numel() != H or D.numel() != H \
             or tuple(state.shape[1:]) != (H, dv, N) or H % G:
         raise KernelError("ssd_chunk_scan: sizes do not match")
-    chunks = T // SSD_CHUNK + R
+    chunks = T // SCAN_CHUNK + R
     new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=xbc.device)
-    sums, decays, dots = new(chunks, H, dv, N), new(chunks, H), new(chunks, G, SSD_CHUNK, SSD_CHUNK)
+    sums, decays, dots = new(chunks, H, dv, N), new(chunks, H), new(chunks, G, SCAN_CHUNK, SCAN_CHUNK)
     o = new(T, H, dv)
     _COUNTER.value += 2                              # the launcher runs three kernels
     at = lambda col: c_void_p(xbc.data_ptr() + 4 * col)
@@ -1183,6 +1183,34 @@ def ssd_chunk_scan(xbc: torch.Tensor, dt: torch.Tensor, A_log: torch.Tensor, D: 
         at(0), at(inner), at(inner + G * N), c_int(xbc.stride(0)), _ptr(dt), _ptr(A_log), _ptr(D), _ptr(state),
         _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(sums), _ptr(decays), _ptr(dots), _ptr(o),
         c_int(T), c_int(R), c_int(H), c_int(G), c_int(N), c_int(dv), _stream()), "ssd_chunk_scan")
+    return o
+
+
+def channel_chunk_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, bonus: torch.Tensor,
+                       state: torch.Tensor, batch, H: int, d: int, dv: int) -> torch.Tensor:
+    """o = (S + diag(bonus_h) k v^T)^T r, then S <- diag(w) S + k v^T per head along each request's tokens, as ``state_scan``
+    with the channel rule computes it token by token, in chunks of 64 tokens side by side.  ``r``, ``k``, ``w``: float32
+    [T, H d] views, ``v`` [T, H dv], ``bonus`` [H, d], ``state`` [slots, H, dv, d] (S transposed).  Returns o [T, H, dv]
+    float32."""
+    for t, name in ((r, "r"), (k, "k"), (v, "v"), (w, "w")):
+        _check_rows(t, name, torch.float32)
+    _check(bonus, "bonus", torch.float32)
+    _check(state, "state", torch.float32)
+    T, R = r.shape[0], batch.num_requests
+    if any(t.shape != (T, H * d) for t in (r, k, w)) or v.shape != (T, H * dv) or bonus.numel() != H * d \
+            or tuple(state.shape[1:]) != (H, dv, d):
+        raise KernelError("channel_chunk_scan: sizes do not match")
+    chunks = T // SCAN_CHUNK + R
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=r.device)
+    qd, kd, sums, decays, dots = (new(T, H * d), new(T, H * d), new(chunks, H, dv, d), new(chunks, H * d),
+                                  new(chunks, H, SCAN_CHUNK, SCAN_CHUNK))
+    o = new(T, H, dv)
+    _COUNTER.value += 3                              # the launcher runs four kernels
+    _ok(_fn("channel_chunk", "rg_channel_chunk_scan")(
+        _ptr(r), c_int(r.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(v.stride(0)), _ptr(w), c_int(w.stride(0)),
+        _ptr(bonus), _ptr(state), _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(qd), _ptr(kd),
+        _ptr(sums), _ptr(decays), _ptr(dots), _ptr(o), c_int(T), c_int(R), c_int(H), c_int(d), c_int(dv), _stream()),
+        "channel_chunk_scan")
     return o
 
 

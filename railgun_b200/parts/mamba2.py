@@ -98,7 +98,7 @@ class Mamba2(Mixer):
         if writes and conv_state is not None:
             ops.conv_state_update(proj, inner, conv_state, batch)
         dt, g = ops.ssd_prepare(raw_dt, self.dt_bias, self.A_log)
-        if batch.max_query_len >= ops.SSD_CHUNKED_MIN_TOKENS:
+        if batch.max_query_len >= ops.SCAN_CHUNKED_MIN_TOKENS:
             o = ops.ssd_chunk_scan(xbc, dt, self.A_log, self.D, state, batch, H, G, N, dv)
         else:
             o = ops.state_scan(xbc[:, inner + G * N:], xbc[:, inner:inner + G * N], xbc[:, :inner], state, batch, H, N, dv,

@@ -12,6 +12,8 @@ above, each of r, k, v, g and w reads a mix h + (h' - h) mu_s of its own:
   o_t = (S_(t-1) + diag(u) k_t v_t^T)^T r_t;   S_t = diag(w_t) S_(t-1) + k_t v_t^T
   out = W_o (unit_rms(o_t) per head * norm * gate)
 The four wide products are one batched library product into 32-bit rows.  The
+recurrence runs token by token, or in chunks of 64 tokens side by side once a
+portion is long.  The
 decay is 32-bit from its mix on: in bfloat16 mode the mix enters its product
 as two bfloat16 numbers (hi + lo to 2^-17) against the matrix stacked twice,
 accumulated in 32-bit.
@@ -143,7 +145,10 @@ class RwkvTimeMixing(Mixer):
         else:
             r, k, v, g = torch.bmm(mixes, wide, out_dtype=torch.float32)
         w = ops.lowrank_decay(ops.linear(last, self.w1, out_dtype=torch.float32), self.w2, self.w0)
-        o = ops.state_scan(r, k, v, cache.parts[0].state, batch, H, d, d, rule="channel", w=w, bonus=self.u)
+        if batch.max_query_len >= ops.SCAN_CHUNKED_MIN_TOKENS:
+            o = ops.channel_chunk_scan(r, k, v, w, self.u, cache.parts[0].state, batch, H, d, d)
+        else:
+            o = ops.state_scan(r, k, v, cache.parts[0].state, batch, H, d, d, rule="channel", w=w, bonus=self.u)
         return ops.head_norm_gate(o, g, self.norm, self.eps, self.env.dtype, out=out, out_scale=out_scale)
 
     def forward(self, x, batch, cache, writes=True):

@@ -138,32 +138,43 @@ def test_lowrank_decay_alone(T, N, rank, dtype):
 # ---- the matrix states ---------------------------------------------------------------------------------------
 
 @pytest.mark.parametrize("H,d,dv", [(1, 10, 10), (3, 12, 12), (2, 7, 7), (4, 64, 64), (2, 128, 128), (1, 200, 40), (2, 256, 256)])
-def test_scan_with_a_decay_per_channel(H, d, dv):
+@pytest.mark.parametrize("form", ["tokens", "chunks"])
+def test_scan_with_a_decay_per_channel(form, H, d, dv):
     """S carried in the slot from an earlier step beside a new request in a dirty slot and a single token; the current
-    token counts through the bonus only and is decayed by nobody; a far key made loud is still heard."""
+    token counts through the bonus only and is decayed by nobody; a far key made loud is still heard; channels that
+    forget at once (a decay of exactly 0) and never (1).  Token by token, and in chunks side by side (whole ones, ends of
+    one token and more, requests of less than one)."""
     from railgun_b200 import ops
     rng = np.random.default_rng(H + d)
-    lengths, starts, slots = [40, 75, 1], [0, 33, 9], [2, 0, 3]
-    T = sum(lengths)
+    lengths, starts, slots = ([40, 75, 1], [0, 33, 9], [2, 0, 3]) if form == "tokens" else (
+        [64, 129, 1, 200, 63], [0, 33, 9, 5, 0], [2, 0, 3, 4, -1])
+    T, at = sum(lengths), lengths[0]
     r, k, v = (torch.tensor(rng.normal(size=(T, H * n)) * 0.5, dtype=torch.float32) for n in (d, d, dv))
-    w = torch.tensor(np.exp(-np.exp(rng.uniform(-6.0, 0.0, size=(T, H * d)))), dtype=torch.float32)
-    w[40:, :d] = torch.clamp(w[40:, :d], min=0.99)
-    k[45, :d], r[114, :d] = 3.0, 3.0                                           # a loud key, and the query that asks for it
+    w = np.exp(-np.exp(rng.uniform(-6.0, 0.0, size=(T, H * d))))
+    w[:, 1], w[:, 2], w[7::9, 3] = 0.0, 1.0, 0.0
+    w[at:, 4:d] = np.maximum(w[at:, 4:d], 0.99)
+    w = torch.tensor(w, dtype=torch.float32)
+    far, ask = at + 5, at + lengths[1] - 1
+    k[far, :d], r[ask, :d] = 3.0, 3.0                                          # a loud key, and the query that asks for it
     u = rng.normal(size=(H, d))
-    state0 = rng.normal(size=(4, H, dv, d)) * 0.3
+    state0 = rng.normal(size=(5, H, dv, d)) * 0.3
     state = dev(state0, torch.float32)
-    o = ops.state_scan(dev(r), dev(k), dev(v), state, step_batch(lengths, starts, slots), H, d, dv, rule="channel",
-                       w=dev(w), bonus=dev(u, torch.float32))
+    batch = step_batch(lengths, starts, slots)
+    if form == "tokens":
+        o = ops.state_scan(dev(r), dev(k), dev(v), state, batch, H, d, dv, rule="channel", w=dev(w), bonus=dev(u, torch.float32))
+    else:
+        o = ops.channel_chunk_scan(dev(r), dev(k), dev(v), dev(w), dev(u, torch.float32), state, batch, H, d, dv)
     f = lambda t, n: t.double().numpy().reshape(T, H, n)
     refs = []
     for sl, start, slot in zip(split(lengths), starts, slots):
-        S0 = None if start == 0 else np.transpose(state0[slot], (0, 2, 1))
+        S0 = None if start == 0 or slot < 0 else np.transpose(state0[slot], (0, 2, 1))
         ro, S = P.rwkv_scan(f(r, d)[sl], f(k, d)[sl], f(v, dv)[sl], f(w, d)[sl], u, S0)
         refs.append(ro)
-        assert rel(state[slot], np.transpose(S, (0, 2, 1))) < 3e-5
+        if slot >= 0:
+            assert rel(state[slot], np.transpose(S, (0, 2, 1))) < 3e-5
     ref = np.concatenate(refs)
     assert rel(o, ref) < 3e-5 and rel(state[1], state0[1]) < 1e-7
-    assert np.abs(ref[114, 0]).max() > 3 * np.median(np.abs(ref[:, 0]))
+    assert np.abs(ref[ask, 0]).max() > 3 * np.median(np.abs(ref[:, 0]))
 
 
 @pytest.mark.parametrize("H,G,N,dv", [(1, 1, 9, 6), (6, 3, 16, 8), (4, 2, 24, 16), (5, 5, 10, 6), (8, 2, 128, 64), (2, 1, 200, 40),
