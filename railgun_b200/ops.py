@@ -1205,7 +1205,7 @@ def channel_chunk_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: tor
     qd, kd, sums, decays, dots = (new(T, H * d), new(T, H * d), new(chunks, H, dv, d), new(chunks, H * d),
                                   new(chunks, H, SCAN_CHUNK, SCAN_CHUNK))
     o = new(T, H, dv)
-    _COUNTER.value += 3                              # the launcher runs four kernels
+    _COUNTER.value += 4                              # the launcher runs five kernels
     _ok(_fn("channel_chunk", "rg_channel_chunk_scan")(
         _ptr(r), c_int(r.stride(0)), _ptr(k), c_int(k.stride(0)), _ptr(v), c_int(v.stride(0)), _ptr(w), c_int(w.stride(0)),
         _ptr(bonus), _ptr(state), _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(qd), _ptr(kd),
