@@ -14,7 +14,7 @@ pytestmark = pytest.mark.gpu
 CASE_W = dict(
     architecture="Sagizen", width=1024, vocab=512, norm=dict(eps=1e-6),
     layers=[C.layer(C.mamba(16, 64, 128, 2, 4, 2), 2048),
-            C.layer(C.parallel(C.left(4, 2, 128, 128, 100, 8, dims=64, factor=4.0), 4, 128, 0.6, 0.7), 1024),
+            C.layer(C.parallel(C.left(4, 2, 128, 128, 100, 6, dims=96, factor=2.5), 4, 128, 0.6, 0.7), 1024),
             C.layer(C.mamba(16, 64, 128, 1, 4, 1), None)])
 LENGTHS = [330, 40, 197, 3]
 _state: dict = {}
