@@ -50,6 +50,7 @@ class PagedKVNeed:
     dtype: str | None = None   # None: the model's
     page_shape: tuple | None = None
     tokens_per_entry: int = 1
+    chunk: int = 0             # not 0: a query sees only its own chunk of this many positions, counted from 0 (no window)
 
     def shape_of_page(self, page_size: int) -> tuple:
         if self.page_shape is None:
@@ -84,6 +85,7 @@ def _lib():
         lib.rg_cache_destroy.argtypes = [c_void_p]
         lib.rg_cache_destroy.restype = None
         lib.rg_cache_set_keep_first.argtypes = [c_void_p, c_int, c_int]
+        lib.rg_cache_set_chunk.argtypes = [c_void_p, c_int, c_int]
         for name in ("add_request", "release", "has", "num_computed", "slot"):
             getattr(lib, f"rg_cache_{name}").argtypes = [c_void_p, c_longlong]
         for name in ("reserve", "commit"):
@@ -143,7 +145,8 @@ class PageAllocator:
     """The C++ cache manager: page groups, block tables, state slots and the slots' request records.  No
     device memory."""
 
-    def __init__(self, page_sizes, num_pages, windows, max_requests: int, keep_first=None):
+    def __init__(self, page_sizes, num_pages, windows, max_requests: int, keep_first=None,
+                 chunks=None):
         self._lib = _lib()
         n = len(page_sizes)
         if not (len(num_pages) == len(windows) == n):
@@ -162,6 +165,11 @@ class PageAllocator:
         for g, keep in enumerate(self.keep_first):
             if keep and self._lib.rg_cache_set_keep_first(self._h, g, keep):
                 raise CacheError(f"group {g}: cannot keep the first {keep} positions")
+        # groups whose queries see only their own chunk of positions
+        self.chunks = [int(x) for x in (chunks or [0] * n)]
+        for g, chunk in enumerate(self.chunks):
+            if chunk and self._lib.rg_cache_set_chunk(self._h, g, chunk):
+                raise CacheError(f"group {g}: cannot have chunks of {chunk} positions")
         self._buf = np.empty(64, dtype=np.int32)
         self._any_sampled = c_int(0)
         if self._lib.rg_cache_record_bytes() != REQUEST_RECORD.itemsize:
@@ -379,7 +387,8 @@ class CacheManager:
             self.groups.append(GroupInfo(need, ps, (pool + ps - 1) // ps + spare, cids))
         self.alloc = PageAllocator([g.page_size for g in self.groups], [g.num_pages for g in self.groups],
                                    [g.need.window for g in self.groups], max_requests,
-                                   keep_first=[g.need.keep_first for g in self.groups])
+                                   keep_first=[g.need.keep_first for g in self.groups],
+                                   chunks=[g.need.chunk for g in self.groups])
         self.max_requests = int(max_requests)
         self.dtype = dtype
         self.device = device

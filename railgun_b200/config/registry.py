@@ -82,3 +82,5 @@ def _ensure_builtin():
         from ..models import kasarax  # noqa: F401
     if "Sagizen" not in _ARCHITECTURES:
         from ..models import sagizen  # noqa: F401
+    if "Bunudra" not in _ARCHITECTURES:
+        from ..models import bunudra  # noqa: F401

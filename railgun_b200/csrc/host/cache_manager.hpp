@@ -6,7 +6,8 @@
 // pages that every future query has passed are given back at commit time and
 // their block-table entries become -1 (except the pages that hold any of the
 // group's first keep_first positions, which a window that keeps the first
-// tokens goes on reading).  Beside the pages, every live request
+// tokens goes on reading).  A group whose queries see only their own chunk of
+// positions gives back the pages of every chunk that is complete.  Beside the pages, every live request
 // holds one state slot: an index into fixed-size per-request buffers, and the
 // place of its RequestRecord, the one fixed-size description of a live request
 // (position, lengths, sampling parameters, seed) that decode steps are packed
@@ -41,6 +42,7 @@ struct CacheGroup {
     int page_size = 16;
     int num_pages = 0;
     int window = 0;                 // 0: every key is kept
+    int chunk = 0;                  // 0: none; else a query sees its own chunk of that many positions only
     int keep_first = 0;             // with a window: the first positions that stay visible, so their pages stay
     std::deque<int> free_list;
     std::vector<int> refcount;
@@ -91,6 +93,13 @@ public:
     int set_keep_first(int g, int keep) {
         if (g < 0 || g >= (int)groups_.size() || keep < 0 || !reqs_.empty()) return CACHE_BAD_ARGUMENT;
         groups_[g].keep_first = keep;
+        return CACHE_OK;
+    }
+    // A group whose queries see only the chunk of `chunk` positions (counted from position 0) that they lie in.
+    int set_chunk(int g, int chunk) {
+        if (g < 0 || g >= (int)groups_.size() || chunk < 0 || !reqs_.empty() || (chunk && groups_[g].window))
+            return CACHE_BAD_ARGUMENT;
+        groups_[g].chunk = chunk;
         return CACHE_OK;
     }
     int free_pages(int g) const { return (int)groups_[g].free_list.size(); }
@@ -179,8 +188,9 @@ public:
         records_[r.slot].num_computed = new_len;
         for (size_t g = 0; g < groups_.size(); ++g) {
             CacheGroup& G = groups_[g];
-            if (G.window <= 0) continue;
-            const int first_needed = new_len - G.window + 1;     // lowest key any later query reads
+            if (G.window <= 0 && G.chunk <= 0) continue;
+            // lowest key any later query reads
+            const int first_needed = G.chunk > 0 ? new_len / G.chunk * G.chunk : new_len - G.window + 1;
             for (size_t i = 0; i < r.tables[g].size(); ++i) {
                 if ((int)(i + 1) * G.page_size > first_needed) break;
                 if ((int)i * G.page_size < G.keep_first) continue;

@@ -279,7 +279,7 @@ private:
     bool fits_alone(int len) const {
         for (int g = 0; g < cache_->num_groups(); ++g) {
             const CacheGroup& G = cache_->group(g);
-            if (G.window > 0) continue;      // a windowed group gives pages back as it goes
+            if (G.window > 0 || G.chunk > 0) continue;      // a windowed group gives pages back as it goes
             if ((len + G.page_size - 1) / G.page_size > G.num_pages) return false;
         }
         return true;

@@ -119,22 +119,13 @@ extern "C" int rg_softcap(float* z, float cap, long long n, void* stream) {
                      (cudaStream_t)stream, 1, z, cap, (size_t)n);
 }
 
-// Elementwise activations of a dense feed-forward, computed in 32-bit: 0 relu(z)^2, 1 relu, 2 gelu (tanh form), 3 silu.
-__device__ __forceinline__ float act_apply(float z, int kind) {
-    switch (kind) {
-        case 0: { const float r = fmaxf(z, 0.f); return r * r; }
-        case 1: return fmaxf(z, 0.f);
-        case 2: return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-        default: return z / (1.f + expf(-z));
-    }
-}
-
+// Elementwise activations of a dense feed-forward, computed in 32-bit (plain_act of common.cuh).
 template <typename A>
 __global__ void activation_kernel(const A* __restrict__ in, A* __restrict__ out, int kind, size_t n) {
     pdl_wait();
     pdl_trigger();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) out[i] = from_f32<A>(act_apply(to_f32(in[i]), kind));
+    if (i < n) out[i] = from_f32<A>(plain_act(to_f32(in[i]), kind));
 }
 
 // Eight bfloat16 numbers per thread with 16-byte loads and stores.
@@ -150,14 +141,14 @@ __global__ void activation_vec8_kernel(const bf16* __restrict__ in, bf16* __rest
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const float2 f = __bfloat1622float2(v2[i]);
-        o2[i] = __floats2bfloat162_rn(act_apply(f.x, kind), act_apply(f.y, kind));
+        o2[i] = __floats2bfloat162_rn(plain_act(f.x, kind), plain_act(f.y, kind));
     }
     *reinterpret_cast<uint4*>(out + g * 8) = o;
 }
 
 extern "C" int rg_activation(const void* in, void* out, int dtype, int kind, long long n, void* stream) {
     if (n <= 0) return 0;
-    if (kind < 0 || kind > 3) return RG_ERR_UNSUPPORTED;
+    if (kind < 0 || kind > 4) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = 256;
     if (dtype == RG_DTYPE_BF16 && n % 8 == 0 && ((uintptr_t)in % 16) == 0 && ((uintptr_t)out % 16) == 0) {
@@ -227,5 +218,57 @@ extern "C" int rg_gated_activation(const void* gu, void* out, int dtype, int T, 
     if (dtype == RG_DTYPE_F32)
         return rg_launch(gated_activation_kernel<float>, dim3(blocks), dim3(256), 0, s, 1, (const float*)gu, (float*)out, I,
                          kind, limit, total);
+    return RG_ERR_UNSUPPORTED;
+}
+
+// x <- x * sigmoid(gate) in place: of every group of `stride` numbers of a row of x the first n have a partner among the
+// gate's n numbers of that group (gate rows gate_ld apart).  V numbers per thread (n, stride and both rows' starts
+// divisible by it).
+template <typename A, int V>
+__global__ void sigmoid_gate_kernel(A* __restrict__ x, const A* __restrict__ gate, int gate_ld, int groups, int n, int stride,
+                                    size_t total) {
+    pdl_wait();
+    pdl_trigger();
+    const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (idx >= total) return;
+    const int per_row = groups * (n / V);
+    const size_t t = idx / per_row;
+    const int k = (int)(idx - t * per_row) * V, g = k / n;
+    A* px = x + t * (size_t)groups * stride + (size_t)g * stride + (k - g * n);
+    const A* pg = gate + t * (size_t)gate_ld + k;
+    if (V == 8) {
+        uint4 xv = *reinterpret_cast<const uint4*>(px);
+        const uint4 gv = *reinterpret_cast<const uint4*>(pg);
+        __nv_bfloat162* x2 = reinterpret_cast<__nv_bfloat162*>(&xv);
+        const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const float2 a = __bfloat1622float2(x2[i]), b = __bfloat1622float2(g2[i]);
+            x2[i] = __floats2bfloat162_rn(a.x / (1.f + expf(-b.x)), a.y / (1.f + expf(-b.y)));
+        }
+        *reinterpret_cast<uint4*>(px) = xv;
+    } else {
+        px[0] = from_f32<A>(to_f32(px[0]) / (1.f + expf(-to_f32(pg[0]))));
+    }
+}
+
+extern "C" int rg_sigmoid_gate(void* x, const void* gate, int dtype, int gate_ld, int T, int groups, int n, int stride,
+                               void* stream) {
+    if (T <= 0 || groups <= 0 || n <= 0) return 0;
+    if (stride < n) return RG_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    const size_t total = (size_t)T * groups * n;
+    const int threads = 256;
+    if (dtype == RG_DTYPE_BF16 && n % 8 == 0 && stride % 8 == 0 && gate_ld % 8 == 0 &&
+        (((uintptr_t)x | (uintptr_t)gate) & 15) == 0)
+        return rg_launch(sigmoid_gate_kernel<bf16, 8>, dim3((unsigned)((total / 8 + threads - 1) / threads)), dim3(threads), 0, s,
+                         1, (bf16*)x, (const bf16*)gate, gate_ld, groups, n, stride, total / 8);
+    const unsigned blocks = (unsigned)((total + threads - 1) / threads);
+    if (dtype == RG_DTYPE_BF16)
+        return rg_launch(sigmoid_gate_kernel<bf16, 1>, dim3(blocks), dim3(threads), 0, s, 1, (bf16*)x, (const bf16*)gate,
+                         gate_ld, groups, n, stride, total);
+    if (dtype == RG_DTYPE_F32)
+        return rg_launch(sigmoid_gate_kernel<float, 1>, dim3(blocks), dim3(threads), 0, s, 1, (float*)x, (const float*)gate,
+                         gate_ld, groups, n, stride, total);
     return RG_ERR_UNSUPPORTED;
 }

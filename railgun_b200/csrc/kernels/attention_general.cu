@@ -2,7 +2,8 @@
 // size up to 256, any page size, 32-bit or bfloat16 storage, all arithmetic in
 // 32-bit.  It serves the true 32-bit path and every shape the fast kernels
 // refuse.  A query at absolute position p of request r attends the keys of r
-// at positions [max(0, p - window + 1), p] and, with keep_first, also the first
+// at positions [max(0, p - window + 1), p] (window < 0: those of its own chunk
+// of -window positions up to its own) and, with keep_first, also the first
 // keep_first positions of r whatever the window (kept tokens keep their own
 // positions), read from the paged cache through r's block table (the step's
 // own keys are written before it runs).  Optional: `sink` [nh], one more term
@@ -44,7 +45,7 @@ __global__ void paged_attention_general_kernel(
     const int kvh = h / (nh / nkv);
     const int r = req_of_token[t];
     const int pos = positions[t];
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_seen(pos, window);
     const int* bt = block_table + (size_t)r * max_blocks;
     const A* qrow = q + (size_t)t * q_stride + (size_t)h * d;
     for (int i = threadIdx.x; i < d; i += blockDim.x) qs[i] = to_f32(qrow[i]) * scale;
@@ -55,7 +56,7 @@ __global__ void paged_attention_general_kernel(
     const size_t page_elems = (size_t)2 * nkv * page_size * d;
     // the keys a query sees, numbered 0 .. n_sink + (pos - lo): the kept first tokens that the window has passed, then the window
     // (pooled entries are numbered the same way, before the window)
-    const int n_sink = pool > 0 ? (pos - window + 1 >= pool ? (pos - window + 1) / pool : 0) : min(keep_first, lo);
+    const int n_sink = pool > 0 ? (pos - window + 1 >= pool ? (pos - window + 1) / pool : 0) : (window > 0 ? min(keep_first, lo) : 0);
     const int* pbt = pool > 0 ? pool_table + (size_t)r * pool_blocks : bt;
     const A* first_kv = pool > 0 ? pool_kv : kv_cache;
     const int n_seen = n_sink + pos - lo + 1;

@@ -53,7 +53,7 @@ __global__ void latent_rope_cache_kernel(const A* __restrict__ proj, int ld, int
                                          A* __restrict__ cache, const float* __restrict__ norm_w, float eps,
                                          const double* __restrict__ freq, int rot_dims, int interleaved,
                                          const int* __restrict__ positions, const int* __restrict__ slots,
-                                         int H, int dn, int dr, int R, A* __restrict__ q_back) {
+                                         int H, int dn, int dr, int R, A* __restrict__ q_back, float mult) {
     __shared__ float scratch[33];
     extern __shared__ float cs[];                    // cos | sin of the token's rot_dims / 2 angles; then H * dr rotated numbers
     float* rot_q = cs + rot_dims;
@@ -63,8 +63,12 @@ __global__ void latent_rope_cache_kernel(const A* __restrict__ proj, int ld, int
     const double pos = (double)positions[t];
     const A* row = proj + (size_t)t * ld;
     const int D = R + dr;
-    for (int i = threadIdx.x; i < (rot_dims >> 1); i += blockDim.x)        // angles in 64-bit: a handful per token
-        rotary_cos_sin(pos, freq[i], &cs[i], &cs[(rot_dims >> 1) + i]);
+    for (int i = threadIdx.x; i < (rot_dims >> 1); i += blockDim.x) {      // angles in 64-bit: a handful per token
+        float c, sn;
+        rotary_cos_sin(pos, freq[i], &c, &sn);
+        cs[i] = c * mult;
+        cs[(rot_dims >> 1) + i] = sn * mult;
+    }
     __syncthreads();
     for (int i = threadIdx.x; i < H * dr; i += blockDim.x) {     // all heads' rotated parts at once
         const int h = i / dr, j = i - h * dr;
@@ -92,11 +96,12 @@ __global__ void latent_rope_cache_kernel(const A* __restrict__ proj, int ld, int
     rotate_pairs(lat + R, dst + R, dr, rot_dims, interleaved != 0, cs);
 }
 
-// q_in_place: the rotated query parts also replace the unrotated ones in proj (qa may then be null).
+// mult: what cos and sin are multiplied by.  q_in_place: the rotated query parts also replace the unrotated ones in
+// proj (qa may then be null).
 extern "C" int rg_latent_rope_cache(const void* proj, int ld, int kv_off, void* qa, void* cache, int dtype,
                                     const float* norm_w, float eps, const double* freq, int rot_dims,
                                     int interleaved, const int* positions, const int* slots, int T, int H, int dn, int dr, int R,
-                                    int q_in_place, void* stream) {
+                                    int q_in_place, float mult, void* stream) {
     if (T <= 0) return 0;
     if (rot_dims < 0 || rot_dims > dr || (rot_dims & 1) || R < 1 || H < 1 || rot_dims > 8192) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
@@ -107,11 +112,11 @@ extern "C" int rg_latent_rope_cache(const void* proj, int ld, int kv_off, void* 
     if (dtype == RG_DTYPE_BF16)
         return rg_launch(latent_rope_cache_kernel<bf16>, dim3(T), dim3(rope_threads), cs_bytes, s, 1, (const bf16*)proj, ld,
                          kv_off, (bf16*)qa, (bf16*)cache, norm_w, eps, freq, rot_dims, interleaved, positions, slots, H, dn, dr, R,
-                         q_in_place ? (bf16*)proj : (bf16*)nullptr);
+                         q_in_place ? (bf16*)proj : (bf16*)nullptr, mult);
     if (dtype == RG_DTYPE_F32)
         return rg_launch(latent_rope_cache_kernel<float>, dim3(T), dim3(rope_threads), cs_bytes, s, 1, (const float*)proj, ld,
                          kv_off, (float*)qa, (float*)cache, norm_w, eps, freq, rot_dims, interleaved, positions, slots, H, dn, dr, R,
-                         q_in_place ? (float*)proj : (float*)nullptr);
+                         q_in_place ? (float*)proj : (float*)nullptr, mult);
     return RG_ERR_UNSUPPORTED;
 }
 
@@ -270,11 +275,14 @@ __global__ void latent_pack_kv_kernel(const A* __restrict__ kn, const A* __restr
     const int ctx = context_lens[r];
     if (j * page_size >= ctx) return;
     const int page = block_table[(size_t)r * max_blocks + j];
-    if (page < 0) return;
     const int n = min(page_size, ctx - j * page_size);
     const int d = dn + dr, D = R + dr;
     const size_t tp = (size_t)r * max_blocks + j;                  // the temporary page
     A* kdst = kv + tp * 2 * H * page_size * d;
+    if (page < 0) {                                                // a window has passed it: masked, but read beside the edge
+        for (int i = threadIdx.x; i < 2 * H * page_size * d; i += blockDim.x) kdst[i] = from_f32<A>(0.f);
+        return;
+    }
     A* vdst = kdst + (size_t)H * page_size * d;
     const size_t row0 = tp * page_size;
     const A* krot = cache + (size_t)page * page_size * D + R;

@@ -24,6 +24,8 @@
 // Output rows may be further apart than their width (out_ld), and the output may be multiplied by a constant
 // (out_scale) before its one rounding.
 //
+// A negative window stands for chunks: a query sees the keys of its own chunk of -window positions, counted from
+// position 0, up to its own.
 // With a window, and with `pool` > 0, tokens that have left the window are seen in blocks of `pool` instead: entry b
 // of a second set of pages (pool_kv, its own block table; pages of as many entries as the others have tokens) stands
 // for the positions b pool .. (b + 1) pool - 1, and the query at position p sees it once the block lies wholly before
@@ -175,7 +177,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const int* bt = block_table + (size_t)r * max_blocks;
     const int p0 = positions[row0];
     const int hi = p0 + nrows - 1;                                 // last key any row of the tile attends
-    const int lo = window > 0 ? max(0, p0 - window + 1) : 0;
+    const int lo = first_seen(p0, window);
     int kt0 = lo / BN;
     const int kt1 = hi / BN;
     // keep: with a window, the request's first `keep` tokens stay visible.  Their nk tiles come first, then the
@@ -222,6 +224,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;      // rows g and g + 8 of this warp's 16
     const int g = lane >> 2, tq = lane & 3;
     const int prow0 = p0 + warp * 16 + g, prow1 = prow0 + 8;       // absolute positions of the two rows
+    const int from0 = first_seen(prow0, window), from1 = first_seen(prow1, window);
     // ldmatrix source coordinates
     const int a_row = warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, a_col = (lane >> 4) * 8;
     const int b_key = (lane & 7) + (lane >> 4) * 8, b_dim = ((lane >> 3) & 1) * 8;          // K as B operand
@@ -253,7 +256,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
         const int wfirst = p0 + warp * 16, wlast = wfirst + 15;      // warp-uniform: every lane takes the same branch
         const bool pool_tile = pooled(vt);
         const bool skip = pool_tile ? key_base >= pooled_seen(wlast, window, pool)
-                                    : key_base > wlast || (window > 0 && key_base + BN - 1 < wfirst - window + 1 && key_base >= keep);
+                                    : key_base > wlast || (key_base + BN - 1 < first_seen(wfirst, window) && key_base >= keep);
         if (!skip) {
             float s[BN / 8][4];
 #pragma unroll
@@ -275,7 +278,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
             }
             // scale into the log2 domain; mask by absolute position where the tile is not wholly attended
             const bool edge = pool_tile ? key_base + BN > pooled_seen(wfirst, window, pool)
-                                        : key_base + BN - 1 > wfirst || (window > 0 && key_base < wlast - window + 1);
+                                        : key_base + BN - 1 > wfirst || key_base < first_seen(wlast, window);
             const int see0 = pool_tile ? pooled_seen(prow0, window, pool) : 0, see1 = pool_tile ? pooled_seen(prow1, window, pool) : 0;
             float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
@@ -287,7 +290,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
                         const int key = key_base + j * 8 + tq * 2 + (e & 1);
                         const int prow = (e < 2) ? prow0 : prow1;
                         const bool ok = pool_tile ? key < (e < 2 ? see0 : see1)
-                                                  : key <= prow && (window <= 0 || key > prow - window || key < keep);
+                                                  : key <= prow && (key >= (e < 2 ? from0 : from1) || key < keep);
                         if (!ok) v = -INFINITY;
                     }
                     s[j][e] = v;
@@ -417,7 +420,7 @@ decode_attention_kernel(const bf16* __restrict__ q, int q_stride, const bf16* __
     const int r = req_of_token[t];
     const int pos = positions[t];
     const int* bt = block_table + (size_t)r * max_blocks;
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    const int lo = first_seen(pos, window);
     int lo_al = (lo / BN) * BN;
     // keep: with a window, the request's first `keep` tokens stay visible.  Their tiles (kept_al keys) come first
     // in the splits' key numbers, directly before the window's first tile: a key number below lo_al stands for
@@ -828,6 +831,7 @@ extern "C" int rg_prefill_attention_sink(const void* q, int q_stride, void* out,
     if (n_tiles <= 0) return 0;
     if (keep_first < 0 || !pool_ok(pool_kv, pool_table, pool, window, keep_first) || out_ld < nh * d || out_ld % 2)
         return RG_ERR_UNSUPPORTED;
+    if (q_stride % 8 || ((uintptr_t)q & 15)) return RG_ERR_UNSUPPORTED;          // 16-byte copies of q's rows
     if (d % 16 || d < 16 || d > 256 || nkv < 1 || nh < nkv || nh % nkv || (long long)n_tiles * nh > 0x7fffffffll)
         return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
@@ -940,6 +944,7 @@ static int rg_decode_attention_any(const void* q, int q_stride, void* out, const
     if (n_tokens <= 0) return 0;
     if (out_ld == 0) out_ld = nh * d;
     if (cluster_merge && (sink || gate || pool)) return RG_ERR_UNSUPPORTED;
+    if (q_stride % 8 || ((uintptr_t)q & 15)) return RG_ERR_UNSUPPORTED;          // 16-byte copies of q's rows
     if (d % 16 || d < 16 || d > 256 || nkv < 1 || nh < nkv || nh % nkv || num_splits < 1) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const float scale_log2 = scale * 1.4426950408889634f;

@@ -85,12 +85,21 @@ __device__ __forceinline__ float gated_act(float g, float u, int kind, float lim
     return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
 }
 
-// Activations without a gate, in 32-bit.  kind 0: the square of relu; 1: relu; 2: gelu (tanh form); 3: silu.
+// Activations without a gate, in 32-bit.  kind 0: the square of relu; 1: relu; 2: gelu (tanh form); 3: silu; 4: gelu
+// (exact, by the error function).
 __device__ __forceinline__ float plain_act(float v, int kind) {
     if (kind == 0) { const float r = fmaxf(v, 0.f); return r * r; }
     if (kind == 1) return fmaxf(v, 0.f);
     if (kind == 2) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+    if (kind == 4) return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
     return v / (1.f + expf(-v));
+}
+
+// The first position that the query at position p sees.  window > 0: a sliding window, p and the window - 1 positions
+// before it; window < 0: chunks of -window positions counted from position 0, the query's own chunk; 0: everything.
+// Never decreases with p.
+__device__ __forceinline__ int first_seen(int p, int window) {
+    return window > 0 ? max(0, p - window + 1) : (window < 0 ? p - p % -window : 0);
 }
 
 #define RG_LAUNCH_RESULT() ((int)cudaGetLastError())

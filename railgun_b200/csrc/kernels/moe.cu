@@ -2,8 +2,9 @@
 // those groups, and the weighted sum.
 //
 //   z = W_r h (32-bit), s = softmax(z) over all N router outputs (or, scoring 1, s = sigmoid(z), each on its own)
-//   the `top` outputs with the largest s + correction are chosen; their weights are s / (sum of the chosen s
-//   + 1e-20).  Outputs E..N-1 stand for identity experts (the expert's result is h itself); outputs 0..E-1
+//   the `top` outputs with the largest s + correction are chosen, all outputs or only those of the `keep` best of
+//   `groups` equal groups of neighbours (a group is as good as its best output); their weights are s / (sum of the
+//   chosen s + 1e-20), or s, times a constant.  Outputs E..N-1 stand for identity experts (the expert's result is h itself); outputs 0..E-1
 //   for gated experts  down(silu(gate h) * (up h)).
 //   out = sum_k weight_k * expert_k(h)  (+ an always-on shared expert's result, computed elsewhere)
 //
@@ -23,8 +24,12 @@ template <typename A>
 __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restrict__ router,
                                  const float* __restrict__ correction, int* __restrict__ ids,
                                  float* __restrict__ weights, int T, int W, int N, int top, int renormalize,
-                                 int scoring) {
-    extern __shared__ float sm[];                 // per token of the block: N scores, N choice scores
+                                 int scoring, int groups, int keep, float scale, const float* __restrict__ gate_row,
+                                 float* __restrict__ gate) {
+    extern __shared__ float sm[];                 // per token of the block: N scores, N choice scores, groups' bests, a gate
+    const int stride = 2 * N + groups + 1;
+    // gate_row: one more row of the router whose logit's sigmoid is left in gate[t] (a shared expert's weight)
+    const int rows = N + (gate_row ? 1 : 0);
     pdl_wait();
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
@@ -34,8 +39,8 @@ __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restric
     // every lane adds its own elements in index order (four at a time where rows start on 16-byte boundaries),
     // then the lanes are added up: a token's logits do not depend on what else is in the step
     const bool vec = (W & 3) == 0 && sizeof(A) == 2;
-    for (int n = warp; n < N; n += nwarps) {
-        const float* wr = router + (size_t)n * W;
+    for (int n = warp; n < rows; n += nwarps) {
+        const float* wr = n < N ? router + (size_t)n * W : gate_row;
         float dot[ROUTE_TOKENS];
 #pragma unroll
         for (int j = 0; j < ROUTE_TOKENS; ++j) dot[j] = 0.f;
@@ -67,14 +72,15 @@ __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restric
 #pragma unroll
         for (int j = 0; j < ROUTE_TOKENS; ++j) {
             const float d = warp_sum(dot[j]);
-            if (lane == 0) base[(size_t)j * 2 * N + n] = d;
+            if (lane == 0) base[(size_t)j * stride + (n < N ? n : 2 * N + groups)] = d;
         }
     }
     __syncthreads();
     for (int j = warp; j < nt; j += nwarps) {
         const int t = t0 + j;
-        float* s = base + (size_t)j * 2 * N;
+        float* s = base + (size_t)j * stride;
         float* c = s + N;
+        if (gate_row && lane == 0) gate[t] = 1.f / (1.f + expf(-s[2 * N + groups]));
         if (scoring == 1) {
             // without a correction the largest scores are the largest logits, which do not saturate
             for (int n = lane; n < N; n += 32) {
@@ -94,6 +100,28 @@ __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restric
             for (int n = lane; n < N; n += 32) { const float p = s[n] * inv; s[n] = p; c[n] = p + (correction ? correction[n] : 0.f); }
         }
         __syncwarp();
+        if (groups > 0) {
+            // the outputs of all but the best `keep` groups drop out (of equal groups the first)
+            float* best_of = c + N;
+            const int gs = N / groups;
+            for (int g = 0; g < groups; ++g) {
+                float b = -INFINITY;
+                for (int n = lane; n < gs; n += 32) b = fmaxf(b, c[g * gs + n]);
+                b = warp_max(b);
+                if (lane == 0) best_of[g] = b;
+            }
+            __syncwarp();
+            for (int g = 0; g < groups; ++g) {
+                const float b = best_of[g];
+                int ahead = 0;
+                for (int o = lane; o < groups; o += 32) ahead += best_of[o] > b || (best_of[o] == b && o < g);
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) ahead += __shfl_xor_sync(0xffffffffu, ahead, o);
+                if (ahead >= keep)
+                    for (int n = lane; n < gs; n += 32) c[g * gs + n] = -INFINITY;
+            }
+            __syncwarp();
+        }
         float chosen_sum = 0.f;
         for (int k = 0; k < top; ++k) {
             float best = -INFINITY;
@@ -116,27 +144,30 @@ __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restric
             }
             __syncwarp();
         }
-        const float norm = renormalize ? 1.f / (chosen_sum + 1e-20f) : 1.f;
+        const float norm = (renormalize ? 1.f / (chosen_sum + 1e-20f) : 1.f) * scale;
         for (int k = lane; k < top; k += 32) weights[(size_t)t * top + k] *= norm;
         __syncwarp();
     }
 }
 
 extern "C" int rg_moe_route(const void* x, int dtype, const float* router, const float* correction, int* ids,
-                            float* weights, int T, int W, int N, int top, int renormalize, int scoring, void* stream) {
+                            float* weights, int T, int W, int N, int top, int renormalize, int scoring, int groups, int keep,
+                            float scale, const float* gate_row, float* gate, void* stream) {
     if (T <= 0) return 0;
-    if (top < 1 || top > N || scoring < 0 || scoring > 1) return RG_ERR_UNSUPPORTED;
-    const size_t smem = (size_t)ROUTE_TOKENS * 2 * N * sizeof(float);
+    if (top < 1 || top > N || scoring < 0 || scoring > 1 || groups < 0 || (gate_row && !gate)) return RG_ERR_UNSUPPORTED;
+    if (groups > 0 && (N % groups || keep < 1 || keep > groups || top > keep * (N / groups))) return RG_ERR_UNSUPPORTED;
+    const size_t smem = (size_t)ROUTE_TOKENS * (2 * N + groups + 1) * sizeof(float);
     if (smem > 48 * 1024) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    const int warps = N < 4 ? 4 : (N > 32 ? 32 : N);               // a warp per router row, up to 32
+    const int rows = N + (gate_row ? 1 : 0);
+    const int warps = rows < 4 ? 4 : (rows > 32 ? 32 : rows);      // a warp per router row, up to 32
     dim3 grid((T + ROUTE_TOKENS - 1) / ROUTE_TOKENS), block(warps * 32);
     if (dtype == RG_DTYPE_BF16)
         return rg_launch(moe_route_kernel<bf16>, grid, block, smem, s, 1, (const bf16*)x, router, correction, ids,
-                         weights, T, W, N, top, renormalize, scoring);
+                         weights, T, W, N, top, renormalize, scoring, groups, keep, scale, gate_row, gate);
     if (dtype == RG_DTYPE_F32)
         return rg_launch(moe_route_kernel<float>, grid, block, smem, s, 1, (const float*)x, router, correction, ids,
-                         weights, T, W, N, top, renormalize, scoring);
+                         weights, T, W, N, top, renormalize, scoring, groups, keep, scale, gate_row, gate);
     return RG_ERR_UNSUPPORTED;
 }
 
@@ -297,11 +328,13 @@ extern "C" int rg_moe_grouped_gemm(const void* a, int lda, const int* src, int s
     return RG_ERR_UNSUPPORTED;
 }
 
-// out[t] (32-bit) = sum_k weights[t, k] * (ids[t, k] < E ? y[pair_pos[t, k]] : x[t])  (+ shared[t]); weights null: all 1
+// out[t] (32-bit) = sum_k weights[t, k] * (ids[t, k] < E ? y[pair_pos[t, k]] : x[t])  (+ shared_w[t] shared[t]); weights
+// null: all 1, shared_w null: 1
 template <typename A>
 __global__ void moe_combine_kernel(const A* __restrict__ x, const A* __restrict__ y, const A* __restrict__ shared,
                                    const int* __restrict__ ids, const float* __restrict__ weights,
-                                   const int* __restrict__ pair_pos, float* __restrict__ out, int W, int E, int top) {
+                                   const int* __restrict__ pair_pos, const float* __restrict__ shared_w,
+                                   float* __restrict__ out, int W, int E, int top) {
     pdl_wait();
     pdl_trigger();
     extern __shared__ float csm[];                 // per choice: weight, row of y (-1: the token's own row)
@@ -314,6 +347,7 @@ __global__ void moe_combine_kernel(const A* __restrict__ x, const A* __restrict_
         crow[k] = ids[p] < E ? pair_pos[p] : -1;
     }
     __syncthreads();
+    const float sw = shared && shared_w ? shared_w[t] : 1.f;
     for (int i = threadIdx.x; i < W; i += blockDim.x) {
         float v = 0.f;
         const float own = to_f32(x[(size_t)t * W + i]);
@@ -321,25 +355,62 @@ __global__ void moe_combine_kernel(const A* __restrict__ x, const A* __restrict_
             const int row = crow[k];
             v += cw[k] * (row >= 0 ? to_f32(y[(size_t)row * W + i]) : own);
         }
-        if (shared) v += to_f32(shared[(size_t)t * W + i]);
+        if (shared) v += sw * to_f32(shared[(size_t)t * W + i]);
         out[(size_t)t * W + i] = v;
     }
 }
 
+// The same from bfloat16 rows with four numbers per thread and step, where every choice has an expert behind it.
+__global__ void moe_combine4_kernel(const bf16* __restrict__ y, const bf16* __restrict__ shared,
+                                    const float* __restrict__ weights, const int* __restrict__ pair_pos,
+                                    const float* __restrict__ shared_w, float* __restrict__ out, int W, int top) {
+    pdl_wait();
+    pdl_trigger();
+    extern __shared__ float csm[];
+    const int t = blockIdx.x;
+    float* cw = csm;
+    int* crow = reinterpret_cast<int*>(csm + top);
+    for (int k = threadIdx.x; k < top; k += blockDim.x) {
+        const size_t p = (size_t)t * top + k;
+        cw[k] = weights ? weights[p] : 1.f;
+        crow[k] = pair_pos[p];
+    }
+    __syncthreads();
+    const float sw = shared && shared_w ? shared_w[t] : 1.f;
+    auto add = [](float4& v, float w, const bf16* p) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+        v.x += w * a.x; v.y += w * a.y; v.z += w * b.x; v.w += w * b.y;
+    };
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int k = 0; k < top; ++k) add(v, cw[k], y + (size_t)crow[k] * W + i);
+        if (shared) add(v, sw, shared + (size_t)t * W + i);
+        *reinterpret_cast<float4*>(out + (size_t)t * W + i) = v;
+    }
+}
+
+// all_experts: no choice stands for an identity expert
 extern "C" int rg_moe_combine(const void* x, const void* y, const void* shared, int dtype, const int* ids,
-                              const float* weights, const int* pair_pos, float* out, int T, int W, int E, int top,
-                              void* stream) {
+                              const float* weights, const int* pair_pos, const float* shared_w, float* out, int T, int W,
+                              int E, int top, int all_experts, void* stream) {
     if (T <= 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = W >= 1024 ? 256 : 128;
     const size_t csmem = (size_t)top * 8;
     if (top < 1 || csmem > 48 * 1024) return RG_ERR_UNSUPPORTED;
+    if (dtype == RG_DTYPE_BF16 && all_experts && W % 4 == 0 && (((uintptr_t)y | (uintptr_t)shared) & 7) == 0 &&
+        ((uintptr_t)out & 15) == 0)
+        return rg_launch(moe_combine4_kernel, dim3(T), dim3(W >= 2048 ? 256 : 128), csmem, s, 1, (const bf16*)y,
+                         (const bf16*)shared, weights, pair_pos, shared_w, out, W, top);
     if (dtype == RG_DTYPE_BF16)
         return rg_launch(moe_combine_kernel<bf16>, dim3(T), dim3(threads), csmem, s, 1, (const bf16*)x, (const bf16*)y,
-                         (const bf16*)shared, ids, weights, pair_pos, out, W, E, top);
+                         (const bf16*)shared, ids, weights, pair_pos, shared_w, out, W, E, top);
     if (dtype == RG_DTYPE_F32)
         return rg_launch(moe_combine_kernel<float>, dim3(T), dim3(threads), csmem, s, 1, (const float*)x, (const float*)y,
-                         (const float*)shared, ids, weights, pair_pos, out, W, E, top);
+                         (const float*)shared, ids, weights, pair_pos, shared_w, out, W, E, top);
     return RG_ERR_UNSUPPORTED;
 }
 

@@ -13,17 +13,31 @@
 // Structured State Space Duality").  The products are 32-bit fused multiply-adds; the exponents' sums are 64-bit, since
 // their differences are small beside them where a head forgets fast.
 //
+// The same recurrence with the logarithm of every token's decay given instead of A_log and dt (then dt holds the weights of
+// the new terms only), without D, and with n, the sum of the B's with the same decays and weights, carried as one more
+// row of the state ("ones": the column of a value that is always 1), for memories that divide by n . C.  n and n . C are
+// sums that the light blocks of the launches work out.
+//
 // The step's tokens are packed request by request (cu_seqlens); a request's chunks start at its first token of the step.
 #include "chunk_scan.cuh"
 
-// c_i of the chunk's tokens for head h (64-bit), by the block's first warp; dt of the tokens into sdt.
-__device__ __forceinline__ void chunk_sums(const float* __restrict__ dt, float A_log, int lo, int n, int H, int h,
+// c_i of the chunk's tokens for head h (64-bit), by the block's first warp; dt of the tokens into sdt.  a_t is loga's
+// number, or without loga -exp(A_log) dt_t.
+__device__ __forceinline__ void chunk_sums(const float* __restrict__ dt, const float* __restrict__ loga,
+                                           const float* __restrict__ A_log, int lo, int n, int H, int h,
                                            double* __restrict__ cum, float* __restrict__ sdt) {
     if (threadIdx.x < 32) {
         const int i0 = 2 * threadIdx.x, i1 = i0 + 1;
         const float d0 = i0 < n ? dt[(size_t)(lo + i0) * H + h] : 0.f, d1 = i1 < n ? dt[(size_t)(lo + i1) * H + h] : 0.f;
-        const float rate = -expf(A_log);
-        const double a0 = (double)(rate * d0), a1 = (double)(rate * d1);
+        double a0, a1;
+        if (loga) {
+            a0 = i0 < n ? (double)loga[(size_t)(lo + i0) * H + h] : 0.0;
+            a1 = i1 < n ? (double)loga[(size_t)(lo + i1) * H + h] : 0.0;
+        } else {
+            const float rate = -expf(A_log[h]);
+            a0 = (double)(rate * d0);
+            a1 = (double)(rate * d1);
+        }
         double s = a0 + a1;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -37,14 +51,14 @@ __device__ __forceinline__ void chunk_sums(const float* __restrict__ dt, float A
     }
 }
 
-// x, B, C: rows ld apart (head h's x at column h dv, group g's B and C at column g N).  sums [chunks, H, dv, N], decays
-// [chunks, H], dots [chunks, G, 64, 64] = B_j . C_i at [j][i].  grid: chunks, H (tiles of S: z) and then G (z = 0).
+// x, B, C: rows ld apart (head h's x at column h dv, group g's B and C at column g N).  sums [chunks, H, dv + ones, N],
+// decays [chunks, H], dots [chunks, G, 64, 64] = B_j . C_i at [j][i].  grid: chunks, H (tiles of S: z) and then G (z = 0).
 template <int W>
 __global__ void __launch_bounds__(NTH)
 chunk_states_kernel(const float* __restrict__ x, const float* __restrict__ B, const float* __restrict__ C, int ld,
-                    const float* __restrict__ dt, const float* __restrict__ A_log, const int* __restrict__ cu, int R,
-                    float* __restrict__ sums, float* __restrict__ decays, float* __restrict__ dots, int H, int G, int N,
-                    int dv, int ntiles) {
+                    const float* __restrict__ dt, const float* __restrict__ loga, const float* __restrict__ A_log,
+                    const int* __restrict__ cu, int R, float* __restrict__ sums, float* __restrict__ decays,
+                    float* __restrict__ dots, int H, int G, int N, int dv, int ntiles, int ones) {
     extern __shared__ __align__(16) float sm[];
     float (*sA)[PITCH] = reinterpret_cast<float (*)[PITCH]>(sm);                            // [CH][PITCH]
     float (*sB)[TILE * W + 4] = reinterpret_cast<float (*)[TILE * W + 4]>(sm + CH * PITCH);     // [CH][TILE W + 4]
@@ -80,11 +94,27 @@ chunk_states_kernel(const float* __restrict__ x, const float* __restrict__ B, co
 #pragma unroll
         for (int i = 0; i < 4; ++i)
             *reinterpret_cast<float4*>(out + (4 * ty + i) * CH + 4 * tx) = make_float4(a1[i][0], a1[i][1], a1[i][2], a1[i][3]);
+        if (!ones) return;
+        for (int h = g * (H / G); h < (g + 1) * (H / G); ++h) {         // the row of n: every head of the group
+            __syncthreads();
+            chunk_sums(dt, loga, A_log, lo, n, H, h, cum, sdt);
+            __syncthreads();
+            const double last = cum[CH - 1];
+            __syncthreads();
+            if (threadIdx.x < n) sdt[threadIdx.x] *= expf((float)(last - cum[threadIdx.x]));
+            __syncthreads();
+            for (int k = threadIdx.x; k < N; k += NTH) {
+                float s = 0.f;
+#pragma unroll 8
+                for (int t = 0; t < n; ++t) s += B[(size_t)(lo + t) * ld + (size_t)g * N + k] * sdt[t];
+                sums[(((size_t)blockIdx.x * H + h) * (dv + 1) + dv) * N + k] = s;
+            }
+        }
         return;
     }
     const int h = blockIdx.y, grp = h / (H / G);
     const int j0 = (blockIdx.z / ntiles) * TILE, n0 = (blockIdx.z % ntiles) * TILE * W;      // columns of S, rows of S
-    chunk_sums(dt, A_log[h], lo, n, H, h, cum, sdt);
+    chunk_sums(dt, loga, A_log, lo, n, H, h, cum, sdt);
     __syncthreads();
     const double end = cum[CH - 1];
     for (int e = threadIdx.x; e < CH * TILE; e += NTH) {
@@ -98,7 +128,7 @@ chunk_states_kernel(const float* __restrict__ x, const float* __restrict__ B, co
     }
     __syncthreads();
     multiply<W>(acc, sA, sB, n, ty, tx);
-    float* out = sums + ((size_t)blockIdx.x * H + h) * dv * N;
+    float* out = sums + ((size_t)blockIdx.x * H + h) * (dv + ones) * N;
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
         const int j = j0 + 4 * ty + i;
@@ -119,12 +149,13 @@ chunk_states_kernel(const float* __restrict__ x, const float* __restrict__ B, co
     if (blockIdx.z == 0 && threadIdx.x == 0) decays[(size_t)blockIdx.x * H + h] = expf((float)end);
 }
 
-// before [chunks, H, dv, N]: the state before every chunk.  o [T, H, dv].  grid: chunks, H, tiles of 64 columns.
+// before [chunks, H, dv + ones, N]: the state before every chunk.  o [T, H, dv + ones].  grid: chunks, H, tiles of 64
+// columns, and with `ones` a light block for n . C.
 __global__ void __launch_bounds__(NTH)
 chunk_outputs_kernel(const float* __restrict__ x, const float* __restrict__ C, int ld, const float* __restrict__ dt,
-                     const float* __restrict__ A_log, const float* __restrict__ D, const int* __restrict__ cu, int R,
-                     const float* __restrict__ before, const float* __restrict__ dots, float* __restrict__ o, int H, int G,
-                     int N, int dv) {
+                     const float* __restrict__ loga, const float* __restrict__ A_log, const float* __restrict__ D,
+                     const int* __restrict__ cu, int R, const float* __restrict__ before, const float* __restrict__ dots,
+                     float* __restrict__ o, int H, int G, int N, int dv, int ones) {
     __shared__ __align__(16) float sA[CH][PITCH];
     __shared__ __align__(16) float sB[CH][PITCH];
     __shared__ double cum[CH];
@@ -135,8 +166,25 @@ chunk_outputs_kernel(const float* __restrict__ x, const float* __restrict__ C, i
     if (!find_chunk(cu, R, blockIdx.x, r, lo, n)) return;
     const int h = blockIdx.y, grp = h / (H / G), j0 = blockIdx.z * TILE;
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
-    chunk_sums(dt, A_log[h], lo, n, H, h, cum, sdt);
+    chunk_sums(dt, loga, A_log, lo, n, H, h, cum, sdt);
     __syncthreads();
+    if (j0 >= dv) {
+        // n . C_i: four threads a token (neighbouring lanes) share its sums over the chunk's tokens and over n's numbers
+        const float* dd = dots + ((size_t)blockIdx.x * G + grp) * CH * CH;
+        const float* nb = before + (((size_t)blockIdx.x * H + h) * (dv + 1) + dv) * N;
+        const int i = threadIdx.x >> 2, part = threadIdx.x & 3;
+        float s = 0.f, b = 0.f;
+        if (i < n) {
+            const float* c = C + (size_t)(lo + i) * ld + (size_t)grp * N;
+            for (int j = part; j <= i; j += 4) s += dd[j * CH + i] * sdt[j] * expf((float)(cum[i] - cum[j]));
+            for (int k = part; k < N; k += 4) b += nb[k] * c[k];
+            s += b * expf((float)cum[i]);
+        }
+        s += __shfl_xor_sync(0xffffffffu, s, 1);
+        s += __shfl_xor_sync(0xffffffffu, s, 2);
+        if (i < n && part == 0) o[((size_t)(lo + i) * H + h) * (dv + 1) + dv] = s;
+        return;
+    }
     if (threadIdx.x < CH) grown[threadIdx.x] = expf((float)cum[threadIdx.x]);
     // within the chunk
     const float* d = dots + ((size_t)blockIdx.x * G + grp) * CH * CH;
@@ -150,14 +198,14 @@ chunk_outputs_kernel(const float* __restrict__ x, const float* __restrict__ C, i
     }
     __syncthreads();
     float acc[4][4];
-    const float skip = D[h];
+    const float skip = D ? D[h] : 0.f;
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) acc[i][j] = skip * sB[4 * ty + i][4 * tx + j];
     multiply<1>(acc, sA, sB, min(n, 4 * (ty | 1) + 4), ty, tx);     // token j counts for the tokens from j on only
     // from the state before it
-    const float* S = before + (((size_t)blockIdx.x * H + h) * dv + j0) * N;
+    const float* S = before + (((size_t)blockIdx.x * H + h) * (dv + ones) + j0) * N;
     for (int k0 = 0; k0 < N; k0 += TILE) {
         __syncthreads();
         load_transposed(sA, C + (size_t)lo * ld + (size_t)grp * N, ld, n, N, k0, grown);
@@ -169,20 +217,22 @@ chunk_outputs_kernel(const float* __restrict__ x, const float* __restrict__ C, i
     for (int i = 0; i < 4; ++i) {
         const int t = 4 * ty + i;
         if (t >= n) continue;
-        float* out = o + ((size_t)(lo + t) * H + h) * dv + j0 + 4 * tx;
+        float* out = o + ((size_t)(lo + t) * H + h) * (dv + ones) + j0 + 4 * tx;
 #pragma unroll
         for (int j = 0; j < 4; ++j)
             if (j0 + 4 * tx + j < dv) out[j] = acc[i][j];
     }
 }
 
-// Scratch of the caller: sums [chunks, H, dv, N], decays [chunks, H], dots [chunks, G, 64, 64], with chunks at least
+// loga [T, H] or null (then A_log [H]); D [H] or null.  state [slots, H, dv + ones, N].
+// Scratch of the caller: sums [chunks, H, dv + ones, N], decays [chunks, H], dots [chunks, G, 64, 64], with chunks at least
 // T / 64 + R (rounded down).
-extern "C" int rg_ssd_chunk_scan(const float* x, const float* B, const float* C, int ld, const float* dt, const float* A_log,
-                                 const float* D, float* state, const int* cu_seqlens, const int* start_pos, const int* slots,
-                                 float* sums, float* decays, float* dots, float* o, int T, int R, int H, int G, int N, int dv,
-                                 void* stream) {
+extern "C" int rg_ssd_chunk_scan(const float* x, const float* B, const float* C, int ld, const float* dt, const float* loga,
+                                 const float* A_log, const float* D, float* state, const int* cu_seqlens, const int* start_pos,
+                                 const int* slots, float* sums, float* decays, float* dots, float* o, int T, int R, int H,
+                                 int G, int N, int dv, int ones, void* stream) {
     if (T <= 0 || R <= 0) return 0;
+    if ((!loga && !A_log) || ones < 0 || ones > 1) return RG_ERR_UNSUPPORTED;
     if (H < 1 || G < 1 || H % G || N < 1 || dv < 1 || H + G > 65535 || R > 65535) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const int chunks = T / CH + R;
@@ -194,19 +244,19 @@ extern "C" int rg_ssd_chunk_scan(const float* x, const float* B, const float* C,
     int e = 0;
 #define SSD_STATES(W) { \
         if (smem > 46 * 1024) e = (int)cudaFuncSetAttribute(chunk_states_kernel<W>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        if (e == 0) e = rg_launch(chunk_states_kernel<W>, g1, dim3(NTH), smem, s, 1, x, B, C, ld, dt, A_log, cu_seqlens, R, \
-                                  sums, decays, dots, H, G, N, dv, nt); }
+        if (e == 0) e = rg_launch(chunk_states_kernel<W>, g1, dim3(NTH), smem, s, 1, x, B, C, ld, dt, loga, A_log, \
+                                  cu_seqlens, R, sums, decays, dots, H, G, N, dv, nt, ones); }
     if (wide == 2) SSD_STATES(2) else SSD_STATES(1)
 #undef SSD_STATES
     if (e) return e;
-    const int M = dv * N;
+    const int M = (dv + ones) * N;
     const bool vec = M % 4 == 0 && ((uintptr_t)state & 15) == 0;
     const long long work = vec ? (long long)H * M / 4 : (long long)H * M;
     dim3 g2((unsigned)((work + 255) / 256), R);
     e = vec ? rg_launch(chunk_pass_kernel<4, false>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M, N)
             : rg_launch(chunk_pass_kernel<1, false>, g2, dim3(256), 0, s, 1, sums, (const float*)decays, state, cu_seqlens, start_pos, slots, H, M, N);
     if (e) return e;
-    dim3 g3(chunks, H, jt);
-    return rg_launch(chunk_outputs_kernel, g3, dim3(NTH), 0, s, 1, x, C, ld, dt, A_log, D, cu_seqlens, R, (const float*)sums,
-                     (const float*)dots, o, H, G, N, dv);
+    dim3 g3(chunks, H, jt + ones);
+    return rg_launch(chunk_outputs_kernel, g3, dim3(NTH), 0, s, 1, x, C, ld, dt, loga, A_log, D, cu_seqlens, R,
+                     (const float*)sums, (const float*)dots, o, H, G, N, dv, ones);
 }

@@ -313,7 +313,8 @@ extern "C" int rg_delta_prepare(float* qk, int ld, int G, int d, float q_scale, 
 // reads q/k head h / (H / Hqk).  v: rows v_ld apart (float or bfloat16), head h at column h dv.  decay [H] or g [T, H];
 // beta [T, H] or null (1); skip [H] or null (0); channel decay: w like k (rows w_ld apart, its own head h), bonus
 // [H, d].  state [slots, H, dv, d]: S transposed, a
-// thread's rows side by side.  o [T, H, dv] float.
+// thread's rows side by side.  o [T, H, dv] float.  ones 1: the last of the dv columns has no values in v (head h then is
+// at column h (dv - 1)); its value is always 1.
 //
 // The delta rule per token, with a = S_old^T k, b = S_old^T q (one pass over S, reduced together) and c = k . q:
 //   u = beta (v - g a);  o = g b + u c;  S <- g S + k u^T
@@ -343,7 +344,7 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
                   const float* __restrict__ w, int w_ld, const float* __restrict__ bonus,
                   float* __restrict__ state, const int* __restrict__ cu_seqlens,
                   const int* __restrict__ start_pos, const int* __restrict__ slots,
-                  float* __restrict__ o, int H, int Hqk, int d, int dv, int CB, int chunk, int vec) {
+                  float* __restrict__ o, int H, int Hqk, int d, int dv, int CB, int chunk, int vec, int ones) {
     extern __shared__ __align__(16) float sm[];
     constexpr int parts = PARTS;
     constexpr int DP = PARTS * DPER;                 // padded length of a q or k row
@@ -400,7 +401,7 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
         v_tt[x] = e < chunk * ncols ? e / ncols : chunk;
         v_i[x] = e - v_tt[x] * ncols;
     }
-    const V* vh = v + (size_t)h * dv + j0;
+    const V* vh = v + (size_t)h * (dv - ones) + j0;
     const float* qh = q + (size_t)hq * d;
     const float* kh = k + (size_t)hq * d;
     const float* wh = CHANNEL ? w + (size_t)h * d : nullptr;
@@ -440,7 +441,8 @@ state_scan_kernel(const float* __restrict__ q, int q_ld, const float* __restrict
     auto fetch = [&](int base, int n) {
 #pragma unroll
         for (int x = 0; x < SCAN_MAX_PREFETCH; ++x)
-            if (v_tt[x] < n) pv[x] = to_f32(vh[(size_t)(base + v_tt[x]) * v_ld + v_i[x]]);
+            if (v_tt[x] < n)
+                pv[x] = ones && j0 + v_i[x] == dv - 1 ? 1.f : to_f32(vh[(size_t)(base + v_tt[x]) * v_ld + v_i[x]]);
         if ((int)threadIdx.x < n) {
             pg = g ? g[(size_t)(base + threadIdx.x) * H + h] : fixed;
             pb = beta ? beta[(size_t)(base + threadIdx.x) * H + h] : 1.f;
@@ -576,8 +578,9 @@ extern "C" int rg_state_scan(const float* q, int q_ld, const float* k, int k_ld,
                              const float* decay, const float* g, const float* beta, const float* skip,
                              const float* w, int w_ld, const float* bonus, int rule, float* state,
                              const int* cu_seqlens, const int* start_pos, const int* slots, float* o, int R, int H,
-                             int Hqk, int d, int dv, void* stream) {
+                             int Hqk, int d, int dv, int ones, void* stream) {
     if (R <= 0) return 0;
+    if (ones < 0 || ones > 1 || (ones && dv < 2)) return RG_ERR_UNSUPPORTED;
     if (H < 1 || Hqk < 1 || H % Hqk || d < 1 || dv < 1 || d > 256 || rule < SCAN_SCALAR || rule > SCAN_CHANNEL)
         return RG_ERR_UNSUPPORTED;
     if (rule == SCAN_CHANNEL ? (!w || !bonus || decay || g || beta || skip) : (w || bonus || (!decay && !g) || (beta && !g)))
@@ -628,7 +631,7 @@ extern "C" int rg_state_scan(const float* q, int q_ld, const float* k, int k_ld,
     dim3 grid(R, H, col_blocks);
 #define SM_SCAN(DP_, PA_, DE_, V) return rg_launch(state_scan_kernel<DP_, PA_, DE_, V>, grid, dim3(threads), smem, s, 1, \
         q, q_ld, k, k_ld, (const V*)v, v_ld, decay, g, beta, skip, w, w_ld, bonus, state, cu_seqlens, start_pos, slots, o, H, Hqk, d, dv, CB, \
-        chunk, vec)
+        chunk, vec, ones)
 #define SM_SCAN_RULE(DP_, PA_, V) { if (rule == SCAN_DELTA) SM_SCAN(DP_, PA_, SCAN_DELTA, V); \
         if (rule == SCAN_CHANNEL) SM_SCAN(DP_, PA_, SCAN_CHANNEL, V); SM_SCAN(DP_, PA_, SCAN_SCALAR, V); }
 #define SM_SCAN_PARTS(DP_, V) switch (parts) { \

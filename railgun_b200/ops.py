@@ -223,15 +223,16 @@ def norm_sum(ys, weights, consts, eps: float) -> torch.Tensor:
 
 
 class PendingNormed:
-    """A part's output that is still to be RMS-normed (``weight``, ``eps``; the
+    """A part's output that is still to be normed (``weight``, ``eps``; the
     weight holds whatever constant factors follow the norm) before it is added
     to the residual: a norm that follows does both inside its own kernel;
-    ``materialize()`` computes the normed rows in 32-bit."""
+    ``materialize()`` computes the normed rows in 32-bit.  With ``bias`` the
+    norm is a layer norm, else an RMS norm."""
 
-    __slots__ = ("y", "weight", "eps")
+    __slots__ = ("y", "weight", "eps", "bias")
 
-    def __init__(self, y, weight, eps: float):
-        self.y, self.weight, self.eps = y, weight, float(eps)
+    def __init__(self, y, weight, eps: float, bias=None):
+        self.y, self.weight, self.eps, self.bias = y, weight, float(eps), bias
 
     @property
     def shape(self):
@@ -239,8 +240,47 @@ class PendingNormed:
 
     def materialize(self) -> torch.Tensor:
         out = torch.zeros(self.y.shape, dtype=torch.float32, device=self.y.device)
-        add_postnorm_rmsnorm(out, self, None, 0.0, None)
+        if self.bias is not None:
+            stream_norm(out, self, None, None)
+        else:
+            add_postnorm_rmsnorm(out, self, None, 0.0, None)
         return out
+
+
+def stream_norm(resid: torch.Tensor, pending, norm, out_dtype, rows: torch.Tensor | None = None):
+    """resid += ``pending`` (a ``PendingNormed`` with either kind of norm, a plain tensor, None), in place and in
+    32-bit; then the new rows in ``out_dtype`` (None: nothing is returned), normed by ``norm`` = (weight, bias, eps): a
+    layer norm, or an RMS norm when the bias is None; ``norm`` None: as they are.  ``rows`` as in ``add_rmsnorm``."""
+    _check(resid, "resid", torch.float32)
+    T, H = resid.shape
+
+    def kind_of(weight, bias, name):
+        for t in (weight, bias):
+            if t is not None:
+                _check(t, name, torch.float32)
+                if t.numel() != H:
+                    raise KernelError(f"{name} has {t.numel()} elements, rows have {H}")
+        return 0 if weight is None else (1 if bias is None else 2)
+
+    y, post_w, post_b, post_eps = pending, None, None, 0.0
+    if isinstance(pending, PendingNormed):
+        y, post_w, post_b, post_eps = pending.y, pending.weight, pending.bias, pending.eps
+    if y is not None:
+        _check(y, "pending")
+        if y.shape != resid.shape:
+            raise KernelError(f"pending {tuple(y.shape)} vs residual {tuple(resid.shape)}")
+    pre_w, pre_b, pre_eps = norm if norm is not None else (None, None, 0.0)
+    n_out = T
+    if rows is not None:
+        _check(rows, "rows", torch.int32)
+        n_out = rows.numel()
+    out = torch.empty((n_out, H), dtype=out_dtype, device=resid.device) if out_dtype is not None else None
+    _ok(_fn("stream_norm", "rg_stream_norm")(
+        _ptr(resid), _ptr(y), c_int(_dtype_code(y) if y is not None else 0), c_int(kind_of(post_w, post_b, "post-norm")),
+        _ptr(post_w), _ptr(post_b), c_float(post_eps), c_int(kind_of(pre_w, pre_b, "norm")), _ptr(pre_w), _ptr(pre_b),
+        c_float(pre_eps), _ptr(out), c_int(_dtype_code(out) if out is not None else 0), _ptr(rows), c_int(n_out), c_int(H),
+        _stream()), "stream_norm")
+    return out
 
 
 def add_postnorm_rmsnorm(resid: torch.Tensor, pending, weight, eps: float, out_dtype, rows: torch.Tensor | None = None,
@@ -255,7 +295,9 @@ def add_postnorm_rmsnorm(resid: torch.Tensor, pending, weight, eps: float, out_d
     _check(resid, "resid", torch.float32)
     T, H = resid.shape
     post_w, post_eps, y = None, 0.0, pending
-    if isinstance(pending, PendingNormed):
+    if isinstance(pending, PendingNormed) and pending.bias is not None:
+        y = pending.materialize()                              # a layer norm: these kernels know the RMS norm only
+    elif isinstance(pending, PendingNormed):
         post_w, post_eps, y = pending.weight, pending.eps, pending.y
         _check(post_w, "post-norm weight", torch.float32)
         if post_w.numel() != H:
@@ -297,7 +339,7 @@ def softcap_(logits: torch.Tensor, cap: float) -> torch.Tensor:
 
 def latent_rope_cache(proj: torch.Tensor, kv_off: int, qa, cache, norm_w: torch.Tensor, eps: float,
                       freq: torch.Tensor, rot_dims: int, positions: torch.Tensor, slots, H: int, dn: int, dr: int,
-                      R: int, q_in_place: bool = False, interleaved: bool = False) -> None:
+                      R: int, q_in_place: bool = False, interleaved: bool = False, mult: float = 1.0) -> None:
     """Per token of ``proj`` [T, H (dn + dr) + R + dr] (queries per head as
     [dn plain | dr rotated], then at ``kv_off`` the compressed key/value vector
     [R | dr]): rotate every head's rotated part into ``qa`` [T, H, R + dr][:, :, R:],
@@ -305,7 +347,7 @@ def latent_rope_cache(proj: torch.Tensor, kv_off: int, qa, cache, norm_w: torch.
     part] into row ``slots[t]`` of ``cache`` [pages, page, R + dr] (``slots``
     None or a negative slot: no write).  Rotation: pairs (i, i + rot_dims / 2), or
     (2i, 2i + 1) with ``interleaved``, by position * ``freq[i]`` (64-bit
-    frequencies and angles, 32-bit rotation).  ``q_in_place``: the rotated parts also
+    frequencies and angles, 32-bit rotation), rotated numbers times ``mult``.  ``q_in_place``: the rotated parts also
     replace the unrotated ones in ``proj`` (``qa`` may then be None)."""
     _check(proj, "proj")
     if qa is None and not q_in_place:
@@ -332,8 +374,23 @@ def latent_rope_cache(proj: torch.Tensor, kv_off: int, qa, cache, norm_w: torch.
         _ptr(proj), c_int(proj.stride(0)), c_int(kv_off), _ptr(qa), _ptr(cache if slots is not None else None),
         c_int(_dtype_code(proj)), _ptr(norm_w), c_float(eps), _ptr(freq), c_int(rot_dims),
         c_int(1 if interleaved else 0), _ptr(positions),
-        _ptr(slots), c_int(T), c_int(H), c_int(dn), c_int(dr), c_int(R), c_int(1 if q_in_place else 0), _stream()),
-        "latent_rope_cache")
+        _ptr(slots), c_int(T), c_int(H), c_int(dn), c_int(dr), c_int(R), c_int(1 if q_in_place else 0),
+        c_float(mult), _stream()), "latent_rope_cache")
+
+
+def sigmoid_gate_(x: torch.Tensor, gate: torch.Tensor, n: int, stride: int | None = None) -> torch.Tensor:
+    """x <- x * sigmoid(gate), number by number, in place (32-bit, one rounding): ``gate`` [T, G n] view, of whose every n
+    numbers the first of ``x``'s every ``stride`` (default n) are the partners; x's other numbers stay as they are."""
+    _check(x, "x")
+    _check_rows(gate, "gate", x.dtype)
+    stride = n if stride is None else int(stride)
+    T = x.shape[0]
+    groups = x.shape[1] // stride
+    if stride < n or x.shape[1] != groups * stride or tuple(gate.shape) != (T, groups * n):
+        raise KernelError(f"sigmoid_gate: x {tuple(x.shape)}, gate {tuple(gate.shape)}, {n} of every {stride} numbers")
+    _ok(_fn("activation", "rg_sigmoid_gate")(_ptr(x), _ptr(gate), c_int(_dtype_code(x)), c_int(gate.stride(0)), c_int(T),
+                                             c_int(groups), c_int(n), c_int(stride), _stream()), "sigmoid_gate")
+    return x
 
 
 def latent_expand_context(cache: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
@@ -473,13 +530,17 @@ MOE_SCORINGS = {"softmax": 0, "sigmoid": 1}
 
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, correction, top: int, renormalize: bool = True,
-              scoring: str = "softmax"):
+              scoring: str = "softmax", groups=None, scale: float = 1.0, gate_row: torch.Tensor | None = None):
     """Router of a mixture of experts: softmax of the 32-bit logits ``router`` x
     over all N outputs (``scoring`` "sigmoid": the sigmoid of each logit
     instead); the ``top`` outputs with the largest score + correction
     (``correction`` None: the largest scores); weights = their scores over
-    their sum, or with ``renormalize`` False the scores themselves.  Returns
-    (ids int32 [T, top], weights float32 [T, top])."""
+    their sum, or with ``renormalize`` False the scores themselves, times
+    ``scale``.  ``groups`` = (count, keep): the outputs form that many equal
+    groups of neighbours and only those of the ``keep`` groups with the largest
+    best score can be chosen.  Returns (ids int32 [T, top], weights float32
+    [T, top]); with ``gate_row`` (float32 [W]) also sigmoid(gate_row . x),
+    float32 [T]."""
     _check(x, "x")
     _check(router, "router", torch.float32)
     if correction is not None:
@@ -490,12 +551,22 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction, top: int, renor
     N = router.shape[0]
     if router.shape[1] != W or (correction is not None and correction.numel() != N):
         raise KernelError(f"router {tuple(router.shape)} or its correction do not match rows of {W}")
+    count, keep = (int(groups[0]), int(groups[1])) if groups else (0, 0)
+    if groups and (count < 1 or N % count or not 1 <= keep <= count or top > keep * (N // count)):
+        raise KernelError(f"moe_route: {N} outputs, {count} groups of which {keep} are kept, {top} choices")
+    gate = None
+    if gate_row is not None:
+        _check(gate_row, "gate_row", torch.float32)
+        if gate_row.numel() != W:
+            raise KernelError(f"moe_route: a gate row of {gate_row.numel()} numbers for rows of {W}")
+        gate = torch.empty(T, dtype=torch.float32, device=x.device)
     ids = torch.empty((T, top), dtype=torch.int32, device=x.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=x.device)
     _ok(_fn("moe", "rg_moe_route")(_ptr(x), c_int(_dtype_code(x)), _ptr(router), _ptr(correction), _ptr(ids),
                                    _ptr(weights), c_int(T), c_int(W), c_int(N), c_int(top), c_int(1 if renormalize else 0),
-                                   c_int(MOE_SCORINGS[scoring]), _stream()), "moe_route")
-    return ids, weights
+                                   c_int(MOE_SCORINGS[scoring]), c_int(count), c_int(keep), c_float(scale),
+                                   _ptr(gate_row), _ptr(gate), _stream()), "moe_route")
+    return (ids, weights) if gate_row is None else (ids, weights, gate)
 
 
 def moe_align(ids: torch.Tensor, num_experts: int, tile_rows: int = MOE_TILE_ROWS):
@@ -628,10 +699,12 @@ def moe_scaled_rows(x: torch.Tensor, sorted_pair: torch.Tensor, top: int, weight
 
 
 def moe_combine(x: torch.Tensor, y, shared, ids: torch.Tensor, weights, pair_pos: torch.Tensor,
-                num_experts: int) -> torch.Tensor:
+                num_experts: int, shared_weight: torch.Tensor | None = None, all_experts: bool = False) -> torch.Tensor:
     """float32 [T, W] = sum over a token's choices of weight * (the expert's
     row of ``y``, or the token's own row of ``x`` for a choice with no expert
-    behind it), plus ``shared`` if given.  ``weights`` None: every weight is 1."""
+    behind it), plus ``shared`` if given, times ``shared_weight`` [T] (float32).
+    ``weights`` None: every weight is 1.  ``all_experts``: the caller knows that
+    every choice has an expert behind it."""
     _check(x, "x")
     T, W = x.shape
     top = ids.shape[1]
@@ -641,9 +714,14 @@ def moe_combine(x: torch.Tensor, y, shared, ids: torch.Tensor, weights, pair_pos
         _check(shared, "shared", x.dtype)
         if shared.shape != x.shape:
             raise KernelError(f"shared {tuple(shared.shape)} vs x {tuple(x.shape)}")
+    if shared_weight is not None:
+        _check(shared_weight, "shared_weight", torch.float32)
+        if shared_weight.numel() != T:
+            raise KernelError(f"shared_weight has {shared_weight.numel()} elements for {T} rows")
     out = torch.empty((T, W), dtype=torch.float32, device=x.device)
     _ok(_fn("moe", "rg_moe_combine")(_ptr(x), _ptr(y), _ptr(shared), c_int(_dtype_code(x)), _ptr(ids), _ptr(weights),
-                                     _ptr(pair_pos), _ptr(out), c_int(T), c_int(W), c_int(num_experts), c_int(top),
+                                     _ptr(pair_pos), _ptr(shared_weight), _ptr(out), c_int(T), c_int(W),
+                                     c_int(num_experts), c_int(top), c_int(1 if all_experts and y is not None else 0),
                                      _stream()), "moe_combine")
     return out
 
@@ -975,7 +1053,7 @@ SCAN_RULES = {"scalar": 0, "delta": 1, "channel": 2}
 def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, batch, H: int, d: int, dv: int,
                decay: torch.Tensor | None = None, g: torch.Tensor | None = None,
                beta: torch.Tensor | None = None, rule: str | None = None, skip: torch.Tensor | None = None,
-               w: torch.Tensor | None = None, bonus: torch.Tensor | None = None) -> torch.Tensor:
+               w: torch.Tensor | None = None, bonus: torch.Tensor | None = None, ones: bool = False) -> torch.Tensor:
     """A matrix S [d, dv] per head carried along each request's tokens, 32-bit, from the request's slot of ``state``
     [slots, H, dv, d] (S transposed; zeros at position 0) and left there.  ``rule``:
       "scalar"   S <- g S + beta k v^T, o = S^T q + skip_h v, with ``decay`` [H] or ``g`` [T, H], ``beta`` [T, H]
@@ -985,7 +1063,8 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
                  and ``bonus`` [H, d].
     By default "delta" when ``beta`` is given, else "scalar".
     ``q``, ``k``: float32 [T, Hqk * d] views (head h reads head h / (H / Hqk)); ``v``: [T, H * dv] view, float32 or
-    bfloat16.
+    bfloat16.  ``ones``: the last of the ``dv`` columns is that of a value that is always 1 and has no place in ``v``
+    [T, H * (dv - 1)] (its column of S is the sum of the keys with the same decays).
     Returns o [T, H, dv] float32."""
     rule = rule or ("delta" if beta is not None else "scalar")
     if rule not in SCAN_RULES:
@@ -996,7 +1075,7 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
     _check(state, "state", torch.float32)
     T = q.shape[0]
     Hqk = q.shape[1] // d
-    if q.shape[1] != Hqk * d or k.shape != q.shape or v.shape != (T, H * dv) or Hqk < 1 or H % Hqk \
+    if q.shape[1] != Hqk * d or k.shape != q.shape or v.shape != (T, H * (dv - int(ones))) or Hqk < 1 or H % Hqk \
             or tuple(state.shape[1:]) != (H, dv, d):
         raise KernelError(f"state_scan: q {tuple(q.shape)}, k {tuple(k.shape)}, v {tuple(v.shape)}, state "
                           f"{tuple(state.shape)} do not match {H} heads of {d} x {dv}")
@@ -1021,7 +1100,8 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.T
         _ptr(decay), _ptr(g),
         _ptr(beta), _ptr(skip), _ptr(w), c_int(w.stride(0) if w is not None else 0), _ptr(bonus),
         c_int(SCAN_RULES[rule]), _ptr(state), _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots),
-        _ptr(o), c_int(batch.num_requests), c_int(H), c_int(Hqk), c_int(d), c_int(dv), _stream()), "state_scan")
+        _ptr(o), c_int(batch.num_requests), c_int(H), c_int(Hqk), c_int(d), c_int(dv), c_int(1 if ones else 0), _stream()),
+        "state_scan")
     return o
 
 
@@ -1075,7 +1155,9 @@ def postnorm_shift(resid: torch.Tensor, pending, shift, state, batch, out_dtype)
     _check(resid, "resid", torch.float32)
     T, H = resid.shape
     post_w, post_eps, y = None, 0.0, pending
-    if isinstance(pending, PendingNormed):
+    if isinstance(pending, PendingNormed) and pending.bias is not None:
+        y = pending.materialize()                              # a layer norm: these kernels know the RMS norm only
+    elif isinstance(pending, PendingNormed):
         post_w, post_eps, y = pending.weight, pending.eps, pending.y
         _check(post_w, "post-norm weight", torch.float32)
         if post_w.numel() != H:
@@ -1180,10 +1262,104 @@ def ssd_chunk_scan(xbc: torch.Tensor, dt: torch.Tensor, A_log: torch.Tensor, D: 
     _COUNTER.value += 2                              # the launcher runs three kernels
     at = lambda col: c_void_p(xbc.data_ptr() + 4 * col)
     _ok(_fn("ssd_chunk", "rg_ssd_chunk_scan")(
-        at(0), at(inner), at(inner + G * N), c_int(xbc.stride(0)), _ptr(dt), _ptr(A_log), _ptr(D), _ptr(state),
+        at(0), at(inner), at(inner + G * N), c_int(xbc.stride(0)), _ptr(dt), _ptr(None), _ptr(A_log), _ptr(D), _ptr(state),
         _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(sums), _ptr(decays), _ptr(dots), _ptr(o),
-        c_int(T), c_int(R), c_int(H), c_int(G), c_int(N), c_int(dv), _stream()), "ssd_chunk_scan")
+        c_int(T), c_int(R), c_int(H), c_int(G), c_int(N), c_int(dv), c_int(0), _stream()), "ssd_chunk_scan")
     return o
+
+
+def pad_rows(weight: torch.Tensor, multiple: int = 8) -> torch.Tensor:
+    """The matrix with zero rows behind it up to a multiple of ``multiple``: the rows of its product then start on
+    16-byte boundaries."""
+    extra = -weight.shape[0] % multiple
+    if extra:
+        weight = torch.cat([weight, weight.new_zeros((extra, weight.shape[1]))], dim=0)
+    return weight.contiguous()
+
+
+def _mlstm_rows(proj, H: int, d: int, dv: int, ib, fb, state, m):
+    """Checks of what the mLSTM's operations share; the columns at which q, k, v, gate, i and f start in ``proj``'s rows."""
+    _check_rows(proj, "proj", torch.float32)
+    _check(m, "m", torch.float32)
+    for t, name in ((ib, "input gate bias"), (fb, "forget gate bias")):
+        _check(t, name, torch.float32)
+        if t.numel() != H:
+            raise KernelError(f"mlstm: {name} has {t.numel()} elements, expected {H}")
+    offs = (0, H * d, 2 * H * d, 2 * H * d + H * dv, 2 * H * (d + dv), 2 * H * (d + dv) + H)
+    if proj.shape[1] < offs[-1] + H or m.dim() != 2 or m.shape[1] != H:
+        raise KernelError(f"mlstm: rows {tuple(proj.shape)} or m {tuple(m.shape)} do not match {H} heads of {d} x {dv}")
+    if state is not None:
+        _check(state, "state", torch.float32)
+        if tuple(state.shape[1:]) != (H, dv + 1, d):
+            raise KernelError(f"mlstm: state {tuple(state.shape)} is not [slots, {H}, {dv + 1}, {d}]")
+    return offs
+
+
+def mlstm_scan(proj: torch.Tensor, ib: torch.Tensor, fb: torch.Tensor, cap: float, state: torch.Tensor, m: torch.Tensor,
+               batch, H: int, d: int, dv: int, chunked: bool | None = None):
+    """The mLSTM's recurrence over portions of prompts.  ``proj``: float32 rows [q (H d) | k (H d) | v (H dv) | gate (H dv) |
+    raw input gates (H) | raw forget gates (H) | ..]; ``ib``, ``fb`` [H]; ``state`` [slots, H, dv + 1, d] (S transposed, n
+    behind it) and ``m`` [slots, H] are carried on.  ``chunked``: in chunks of 64 tokens side by side, or token by token
+    (default: by the step's longest portion).  Returns (o [T, H, dv + 1] = S^T q and n . q, m [T, H])."""
+    q_off, k_off, v_off, g_off, i_off, f_off = _mlstm_rows(proj, H, d, dv, ib, fb, state, m)
+    T, R = proj.shape[0], batch.num_requests
+    if chunked is None:
+        chunked = batch.max_query_len >= SCAN_CHUNKED_MIN_TOKENS or d > 256
+    new = lambda *shape: torch.empty(shape, dtype=torch.float32, device=proj.device)
+    keep, put, m_rows = new(T, H), new(T, H), new(T, H)
+    _ok(_fn("mlstm", "rg_mlstm_gates")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(i_off), c_int(f_off), _ptr(ib), _ptr(fb), c_float(cap), _ptr(m),
+        _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(keep), _ptr(put), _ptr(m_rows), c_int(R),
+        c_int(H), c_int(1 if chunked else 0), _stream()), "mlstm_gates")
+    if not chunked:
+        o = state_scan(proj[:, :k_off], proj[:, k_off:v_off], proj[:, v_off:g_off], state, batch, H, d, dv + 1, g=keep,
+                       beta=put, rule="scalar", ones=True)
+        return o, m_rows
+    chunks = T // SCAN_CHUNK + R
+    sums, decays, dots = new(chunks, H, dv + 1, d), new(chunks, H), new(chunks, H, SCAN_CHUNK, SCAN_CHUNK)
+    o = new(T, H, dv + 1)
+    _COUNTER.value += 2                              # the launcher runs three kernels
+    at = lambda col: c_void_p(proj.data_ptr() + 4 * col)
+    _ok(_fn("ssd_chunk", "rg_ssd_chunk_scan")(
+        at(v_off), at(k_off), at(q_off), c_int(proj.stride(0)), _ptr(put), _ptr(keep), _ptr(None), _ptr(None), _ptr(state),
+        _ptr(batch.cu_seqlens), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(sums), _ptr(decays), _ptr(dots), _ptr(o),
+        c_int(T), c_int(R), c_int(H), c_int(H), c_int(d), c_int(dv), c_int(1), _stream()), "mlstm_chunk_scan")
+    return o, m_rows
+
+
+def mlstm_step(proj: torch.Tensor, ib: torch.Tensor, fb: torch.Tensor, cap: float, state: torch.Tensor, m: torch.Tensor,
+               batch, H: int, d: int, dv: int) -> torch.Tensor:
+    """``mlstm_scan`` for steps in which every request brings one token, in one kernel that leaves ``m`` as it was (the
+    output's kernel moves it on).  Returns o [T, H, dv + 1]."""
+    q_off, k_off, v_off, g_off, i_off, f_off = _mlstm_rows(proj, H, d, dv, ib, fb, state, m)
+    o = torch.empty((proj.shape[0], H, dv + 1), dtype=torch.float32, device=proj.device)
+    _ok(_fn("mlstm", "rg_mlstm_step")(
+        _ptr(proj), c_int(proj.stride(0)), c_int(q_off), c_int(k_off), c_int(v_off), c_int(i_off), c_int(f_off), _ptr(ib),
+        _ptr(fb), c_float(cap), _ptr(state), _ptr(m), _ptr(batch.req_of_token), _ptr(batch.start_pos),
+        _ptr(batch.state_slots), _ptr(o), c_int(proj.shape[0]), c_int(H), c_int(d), c_int(dv), _stream()), "mlstm_step")
+    return o
+
+
+def mlstm_out(o: torch.Tensor, proj: torch.Tensor, weight: torch.Tensor, eps: float, q_scale: float, m_rows, ib, fb, cap: float,
+              m: torch.Tensor, batch, H: int, d: int, dv: int, out_dtype) -> torch.Tensor:
+    """[T, H dv] in ``out_dtype``: x = q_scale S^T q / (max(|q_scale n . q|, exp(-m)) + 1e-6) from ``o`` [T, H, dv + 1],
+    every head divided by its root mean square, times ``weight`` [H dv], times the sigmoid of the rows' gate.  ``m_rows``
+    [T, H], or None after ``mlstm_step``: m is then worked out from the rows' raw gates and left in the requests' slots."""
+    q_off, k_off, v_off, g_off, i_off, f_off = _mlstm_rows(proj, H, d, dv, ib, fb, None, m)
+    _check(o, "o", torch.float32)
+    _check(weight, "weight", torch.float32)
+    T = proj.shape[0]
+    if tuple(o.shape) != (T, H, dv + 1) or weight.numel() != H * dv:
+        raise KernelError(f"mlstm_out: o {tuple(o.shape)} or weight {tuple(weight.shape)} does not match {H} heads of {dv}")
+    if m_rows is not None:
+        _check(m_rows, "m_rows", torch.float32)
+    out = torch.empty((T, H * dv), dtype=out_dtype, device=o.device)
+    _ok(_fn("mlstm", "rg_mlstm_out")(
+        _ptr(o), c_void_p(proj.data_ptr() + 4 * g_off), c_int(proj.stride(0)), _ptr(weight), c_float(eps), c_float(q_scale),
+        _ptr(m_rows), _ptr(proj), c_int(proj.stride(0)), c_int(i_off), c_int(f_off), _ptr(ib), _ptr(fb), c_float(cap), _ptr(m),
+        _ptr(batch.req_of_token), _ptr(batch.start_pos), _ptr(batch.state_slots), _ptr(out), c_int(_dtype_code(out)), c_int(T),
+        c_int(H), c_int(dv), _stream()), "mlstm_out")
+    return out
 
 
 def channel_chunk_scan(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, bonus: torch.Tensor,
@@ -1355,6 +1531,16 @@ def attention_prepare(qkv: torch.Tensor, kv_cache, q_norm, k_norm, eps: float, f
     return q
 
 
+def _reach(window, chunk: int, keep_first: int = 0) -> int:
+    """Which keys a query at position p sees, as the kernels take it: the last ``window`` positions up to p (0: all of
+    them), or with ``chunk`` those of its own chunk of that many positions, counted from position 0, up to p (a
+    negative number; without a window and kept first tokens)."""
+    window, chunk = int(window or 0), int(chunk or 0)
+    if window < 0 or chunk < 0 or (chunk and (window or keep_first)):
+        raise KernelError(f"a window ({window}) or chunks ({chunk}), not both, and no kept first tokens with chunks")
+    return -chunk if chunk else window
+
+
 def _pooled(pooled, kv_cache, window, keep_first):
     """Checks of the attention kernels' optional ``pooled`` = (entries, block table, pool): pages of the tokens' shape
     whose entry b stands for the positions b pool .. (b + 1) pool - 1 of a request, seen, beside the window, by the
@@ -1385,11 +1571,11 @@ def _sink_and_gate(sink, gate, nh: int, T: int, dtype):
     return gate.stride(0)
 
 
-ACTIVATIONS = {"relu2": 0, "relu": 1, "gelu_tanh": 2, "silu": 3}
+ACTIVATIONS = {"relu2": 0, "relu": 1, "gelu_tanh": 2, "silu": 3, "gelu": 4}
 
 
 def activation(x: torch.Tensor, kind: str, in_place: bool = True) -> torch.Tensor:
-    """Elementwise activation computed in 32-bit: relu2 (the square of relu), relu, gelu_tanh, silu."""
+    """Elementwise activation computed in 32-bit: relu2 (the square of relu), relu, gelu_tanh, silu, gelu (exact)."""
     _check(x, "x")
     if kind not in ACTIVATIONS:
         raise KernelError(f"unknown activation {kind!r}; known: {sorted(ACTIVATIONS)}")
@@ -1661,12 +1847,12 @@ def skinny_rope_ok(x, weight: torch.Tensor, d: int) -> bool:
 def paged_attention_general(q: torch.Tensor, q_stride: int, kv_cache: torch.Tensor, block_table: torch.Tensor,
                             req_of_token: torch.Tensor, positions: torch.Tensor, nh: int, nkv: int, d: int,
                             window: int, scale: float, keep_first: int = 0, sink=None, gate=None, pooled=None,
-                            out: torch.Tensor | None = None, out_scale: float = 1.0) -> torch.Tensor:
+                            out: torch.Tensor | None = None, out_scale: float = 1.0, chunk: int = 0) -> torch.Tensor:
     """The general attention kernel: out [T, nh*d].  ``q`` may be a view whose
     rows are ``q_stride`` elements apart (the q part of a fused qkv buffer).
     ``keep_first``: with a window, the first positions of a request that every
     later query still sees.  ``sink``, ``gate``: see ``_sink_and_gate``; ``pooled``: see ``_pooled``; ``out``: a view
-    to write into; the output is multiplied by ``out_scale``."""
+    to write into; the output is multiplied by ``out_scale``.  ``chunk``: see ``_reach``."""
     if not q.is_cuda:
         raise KernelError("q must be a CUDA tensor (there is no CPU path)")
     _check(kv_cache, "kv_cache", q.dtype)
@@ -1686,7 +1872,7 @@ def paged_attention_general(q: torch.Tensor, q_stride: int, kv_cache: torch.Tens
     _ok(_fn("attention_general", "rg_paged_attention_general")(
         _ptr(q), c_int(q_stride), _ptr(out), _ptr(kv_cache), c_int(_dtype_code(q)), _ptr(block_table),
         c_int(block_table.shape[1]), _ptr(req_of_token), _ptr(positions), c_int(T), c_int(nh), c_int(nkv),
-        c_int(d), c_int(page_size), c_int(window or 0), c_float(scale), c_int(keep_first if window else 0),
+        c_int(d), c_int(page_size), c_int(_reach(window, chunk, keep_first)), c_float(scale), c_int(keep_first if window else 0),
         _ptr(sink), _ptr(gate), c_int(gate_ld), *_pooled(pooled, kv_cache, window, keep_first), c_int(out.stride(0)),
         c_float(out_scale), _stream()),
         "paged_attention_general")
@@ -1710,13 +1896,14 @@ def _check_paged(q, kv_cache, block_table, nkv, d):
 
 def prefill_attention(q, q_stride: int, out, kv_cache, block_table, tiles, positions, nh: int, nkv: int, d: int,
                       window: int, scale: float, keep_first: int = 0, sink=None, gate=None, pooled=None,
-                      out_scale: float = 1.0) -> None:
+                      out_scale: float = 1.0, chunk: int = 0) -> None:
     """Flash-style attention for requests that bring several tokens: ``tiles``
     [n, 3] = (first row, rows <= 64, request index).  Writes the tiles' rows of
     ``out`` [T, nh*d].  ``keep_first``: with a window, the first positions of a
     request that every later query still sees.  ``sink``, ``gate``: see
     ``_sink_and_gate``; ``pooled``: see ``_pooled``.  ``out`` may be a view
-    whose rows are further apart; the output is multiplied by ``out_scale``."""
+    whose rows are further apart; the output is multiplied by ``out_scale``.
+    ``chunk``: see ``_reach``."""
     page_size = _check_paged(q, kv_cache, block_table, nkv, d)
     _check(tiles, "tiles", torch.int32)
     _check(positions, "positions", torch.int32)
@@ -1725,7 +1912,7 @@ def prefill_attention(q, q_stride: int, out, kv_cache, block_table, tiles, posit
     _ok(_fn("attention_mma", "rg_prefill_attention_sink")(
         _ptr(q), c_int(q_stride), _ptr(out), _ptr(kv_cache), _ptr(block_table), c_int(block_table.shape[1]),
         _ptr(tiles), c_int(tiles.shape[0]), _ptr(positions), c_int(nh), c_int(nkv), c_int(d), c_int(page_size),
-        c_int(window or 0), c_int(keep_first if window else 0), c_float(scale), _ptr(sink), _ptr(gate), c_int(gate_ld),
+        c_int(_reach(window, chunk, keep_first)), c_int(keep_first if window else 0), c_float(scale), _ptr(sink), _ptr(gate), c_int(gate_ld),
         *_pooled(pooled, kv_cache, window, keep_first), c_int(out.stride(0)), c_float(out_scale), _stream()),
         "prefill_attention")
 
@@ -1746,7 +1933,7 @@ _decode_counters: dict = {}
 def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_tokens: int, req_of_token, positions,
                      nh: int, nkv: int, d: int, window: int, scale: float, num_splits: int,
                      scratch=None, fused_reduce=None, cluster: bool = False, keep_first: int = 0, sink=None,
-                     gate=None, pooled=None, out_scale: float = 1.0) -> None:
+                     gate=None, pooled=None, out_scale: float = 1.0, chunk: int = 0) -> None:
     """Split attention for single tokens: token rows ``rows`` (None: rows
     0..n_tokens-1) each attend their request's context.  Partial results go
     through scratch memory (allocated here unless given) and are reduced into
@@ -1763,7 +1950,7 @@ def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_token
     ``_sink_and_gate``; they enter where the splits are added up (not with
     ``cluster``).  ``pooled``: see ``_pooled`` (not with ``cluster``).  ``out``
     may be a view whose rows are further apart; the output is multiplied by
-    ``out_scale`` (neither with ``cluster``)."""
+    ``out_scale`` (neither with ``cluster``).  ``chunk``: see ``_reach``."""
     if fused_reduce is None:
         fused_reduce = num_splits == 1
     page_size = _check_paged(q, kv_cache, block_table, nkv, d)
@@ -1783,7 +1970,7 @@ def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_token
         _ok(_fn("attention_mma", "rg_decode_attention_cluster")(
             _ptr(q), c_int(q_stride), _ptr(out), _ptr(kv_cache), _ptr(block_table), c_int(block_table.shape[1]),
             _ptr(rows), c_int(n_tokens), _ptr(req_of_token), _ptr(positions), c_int(nh), c_int(nkv), c_int(d),
-            c_int(page_size), c_int(window or 0), c_float(scale), c_int(num_splits), _stream()), "decode_attention")
+            c_int(page_size), c_int(_reach(window, chunk)), c_float(scale), c_int(num_splits), _stream()), "decode_attention")
         return
     if scratch is None:
         part_o = torch.empty((n_tokens, nh, num_splits, d), dtype=torch.float32, device=q.device)
@@ -1804,7 +1991,7 @@ def decode_attention(q, q_stride: int, out, kv_cache, block_table, rows, n_token
     _ok(_fn("attention_mma", "rg_decode_attention_sink")(
         _ptr(q), c_int(q_stride), _ptr(out), _ptr(kv_cache), _ptr(block_table), c_int(block_table.shape[1]),
         _ptr(rows), c_int(n_tokens), _ptr(req_of_token), _ptr(positions), _ptr(part_o), _ptr(part_ml),
-        _ptr(counters), c_int(nh), c_int(nkv), c_int(d), c_int(page_size), c_int(window or 0),
+        _ptr(counters), c_int(nh), c_int(nkv), c_int(d), c_int(page_size), c_int(_reach(window, chunk, keep_first)),
         c_int(keep_first if window else 0), c_float(scale), c_int(num_splits), _ptr(sink), _ptr(gate), c_int(gate_ld),
         *_pooled(pooled, kv_cache, window, keep_first), c_int(out.stride(0)), c_float(out_scale), _stream()),
         "decode_attention")

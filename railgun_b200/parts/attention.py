@@ -160,10 +160,13 @@ class NormedAttention(Mixer):
     32-bit, before its one rounding; the sink and the gate are applied where the attention kernels divide by
     the denominator.
 
+    Instead of a window, ``chunk``: a query sees the keys of its own chunk of that many positions, counted from the
+    request's first token, up to its own (the pages of complete chunks are given back).
+
     params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``, ``v_dim``, ``scale`` (None:
     head_dim^-1/2), ``rot_dims``, ``rot_base``, ``rot_layout`` ("interleaved": pairs (2i, 2i + 1), or "half":
     pairs (i, i + rot_dims/2)), ``rot_factor`` (what the frequencies are divided by, default 1), ``eps`` (of the q and
-    k norms), ``window`` (0: none), ``keep_first``, ``pool`` (0: none),
+    k norms), ``window`` (0: none), ``keep_first``, ``pool`` (0: none), ``chunk`` (0: none),
     ``bias`` (true, the default; "qkv": not on the output; false), ``bias_in`` (where the bias of q, k and v is added:
     "product", the default, or "rows": by the per-token kernel behind it, in 32-bit, which leaves the product to the
     kernels that have no bias; not with a convolution), ``head_temp`` (default true), ``qk_norm`` (true, the
@@ -225,7 +228,7 @@ class NormedAttention(Mixer):
         pool = int(p.get("pool") or 0) if window else 0
         # pages: the tokens'; with pooled blocks a token stays until its block is complete, also behind the window
         needs = [PagedKVNeed(int(p["num_kv_heads"]), cls._padded(p), max(window, pool),
-                             keep_first=int(p.get("keep_first") or 0) if window else 0)]
+                             keep_first=int(p.get("keep_first") or 0) if window else 0, chunk=int(p.get("chunk") or 0))]
         if pool:
             needs.append(PagedKVNeed(int(p["num_kv_heads"]), cls._padded(p), tokens_per_entry=pool))
         K = cls._taps(p)
@@ -256,6 +259,9 @@ class NormedAttention(Mixer):
         self.pool = int(p.get("pool") or 0) if self.window else 0
         if self.pool and self.keep_first:
             raise ValueError("a window keeps first tokens or sees pooled blocks, not both")
+        self.chunk = int(p.get("chunk") or 0)
+        if self.chunk and self.window:
+            raise ValueError("attention has a window or chunks, not both")
         self.eps = float(p.get("eps") or 0.0)
         scale = float(p["scale"]) if p.get("scale") is not None else float(self.d) ** -0.5
         b = self._base(p, prefix)
@@ -372,7 +378,7 @@ class NormedAttention(Mixer):
         and the gate); the 32-bit path runs the general kernel."""
         H, G, D = self.H, self.G, self.D
         table = batch.block_table[cache.group]
-        more = dict(sink=self.sink, gate=gate, pooled=pooled, out_scale=out_scale)
+        more = dict(sink=self.sink, gate=gate, pooled=pooled, out_scale=out_scale, chunk=self.chunk)
         if q.dtype != torch.bfloat16:
             return ops.paged_attention_general(q, q.shape[1], cache.kv, table, batch.req_of_token, batch.positions,
                                                H, G, D, self.window, 1.0, self.keep_first, out=out, **more)
@@ -382,6 +388,8 @@ class NormedAttention(Mixer):
         reach = batch.max_context_len
         if self.window:
             reach = min(reach, self.window + self.keep_first + (reach // self.pool if self.pool else 0))
+        if self.chunk:
+            reach = min(reach, self.chunk)
         if batch.num_prefill_tiles:
             ops.prefill_attention(q, q.shape[1], out, cache.kv, table, batch.prefill_tiles, batch.positions,
                                   H, G, D, self.window, 1.0, self.keep_first, **more)

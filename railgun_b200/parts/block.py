@@ -68,7 +68,7 @@ class Sandwich(Arrangement):
                 raise ValueError("the 'sandwich' arrangement needs a post_norm on every branch")
             h = normed_input(b.norm, b.part, stream)
             y = b.part.forward(h, batch, cache, writes) if b.role == "mixer" else b.part.forward(h, batch)
-            stream.pending = ops.PendingNormed(y, b.post_norm.weight, b.post_norm.eps)
+            stream.pending = ops.PendingNormed(y, b.post_norm.weight, b.post_norm.eps, getattr(b.post_norm, "bias", None))
 
 
 class PostNorm(Arrangement):
@@ -81,7 +81,7 @@ class PostNorm(Arrangement):
             else:
                 h = normed_input(b.norm, b.part, stream)
                 y = b.part.forward(h, batch, cache, writes) if b.role == "mixer" else b.part.forward(h, batch)
-            stream.pending = ops.PendingNormed(y, b.post_norm.weight, b.post_norm.eps)
+            stream.pending = ops.PendingNormed(y, b.post_norm.weight, b.post_norm.eps, getattr(b.post_norm, "bias", None))
 
 
 class ParallelResidual(Arrangement):

@@ -20,6 +20,7 @@ from . import mlp as _mlp, norm as _norm, rope as _rope  # noqa: F401
 from . import latent_attention as _latent_attention, moe as _moe  # noqa: F401
 from . import talking_attention as _talking_attention, recurrent as _recurrent, parallel as _parallel  # noqa: F401
 from . import state_mixers as _state_mixers, mamba2 as _mamba2, time_mixing as _time_mixing  # noqa: F401
+from . import mlstm as _mlstm  # noqa: F401
 
 
 def _part_registry(role: str):

@@ -7,8 +7,10 @@ weights are the scores themselves over their sum.  The first ``experts``
 outputs stand for gated feed-forwards down(silu(gate h) * (up h)), the
 ``identity`` outputs after them for experts that return their input.  An
 optional shared expert of the same form runs for every token and is added.
-Experts without a gate, down(act(up h)), and experts whose weight multiplies
-their input instead of their output, sum_e expert_e(w_e h), are options.
+Experts without a gate, down(act(up h)), experts whose weight multiplies
+their input instead of their output, sum_e expert_e(w_e h), a choice limited
+to the experts of the best groups, a constant on the weights and a sigmoid
+gate on the shared expert are options.
 
 The experts' matrices are stacked at load ([E, 2F, W] gate rows then up rows,
 [E, W, F]); the step groups its (token, choice) pairs by expert on the device
@@ -22,7 +24,7 @@ import torch
 from .. import ops
 from ..weights.loader import TensorSpec
 from .base import FeedForward
-from .mlp import SwiGLU
+from .mlp import DenseMLP, SwiGLU
 from .registry import register_feed_forward
 
 
@@ -37,7 +39,11 @@ class RoutedExperts(FeedForward):
     "gelu_tanh" or "clamped_swish" with ``limit``: g' sigmoid(1.702 g') (u' + 1),
     g' = min(g, limit), u' = clamp(u, -limit, limit)), ``scoring`` "sigmoid"
     (default "softmax"), ``gated`` False (experts ``<base>e<i>.up|down`` without a
-    gate; ``activation`` is then one of ``ops.ACTIVATIONS``, e.g. "relu2"),
+    gate, and a shared expert of that form; ``activation`` is then one of ``ops.ACTIVATIONS``, e.g. "relu2" or
+    "gelu"), ``groups`` (count, keep): the experts form that many equal groups of neighbours and only those of the
+    ``keep`` groups with the largest best score can be chosen; ``weight_scale``: a constant on the chosen experts'
+    weights; ``shared_gate`` True: the shared expert's output is multiplied by sigmoid(<base>shared.sg h), one number
+    per token (32-bit, computed beside the router's logits);
     ``scale_input`` True (a chosen expert reads its weight times the token's row,
     and the experts' outputs are added as they are; not with identity or shared
     experts)."""
@@ -55,12 +61,21 @@ class RoutedExperts(FeedForward):
             out[f"{b}e{e}.up"] = TensorSpec((F, W))
             out[f"{b}e{e}.down"] = TensorSpec((W, F))
         if p.get("shared_size"):
-            out.update(SwiGLU.tensor_specs(cls._shared_params(p), prefix))
+            out.update(cls._shared_kind(p).tensor_specs(cls._shared_params(p), prefix))
+            if p.get("shared_gate"):
+                out[b + "shared.sg"] = TensorSpec((1, W))
         return out
+
+    @staticmethod
+    def _shared_kind(p):
+        return SwiGLU if p.get("gated", True) else DenseMLP
 
     @staticmethod
     def _shared_params(p):
         b = p.get("base", "mlp.")
+        if not p.get("gated", True):
+            return dict(hidden_size=p["hidden_size"], intermediate_size=p["shared_size"],
+                        activation=p.get("activation") or "silu", names=(b + "shared.up", b + "shared.down"))
         return dict(hidden_size=p["hidden_size"], intermediate_size=p["shared_size"],
                     names=(b + "shared.gate", b + "shared.up", b + "shared.down"))
 
@@ -79,6 +94,12 @@ class RoutedExperts(FeedForward):
         self.gated = bool(p.get("gated", True))
         self.scoring = p.get("scoring") or "softmax"
         self.scale_input = bool(p.get("scale_input", False))
+        self.groups = tuple(int(x) for x in p["groups"]) if p.get("groups") else None
+        if self.groups:
+            count, keep = self.groups
+            if count < 1 or self.N % count or not 1 <= keep <= count or self.top > keep * (self.N // count):
+                raise ValueError(f"{self.N} router outputs in {count} groups of which {keep} are kept, {self.top} choices")
+        self.weight_scale = float(p["weight_scale"]) if p.get("weight_scale") is not None else 1.0
         if self.scoring not in ops.MOE_SCORINGS:
             raise ValueError(f"router scoring {self.scoring!r} is not known; known: {sorted(ops.MOE_SCORINGS)}")
         known = ops.GATED_ACTIVATIONS if self.gated else ops.ACTIVATIONS
@@ -96,11 +117,16 @@ class RoutedExperts(FeedForward):
                                           for e in range(self.E)]).contiguous()                    # [E, 2F, W]
             self.w_down = torch.stack([tensors.get(f"{b}e{e}.down", env.dtype) for e in range(self.E)]).contiguous()
             tensors.drop(*[f"{b}e{e}.{n}" for e in range(self.E) for n in ("gate", "up", "down")])
-        self.shared = SwiGLU(self._shared_params(p), prefix, env, tensors) if p.get("shared_size") else None
+        self.shared = self.shared_gate = None
+        if p.get("shared_size"):
+            self.shared = self._shared_kind(p)(self._shared_params(p), prefix, env, tensors)
+            if p.get("shared_gate"):
+                self.shared_gate = tensors.get(b + "shared.sg", torch.float32).reshape(-1).contiguous()
 
     def forward(self, x, batch):
         T = x.shape[0]
-        ids, weights = ops.moe_route(x, self.router, self.correction, self.top, self.renormalize, self.scoring)
+        ids, weights, *gate = ops.moe_route(x, self.router, self.correction, self.top, self.renormalize, self.scoring,
+                                            groups=self.groups, scale=self.weight_scale, gate_row=self.shared_gate)
         y = pair_pos = None
         if self.E:
             places = T * self.top
@@ -123,7 +149,8 @@ class RoutedExperts(FeedForward):
         else:
             pair_pos = ids
         shared = self.shared.forward(x, batch) if self.shared is not None else None
-        return ops.moe_combine(x, y, shared, ids, weights, pair_pos, self.E)
+        return ops.moe_combine(x, y, shared, ids, weights, pair_pos, self.E, shared_weight=gate[0] if gate else None,
+                               all_experts=self.N == self.E)
 
 
 register_feed_forward("routed_experts", RoutedExperts)

@@ -4,6 +4,8 @@ y = w * r / sqrt(mean(r^2) + eps), r = residual (+ pending), all in 32-bit
 with one rounding at the end.  The reference builds the norm with
 candle_nn::rms_norm(H, eps) (crates/vllm-models/src/llama/architecture.rs:27-28,108)
 and adds residuals with separate ops (:53,58).
+
+"layernorm": the same with the mean taken off first and a bias.
 """
 from __future__ import annotations
 
@@ -56,6 +58,8 @@ class RMSNorm(Norm):
                 pending = pending.materialize()
             return ops.add_group_rmsnorm(resid, pending, [self.weight], self.groups, self.eps, self.env.dtype, rows)[0]
         if isinstance(pending, ops.PendingNormed):
+            if pending.bias is not None:
+                return ops.stream_norm(resid, pending, (self.weight, None, self.eps), self.env.dtype, rows)
             return ops.add_postnorm_rmsnorm(resid, pending, self.weight, self.eps, self.env.dtype, rows)
         if isinstance(pending, ops.PendingLinear):
             # small decode batches: the product adds its result to the residual itself and prepares this
@@ -68,16 +72,45 @@ class RMSNorm(Norm):
         return ops.add_rmsnorm(resid, pending, self.weight, self.eps, self.env.dtype, rows)
 
 
+class LayerNorm(Norm):
+    """w (r - mean(r)) / sqrt(mean((r - mean(r))^2) + eps) + b, all in 32-bit with one rounding at the end.  params:
+    ``size``, ``eps``, ``name`` (weight tensor name after the prefix), ``bias_name`` (default: the weight's with ".b"
+    behind it)."""
+
+    @classmethod
+    def _bias_name(cls, params):
+        return params.get("bias_name") or params["name"] + ".b"
+
+    @classmethod
+    def tensor_specs(cls, params, prefix):
+        size = (params["size"],)
+        return {prefix + params["name"]: TensorSpec(size, init="norm"), prefix + cls._bias_name(params): TensorSpec(size)}
+
+    def __init__(self, params, prefix, env, tensors):
+        super().__init__(params, prefix, env, tensors)
+        self.eps = float(params["eps"])
+        self.weight = tensors.get(prefix + params["name"], torch.float32).contiguous()
+        self.bias = tensors.get(prefix + self._bias_name(params), torch.float32).contiguous()
+
+    fuses_post_norm = True
+
+    def add_norm(self, resid, pending, rows=None):
+        return ops.stream_norm(resid, pending, (self.weight, self.bias, self.eps), self.env.dtype, rows)
+
+
 class Identity(Norm):
     """No norm: the part behind it reads the stream itself, in the activation type.  No parameters."""
 
     fuses_post_norm = True
 
     def add_norm(self, resid, pending, rows=None):
+        if isinstance(pending, ops.PendingNormed) and pending.bias is not None:
+            return ops.stream_norm(resid, pending, None, self.env.dtype, rows)
         if rows is not None:
             return ops.add_postnorm_rmsnorm(resid, pending, None, 0.0, self.env.dtype, rows)
         return ops.postnorm_shift(resid, pending, None, None, None, self.env.dtype)[1]
 
 
 register_norm("rmsnorm", RMSNorm)
+register_norm("layernorm", LayerNorm)
 register_norm("identity", Identity)
