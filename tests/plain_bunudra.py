@@ -143,13 +143,13 @@ def mlstm_scan(q, k, v, i, f, state=None):
         S, n, m = (x.copy() for x in state)
     o = np.zeros((T, H, v.shape[2]))
     for t in range(T):
-        for h in range(H):
-            new = max(f[t, h] + m[h], i[t, h])
-            keep, put = math.exp(f[t, h] + m[h] - new), math.exp(i[t, h] - new)
-            S[h] = keep * S[h] + put * np.outer(k[t, h], v[t, h])
-            n[h] = keep * n[h] + put * k[t, h]
-            m[h] = new
-            o[t, h] = S[h].T @ q[t, h] / (max(abs(n[h] @ q[t, h]), math.exp(-new)) + 1e-6)
+        new = np.maximum(f[t] + m, i[t])
+        keep, put = np.exp(f[t] + m - new), np.exp(i[t] - new)
+        S = keep[:, None, None] * S + put[:, None, None] * k[t][:, :, None] * v[t][:, None, :]
+        n = keep[:, None] * n + put[:, None] * k[t]
+        m = new
+        top = np.einsum("hij,hi->hj", S, q[t])
+        o[t] = top / (np.maximum(np.abs(np.sum(n * q[t], axis=1)), np.exp(-m)) + 1e-6)[:, None]
     return o, (S, n, m)
 
 
@@ -215,9 +215,23 @@ def small_ff(h, w, p):
     return gelu(h @ w[p + "up"].T) @ w[p + "down"].T
 
 
-def experts_ff(h, w, p, m):
+def routing_margin(z, top, groups):
+    """By how much the logits z [N] of one token would have to move for another choice: the smaller of the gaps between
+    the last group kept and the best one that is not, and between the last expert chosen and the best one that is not."""
+    gap = np.inf
+    if groups:
+        best = np.sort(z.reshape(groups["count"], -1).max(axis=1))[::-1]
+        if groups["keep"] < groups["count"]:
+            gap = best[groups["keep"] - 1] - best[groups["keep"]]
+    allowed = np.sort(z[choose_experts(z, len(z) if not groups else len(z) // groups["count"] * groups["keep"], groups)])[::-1]
+    return min(gap, allowed[top - 1] - allowed[top]) if top < len(allowed) else gap
+
+
+def experts_ff(h, w, p, m, margins=None):
     r = m["router"]
     z = h @ w[p + "router"].T
+    if margins is not None:
+        margins.append(np.array([routing_margin(row, r["top"], r.get("groups")) for row in z]))
     e = np.exp(z - z.max(axis=1, keepdims=True))
     s = e / e.sum(axis=1, keepdims=True)
     out = np.zeros_like(h)
@@ -230,7 +244,7 @@ def experts_ff(h, w, p, m):
 
 
 # ---- the model -------------------------------------------------------------------------------------------
-def layer_forward(x, w, cfg, i, pos):
+def layer_forward(x, w, cfg, i, pos, margins=None):
     """x <- x + norm1(mixer(x)); x <- x + norm2(ff(x))."""
     L = cfg["layers"][i]
     eps = cfg["norm"]["eps"]
@@ -238,18 +252,19 @@ def layer_forward(x, w, cfg, i, pos):
     norm = lambda y, name: layer_norm(y, w[p + name], w[p + name + ".b"], eps)
     x = x + norm(MIXERS[L["type"]](x, w, p + "mix.", L["mixer"], pos, eps), "norm1")
     if L.get("mlp") is not None:
-        x = x + norm(experts_ff(x, w, p + "mlp.", L["mlp"]), "norm2")
+        x = x + norm(experts_ff(x, w, p + "mlp.", L["mlp"], margins), "norm2")
     return x
 
 
-def forward(tokens, w, cfg, return_layers=False):
-    """Logits [T, vocab] of one sequence from position 0 (and the stream after every layer)."""
+def forward(tokens, w, cfg, return_layers=False, margins=None):
+    """Logits [T, vocab] of one sequence from position 0 (and the stream after every layer).  ``margins`` (a list)
+    receives one array [T] per layer with experts: the routers' margins."""
     tokens = np.asarray(tokens)
     pos = np.arange(len(tokens))
     x = w["embed"][tokens] * cfg["embedding"]["scale"]
     layers = []
     for i in range(len(cfg["layers"])):
-        x = layer_forward(x, w, cfg, i, pos)
+        x = layer_forward(x, w, cfg, i, pos, margins)
         layers.append(x)
     logits = layer_norm(x, w["final.norm"], w["final.norm.b"], cfg["norm"]["eps"]) @ w["head"].T
     return (logits, np.stack(layers)) if return_layers else logits
