@@ -97,8 +97,20 @@ CASE_E = dict(
             layer(latent(2, 12, 0, 10, 9, 5), experts(5, 3, 14, (5, 4), 1.4, 22)),
             layer(memory(3, 10, 7, 6.0), experts(4, 2, 18, (2, 2), 0.9, 30))])
 
+
+def with_all_experts(cfg):
+    """The same with every expert chosen: no choice that rounding can turn."""
+    cfg = json.loads(json.dumps(cfg))
+    for L in cfg["layers"]:
+        if L["mlp"]:
+            L["mlp"]["router"]["top"] = L["mlp"]["router"]["experts"]
+            L["mlp"]["router"].pop("groups", None)
+    return cfg
+
+
 CASES = {"A": (CASE_A, 3, 8), "B": (CASE_B, 5, 16), "C": (CASE_C, 7, 32), "D": (CASE_D, 9, 16),
          "E": (CASE_E, 11, 4)}                                                                # config, seed, page
+CASES.update({n + "-all": (with_all_experts(CASES[n][0]), *CASES[n][1:]) for n in "ACD"})
 
 _made: dict = {}
 _plain: dict = {}
@@ -174,12 +186,6 @@ class Plain:
 
     def forward(self, ids):
         return self.P.forward(ids, self.w, self.cfg)
-
-    def forward_with_margins(self, ids):
-        """(logits, per position the smallest router margin of any layer; inf without experts)."""
-        m = []
-        logits = self.P.forward(ids, self.w, self.cfg, margins=m)
-        return logits, (np.min(np.stack(m), axis=0) if m else np.full(len(ids), np.inf))
 
     def greedy(self, prompt, n):
         ids = list(prompt)

@@ -22,11 +22,12 @@ DTYPES = ["float32", "bfloat16"]
 TORCH = {"float32": torch.float32, "bfloat16": torch.bfloat16}
 # bfloat16: the test weights are several times larger than a trained model's, so rounding alone moves logits by some
 # 1e-2 of the largest, the same in every cut; a lost key, state or expert is caught by the tests of the mechanisms
-# alone, where it changes a row by its whole size.  Where a router's choice is a close call, rounding may choose
-# another expert: those positions are held to LOOSE only, and so may be a few that come after them in their request.
+# alone, where it changes a row by its whole size.  Where a router's choice is a close call, rounding may choose another
+# expert, and the tokens after it, which read what it left in memories and windows, differ as well: where experts are
+# chosen, one position in seven may be over the tolerance, up to LOOSE.  In the "-all" cases every expert is chosen and
+# every position is held.
 TOL = {"float32": 5e-5, "bfloat16": 6e-2}
 LOOSE = 1.5
-CLOSE_CALL = 0.06                                   # of router logits, in bfloat16
 
 
 def rel(got, ref):
@@ -37,7 +38,7 @@ def rel(got, ref):
 
 def dev(x, dtype=None):
     t = torch.as_tensor(x)
-    return t.to(DEV, dtype=dtype) if dtype is not None else t.to(DEV)
+    return (t.to(DEV, dtype=dtype) if dtype is not None else t.to(DEV)).contiguous()
 
 
 def step_batch(lengths, starts, slots):
@@ -66,8 +67,8 @@ def test_layer_norms_alone(T, W, dtype):
     from railgun_b200 import ops
     rng = np.random.default_rng(W)
     x = torch.tensor(rng.normal(size=(T, W)), dtype=torch.float32)
-    y = torch.tensor(rng.normal(size=(T, W)) * rng.choice([0.01, 30.0], size=(T, 1))
-                     + (rng.choice([0.0, 3000.0], size=(T, 1)) if dtype == "float32" else 0.0), dtype=TORCH[dtype])
+    y = torch.tensor((rng.normal(size=(T, W)) + rng.choice([0.0, 30.0], size=(T, 1))) * rng.choice([0.01, 30.0], size=(T, 1)),
+                     dtype=TORCH[dtype])
     w, b, w2, b2 = (rng.normal(size=W) + 1.0 for _ in range(4))
     f = lambda a: dev(a, torch.float32)
     tol = 3e-5 if dtype == "float32" else 5e-3
@@ -144,6 +145,7 @@ def test_memory_over_portions(form, H, d, dv, cap):
     at = lengths[0]
     far, ask = at + 5, at + lengths[1] - 1
     rows[far, H * d:H * d + d], rows[ask, :d] = 2.0, 2.0
+    rows[far, 2 * H * (d + dv)] = 2.0 * cap                                    # head 0's input gate
     ib, fb = rng.uniform(-1, 1, size=H), rng.uniform(0, 2, size=H)
     weight, eps, q_scale = rng.uniform(0.5, 2, size=H * dv), 1e-5, d ** -0.5
     S0, n0, m0 = rng.normal(size=(5, H, d, dv)) * 0.3, rng.normal(size=(5, H, d)) * 0.3, rng.uniform(0, 2, size=(5, H))
@@ -304,7 +306,7 @@ def test_gelu_and_the_gate_on_heads_alone(dtype):
     for T, H, dv, stride in ((5, 3, 12, 12), (70, 2, 16, 48), (2, 4, 7, 9), (300, 8, 64, 64)):
         x = torch.tensor(rng.normal(size=(T, H * stride)), dtype=TORCH[dtype])
         wide = torch.tensor(rng.normal(size=(T, H * dv + 13)) * 3.0, dtype=TORCH[dtype])
-        got = ops.sigmoid_gate_(dev(x), dev(wide)[:, 5:5 + H * dv], dv, stride).cpu().view(T, H, stride)
+        got = ops.sigmoid_gate_(dev(x), wide.to(DEV)[:, 5:5 + H * dv], dv, stride).cpu().view(T, H, stride)
         ref = x.double().numpy().reshape(T, H, stride)[..., :dv] * P.sigmoid(wide.double().numpy()[:, 5:5 + H * dv]).reshape(T, H, dv)
         assert rel(got[..., :dv], ref) < tol and torch.equal(got[..., dv:], x.view(T, H, stride)[..., dv:])
 
@@ -470,7 +472,7 @@ def test_attention_mixers_alone_at_the_edges(name, layer, dtype):
         moved = json.loads(json.dumps(m))
         moved["mask"]["size"] = size + (1 if L["type"] == "latent_attention" else T)
         other = P.MIXERS[L["type"]](h.double().numpy(), plain.w, f"l{layer}.mix.", moved, np.arange(T), cfg["norm"]["eps"])
-        shows += key == first - 1 and rel(other[-1], ref[-1]) > 0.2
+        shows += key == first - 1 and rel(other[-1], ref[-1]) > 0.03
         tol = 5e-5 if dtype == "float32" else 4e-2
         for cuts in ((), (max(1, key), key + 1, T - 3, T - 2, T - 1), (page + 3, 2 * page + 5, T - 1), (2, 4, T - 5), (T - 70,)):
             got = feed_mixer(runner, layer, dev(h), cuts)
@@ -485,7 +487,8 @@ def test_prompts_take_the_expanded_form_where_it_fits():
     from railgun_b200.engine.runner import ModelRunner
     runner = ModelRunner(C.model_dir("D"), dtype="bfloat16", page_size=16, max_tokens=512, max_requests=2)
     assert runner.model.layers[1].mixer.expands_prompts and not runner.model.layers[3].mixer.expands_prompts
-    assert not ModelRunner(C.model_dir("D"), dtype="float32", page_size=16, max_tokens=512, max_requests=2).model.layers[1].mixer.expands_prompts
+    whole = ModelRunner(C.model_dir("D"), dtype="float32", page_size=16, max_tokens=512, max_requests=2)
+    assert not whole.model.layers[1].mixer.expands_prompts
 
 
 # ---- the model through the step function ---------------------------------------------------------------
@@ -496,37 +499,34 @@ PORTIONS = {"D": (130, 2, 64, 7, 128, 3, 65, 2, 33, 129)}
 MIXED = {"D": (5, 1, 2, 70, 1, 1, 3, 140, 1, 2, 128, 17)}
 TAIL = {"D": 140, "B": 60}
 _oracle: dict = {}
-_margins: dict = {}
 
 
 def oracle(name):
     if name not in _oracle:
         cfg = C.CASES[name][0]
-        reqs = {f"r{i}": p for i, p in enumerate(C.prompts(cfg["vocab"], LENGTHS[name], seed=21))}
+        reqs = {f"r{i}": p for i, p in enumerate(C.prompts(cfg["vocab"], LENGTHS[name[0]], seed=21))}
         plain = C.plain_model(name)
-        both = {k: plain.forward_with_margins(v) for k, v in reqs.items()}
-        _oracle[name] = (reqs, {k: v[0] for k, v in both.items()})
-        _margins[name] = {k: v[1] for k, v in both.items()}
+        _oracle[name] = (reqs, {k: plain.forward(v) for k, v in reqs.items()})
     return _oracle[name]
 
 
-def margins_of(name, dtype):
-    return _margins[name] if dtype == "bfloat16" else None
+def chosen(name, dtype):
+    return dtype == "bfloat16" and not name.endswith("-all")
 
 
 def make_trace(mode, reqs, name):
     if mode == "whole":
         return helpers.trace_whole(reqs)
     if mode == "tail":
-        return helpers.trace_tail_decode(reqs, TAIL.get(name, 32))
+        return helpers.trace_tail_decode(reqs, TAIL.get(name[0], 32))
     if mode == "every_token":
         return helpers.trace_tail_decode(reqs, 10 ** 6)
     if mode == "portions":
-        return helpers.trace_portions(reqs, **({"sizes": PORTIONS[name]} if name in PORTIONS else {}))
+        return helpers.trace_portions(reqs, **({"sizes": PORTIONS[name[0]]} if name[0] in PORTIONS else {}))
     if mode == "twos":
         return helpers.trace_portions(reqs, sizes=(2,))
     if mode == "mixed":
-        return helpers.trace_mixed(reqs, max_live=4, seed=5, **({"sizes": MIXED[name]} if name in MIXED else {}))
+        return helpers.trace_mixed(reqs, max_live=4, seed=5, **({"sizes": MIXED[name[0]]} if name[0] in MIXED else {}))
     raise ValueError(mode)
 
 
@@ -549,29 +549,19 @@ def replay_case(name, dtype, steps, out_dir, page=None, **more):
     return replay(C.model_dir(name), cfg, page or own_page, dtype, steps, out_dir, **more)
 
 
-def compare(rows, reqs, logits, tol, what, margins=None):
-    """Every position within ``tol`` of the largest logit.  With ``margins`` (bfloat16: per request and position the
-    smallest router margin): positions whose routing is a close call are held to LOOSE only, and of the others at
-    most one in fifty may be over ``tol`` (they come after a close call that went the other way)."""
-    worst, held, over = 0.0, 0, 0
+def compare(rows, reqs, logits, tol, what, some_over=False):
+    """Every position within ``tol`` of the largest logit, or with ``some_over`` six in seven and all within LOOSE."""
+    errs = []
     for name, toks in reqs.items():
         ref = logits[name]
         scale = np.abs(ref).max()
         for p in range(len(toks)):
             err = np.abs(rows[(name, p)] - ref[p]).max() / scale
-            if margins is None:
-                assert err <= tol, (f"{what}: request {name} (length {len(toks)}) first differs at position {p}: "
-                                    f"relative error {err:.3e}")
-            else:
-                assert err <= LOOSE, f"{what}: request {name} position {p}: relative error {err:.3e}"
-                clear = margins[name][p] >= CLOSE_CALL
-                held += clear
-                over += bool(clear and err > tol)
-            worst = max(worst, err)
-    if margins is not None:
-        total = sum(len(t) for t in reqs.values())
-        assert held >= 0.5 * total and over <= 1 + 0.02 * held, f"{what}: {over} of {held} clear positions over {tol}"
-    return worst
+            assert err <= (LOOSE if some_over else tol), (
+                f"{what}: request {name} (length {len(toks)}) first differs at position {p}: relative error {err:.3e}")
+            errs.append(err)
+    assert np.mean(np.array(errs) > tol) <= 1 / 7, f"{what}: {np.mean(np.array(errs) > tol):.3f} of the positions over {tol}"
+    return max(errs)
 
 
 @pytest.mark.parametrize("mode", ["whole", "tail", "portions", "mixed"])
@@ -583,18 +573,18 @@ def test_replay_matches_plain(name, dtype, mode, tmp_path):
     request is compared, the first tokens included."""
     reqs, logits = oracle(name)
     rows = replay_case(name, dtype, make_trace(mode, reqs, name), tmp_path)
-    worst = compare(rows, reqs, logits, TOL[dtype], f"{name} {dtype} {mode}", margins_of(name, dtype))
+    worst = compare(rows, reqs, logits, TOL[dtype], f"{name} {dtype} {mode}", chosen(name, dtype))
     print(f"{name} {dtype} {mode}: worst relative error {worst:.3e}")
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["A", "B", "C", "E"])
+@pytest.mark.parametrize("name", ["A-all", "B", "C", "E"])
 def test_every_token_decoded_alone_matches_whole_prompts(name, dtype, tmp_path):
     """Token-by-token decoding from the first token on (through the decode graphs and with graphs off), and two tokens
     at a time: memories that start from nothing, chunks that single tokens open."""
     reqs, logits = oracle(name)
     few = dict(list(reqs.items())[1:5])
-    steps, mg = make_trace("every_token", few, name), margins_of(name, dtype)
+    steps, mg = make_trace("every_token", few, name), chosen(name, dtype)
     compare(replay_case(name, dtype, steps, tmp_path / "g"), few, logits, TOL[dtype], "decoded", mg)
     compare(replay_case(name, dtype, steps, tmp_path / "e", use_graphs=False), few, logits, TOL[dtype], "decoded, no graphs", mg)
     compare(replay_case(name, dtype, make_trace("twos", few, name), tmp_path / "t"), few, logits, TOL[dtype], "in twos", mg)
@@ -607,7 +597,7 @@ def test_other_page_sizes(page, tmp_path):
         steps = make_trace(mode, reqs, "A")
         for dtype in DTYPES:
             compare(replay_case("A", dtype, steps, tmp_path / f"{mode}{dtype}", page=page), reqs, logits, TOL[dtype],
-                    f"page {page} {dtype}", margins_of("A", dtype))
+                    f"page {page} {dtype}", chosen("A", dtype))
 
 
 def test_repeated_layouts_replay_a_graph(tmp_path, monkeypatch):
@@ -617,17 +607,16 @@ def test_repeated_layouts_replay_a_graph(tmp_path, monkeypatch):
     cfg = C.CASE_A
     reqs = {f"g{i}": p for i, p in enumerate(C.prompts(cfg["vocab"], [48] * 5, seed=31))}
     plain = C.plain_model("A")
-    both = {k: plain.forward_with_margins(v) for k, v in reqs.items()}
-    logits, mg = {k: v[0] for k, v in both.items()}, {k: v[1] for k, v in both.items()}
+    logits = {k: plain.forward(v) for k, v in reqs.items()}
     for dtype in DTYPES:
         compare(replay_case("A", dtype, helpers.trace_portions(reqs, sizes=(24,)), tmp_path / dtype), reqs, logits, TOL[dtype],
-                "repeated layouts", mg if dtype == "bfloat16" else None)
+                "repeated layouts", chosen("A", dtype))
 
 
 def test_batch_of_unequal_requests_equals_each_alone(tmp_path):
     """One step with four prompts of unequal length beside one another, then single tokens of all four in one
     step: the rows equal those of each request run alone."""
-    reqs, logits = oracle("D")
+    reqs, logits = oracle("D-all")
     names = list(reqs)[:4]
     together = [{"step": 0, "entries": [{"id": n, "tokens": reqs[n][:-1], "want": list(range(len(reqs[n]) - 1))}
                                          for n in names], "end": []},
@@ -639,12 +628,11 @@ def test_batch_of_unequal_requests_equals_each_alone(tmp_path):
         alone.append({"step": k + 1, "entries": [{"id": n, "tokens": reqs[n][-1:], "want": [0]}], "end": [n]})
         k += 2
     for dtype in DTYPES:
-        a = replay_case("D", dtype, together, tmp_path / f"t{dtype}")
-        b = replay_case("D", dtype, alone, tmp_path / f"a{dtype}")
-        compare(a, {n: reqs[n] for n in names}, logits, TOL[dtype], "together", margins_of("D", dtype))
+        a = replay_case("D-all", dtype, together, tmp_path / f"t{dtype}")
+        b = replay_case("D-all", dtype, alone, tmp_path / f"a{dtype}")
+        compare(a, {n: reqs[n] for n in names}, logits, TOL[dtype], "together", chosen("D-all", dtype))
         far = [np.abs(a[key] - b[key]).max() / np.abs(b[key]).max() for key in a]
-        # in bfloat16 the expanded and the compressed form of a latent round differently, and a close call may tip
-        assert max(far) <= 2e-5 if dtype == "float32" else np.quantile(far, 0.95) <= 0.1
+        assert max(far) <= (2e-5 if dtype == "float32" else 0.1)   # bfloat16: a latent's two forms round differently
 
 
 # ---- models in which one mechanism carries everything -----------------------------------------------------
