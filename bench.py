@@ -1031,6 +1031,144 @@ def run_sagizen(args):
     return 0
 
 
+def bunudra_sizes(name):
+    """(Bunudra configuration, and two designs at equal width, number of layers, vocabulary and feed-forward weights:
+    Dizatar, whose every layer is latent attention over a mixture of experts with a shared expert, and Mepatar with the
+    gated delta rule and windowed attention; its experts have no shared one beside them, so it gets larger ones)."""
+    def all_of(width, heads, kv, d, lat, rank, experts, groups, top, ff, shared, vocab):
+        dn, dr, dv = lat
+        moe = dict(kind="moe", router=dict(experts=experts, top=top, scale=2.5, groups=dict(count=groups[0], keep=groups[1])),
+                   expert=dict(ff=ff), shared=dict(ff=shared))
+        mem = dict(type="mlstm", mixer=dict(heads=heads, dim=d // 2, vdim=d, gate_cap=15.0), mlp=moe)
+        lt = dict(heads=heads, dim=dn, rot_dim=dr, vdim=dv, kv_rank=rank, scale=(dn + dr) ** -0.5)
+        yarn = dict(factor=8.0, original=4096, fast=32.0, slow=1.0)
+        lat = dict(type="latent_attention", mixer=dict(lt, mask=dict(size=512), rot=dict(base=10000.0, dims=dr, scaling=yarn)), mlp=moe)
+        att = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv, dim=d, vdim=d, scale=d ** -0.5, mask=dict(size=768),
+                                                rot=dict(base=10000.0, dims=d)), mlp=moe)
+        bun = dict(architecture="Bunudra", width=width, vocab=vocab, norm=dict(eps=1e-6), embedding=dict(scale=1.0),
+                   layers=[mem, lat, att, mem, lat, att])
+        gff, gshared = ff * 2 // 3, shared * 2 // 3
+        dmoe = dict(kind="moe", router=dict(experts=experts, identity=0, top=top), expert=dict(ff=gff), shared=dict(ff=gshared))
+        dlat = dict(type="latent_attention", mixer=dict(lt, rot=dict(base=10000.0, dims=dr)), mlp=dmoe)
+        diz = dict(architecture="Dizatar", width=width, vocab=vocab, norm=dict(eps=1e-6), residual_mult=1.0, layers=[dlat] * 6)
+        mmoe = dict(kind="moe", router=dict(experts=experts, top=top), expert=dict(ff=gff + gshared // top, limit=7.0))
+        delta = dict(type="delta", mixer=dict(heads=heads, kv_heads=heads // 2, dim=d, vdim=d, conv=4), mlp=mmoe)
+        watt = dict(type="attention", mixer=dict(heads=heads, kv_heads=kv, dim=d, vdim=d, scale=d ** -0.5,
+                                                 rot=dict(base=10000.0, dims=d // 2), mask=dict(size=512, keep_first=4)), mlp=mmoe)
+        mep = dict(architecture="Mepatar", width=width, vocab=vocab, norm=dict(eps=1e-6, groups=4),
+                   embedding=dict(scale=width ** 0.5), canon=dict(taps=4), layers=[delta, watt, watt, delta, watt, watt])
+        return dict(bunudra=bun, dizatar=diz, mepatar=mep)
+
+    if name == "w2048":      # 16 heads of 128 (memory: 64 x 128; latent of 512: 128 + 64); 32 experts of 1,536, 4 chosen of 2 groups of 8
+        return all_of(2048, 16, 2, 128, (128, 64, 128), 512, 32, (4, 2), 4, 1536, 3072, 32768)
+    if name == "w1024":      # 8 heads of 128 (memory: 64 x 128; latent of 256: 64 + 32); 16 experts of 768, 2 chosen of 2 groups of 4
+        return all_of(1024, 8, 2, 128, (64, 32, 64), 256, 16, (4, 2), 2, 768, 1536, 32768)
+    raise ValueError(name)
+
+
+def bunudra_decode_bytes(cfg, batch, context):
+    """Bytes a decode step has to read or write: the weights of every layer (of the experts, those that ``batch`` tokens
+    are expected to touch under uniform routing), the head, and what the live requests keep: memories in 32-bit (read
+    and written), latent rows as far back as the window, keys and values of the open chunk."""
+    W, V = cfg["width"], cfg["vocab"]
+    total = V * W * 2
+    for L in cfg["layers"]:
+        m, f = L["mixer"], L["mlp"]
+        H = m["heads"]
+        if L["type"] == "mlstm":
+            d, dv = m["dim"], m["vdim"]
+            total += (2 * H * (d + dv) + 2 * H) * W * 2 + W * H * dv * 2 + batch * H * ((dv + 1) * d + 1) * 4 * 2
+        elif L["type"] == "latent_attention":
+            dn, dr, dv, R = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            total += ((H * (dn + dr) + R + dr + H * dv) * W + H * (dn + dv) * R + W * H * dv) * 2
+            total += batch * min(context, m["mask"]["size"]) * (R + dr) * 2
+        else:
+            G, d, dv, D = m["kv_heads"], m["dim"], m["vdim"], -(-max(m["dim"], m["vdim"]) // 16) * 16
+            total += ((H + G) * d + G * dv) * W * 2 + W * H * dv * 2 + batch * (context % m["mask"]["size"] + 1) * G * 2 * D * 2
+        if f:
+            E, top, F = f["router"]["experts"], f["router"]["top"], f["expert"]["ff"]
+            touched = E * (1.0 - (1.0 - top / E) ** batch)
+            total += touched * 2 * F * W * 2 + E * W * 4 + 2 * f["shared"]["ff"] * W * 2
+    return total
+
+
+def bunudra_prefill_flops(cfg, T):
+    """FLOPs of one prompt of T tokens: products, attention over the keys a query sees (a latent in the expanded form,
+    with the expansion of every token), the memories' updates and read-outs (4 d dv per head and token)."""
+    W, V = cfg["width"], cfg["vocab"]
+    total = 2 * V * W
+    for L in cfg["layers"]:
+        m, f = L["mixer"], L["mlp"]
+        H = m["heads"]
+        if L["type"] == "mlstm":
+            d, dv = m["dim"], m["vdim"]
+            total += 2 * T * ((2 * H * (d + dv) + 2 * H) * W + W * H * dv) + T * H * 4 * d * dv
+        elif L["type"] == "latent_attention":
+            dn, dr, dv, R, win = m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["mask"]["size"]
+            pairs = sum(min(t + 1, win) for t in range(T))
+            total += 2 * T * ((H * (dn + dr) + R + dr + 2 * H * dv) * W + H * (dn + dv) * R) + H * 2 * (dn + dr + dv) * pairs
+        else:
+            G, d, dv = m["kv_heads"], m["dim"], m["vdim"]
+            pairs = sum(t % m["mask"]["size"] + 1 for t in range(T))
+            total += 2 * T * (((H + G) * d + G * dv) * W + W * H * dv) + H * 2 * (d + dv) * pairs
+        if f:
+            total += 2 * T * (f["router"]["top"] * 2 * f["expert"]["ff"] * W + f["router"]["experts"] * W + 2 * f["shared"]["ff"] * W)
+    return total
+
+
+def run_bunudra(args):
+    """Prefill and decode throughput of Bunudra at layer sizes of real models (random weights), beside the closest two
+    designs at equal width, number of layers, vocabulary and feed-forward weights.  One JSON line per model and size."""
+    import numpy as np
+    import torch
+    from railgun_b200.engine.batch import StepEntry
+    from railgun_b200.engine.engine import Engine
+    page, pool_tokens = 16, 64 * 4096
+    pk, pk_src = peaks()
+    counts = dict(bunudra=(bunudra_decode_bytes, bunudra_prefill_flops), dizatar=(dizatar_decode_bytes, dizatar_prefill_flops),
+                  mepatar=(mepatar_decode_bytes, mepatar_prefill_flops))
+    models = set(args.models.split(",")) if args.models else None
+    for size in (args.sizes.split(",") if args.sizes else ["w1024", "w2048"]):
+        for label, cfg in bunudra_sizes(size).items():
+            if models and label not in models:
+                continue
+            eng = Engine(model_folder(cfg), dtype="bfloat16", block_size=page, num_gpu_blocks=pool_tokens // page,
+                         max_num_seqs=64, max_num_batched_tokens=8192, max_model_len=4096)
+            runner, V, rng = eng.runner, cfg["vocab"], np.random.default_rng(0)
+            _, _, time_decode = decode_tools(runner, V, rng)
+            line = {"mode": "bunudra", "size": size, "model": label, "layer_runs": len(runner.model.order),
+                    "cache_bytes_per_token": runner.cache.bytes_per_token()}
+            with ClockSampler() as clocks:
+                for b in (8, 64):
+                    tok_s, ms, n_launch, _ = time_decode(b, args.steps, args.warmup, 1000 * b, args.context)
+                    line[f"decode_b{b}_tok_s"], line[f"decode_b{b}_ms"] = round(tok_s, 1), round(ms, 4)
+                    line[f"decode_b{b}_launches_per_step"] = n_launch // args.steps
+                    by = counts[label][0](cfg, b, args.context + args.warmup + args.steps // 2)
+                    line[f"decode_b{b}_GB_per_step"] = round(by / 1e9, 3)
+                    line[f"decode_b{b}_frac_hbm"] = round(by / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 3)
+                prompt = rng.integers(0, V, size=args.tokens).tolist()
+                times = []
+                for i in range(args.warmup + 7):
+                    torch.cuda.synchronize()
+                    t0, t1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                    t0.record()
+                    runner.step([StepEntry(7000 + i, prompt, [args.tokens - 1])])
+                    t1.record()
+                    torch.cuda.synchronize()
+                    runner.end([7000 + i])
+                    times.append(t0.elapsed_time(t1))
+            runner.check_device_errors()
+            ms = sorted(times[args.warmup:])[len(times[args.warmup:]) // 2]
+            fl = counts[label][1](cfg, args.tokens)
+            line.update(prefill_tokens=args.tokens, prefill_ms=round(ms, 3), prefill_tok_s=round(args.tokens / ms * 1e3, 1),
+                        prefill_TFLOP=round(fl / 1e12, 3), prefill_frac_flops=round(fl / (ms * 1e-3) / (pk["bf16_tflops"] * 1e12), 3),
+                        peaks=pk_src, clocks=clocks.summary())
+            print(json.dumps(line), flush=True)
+            del eng, runner, time_decode
+            torch.cuda.empty_cache()
+    return 0
+
+
 def run_kernels(args):
     """Times the hot kernels one by one, each as a CUDA graph of 16 calls over 16 different operand sets (so
     that weights and caches come from HBM, not L2), with CUDA events around replays.  One JSON line per case."""
@@ -1688,6 +1826,188 @@ def run_kernels(args):
             ends = int(((pos + 1) % pool == 0).sum())
             out(f"pooled entries of {T} tokens ({ends} blocks)", us,
                 frac=round(ends * (pool + 1) * 2 * G * dd * 2 / us / 1e3 / pk["hbm_gbs"], 3))
+    if on("bunudra_rows"):
+        # Bunudra's own kernels by the bytes they have to move, each beside the like kernel of another design: the layer
+        # norm behind a part beside the RMS norm there, the memory of xLSTM beside retention's and Mamba-2's states, its
+        # output's kernel beside the heads' norm with a gate, the router with groups and a gate beside the one without,
+        # experts with an exact gelu beside gated ones, attention in chunks beside a window, the latent's rows with
+        # scaled rotations and the windowed latent beside those without
+        from types import SimpleNamespace
+        from railgun_b200.parts.latent_attention import rotary_frequencies
+        pk, _ = peaks()
+        gbs = lambda by, us: round(by / us / 1e3 / pk["hbm_gbs"], 3)
+        tfl = lambda fl, us: round(fl / us / 1e6 / pk["bf16_tflops"], 3)
+        W = 2048
+        for T in (64, 4096):
+            R_ = 1 if T > 64 else T
+            per = T // R_
+            batch = SimpleNamespace(cu_seqlens=torch.arange(0, T + 1, per, dtype=torch.int32, device=dev),
+                                    num_requests=R_, req_of_token=(torch.arange(T, device=dev) // per).to(torch.int32),
+                                    start_pos=torch.full((R_,), 1000, dtype=torch.int32, device=dev), decode_only=R_ == T,
+                                    state_slots=torch.arange(R_, dtype=torch.int32, device=dev), max_query_len=per,
+                                    positions=(1000 + torch.arange(T, device=dev) % per).to(torch.int32))
+            ys = [torch.randn(T, W, device=dev).to(torch.bfloat16) for _ in range(L)]
+            y32 = [torch.randn(T, W, device=dev) for _ in range(L)]
+            rs = [torch.randn(T, W, device=dev) for _ in range(L)]
+            nw, nb = torch.ones(W, device=dev), torch.zeros(W, device=dev)
+            us = timed(lambda: [ops.stream_norm(r, ops.PendingNormed(y, nw, 1e-6, nb), None, torch.bfloat16) for r, y in zip(rs, ys)])
+            us32 = timed(lambda: [ops.stream_norm(r, ops.PendingNormed(y, nw, 1e-6, nb), None, torch.bfloat16) for r, y in zip(rs, y32)])
+            us2 = timed(lambda: [ops.postnorm_shift(r, ops.PendingNormed(y, nw, 1e-6), None, None, None, torch.bfloat16)
+                                 for r, y in zip(rs, ys)])
+            by = T * W * (4 + 2 + 4 + 2)
+            out(f"layer norm behind the part, addition W{W} T{T}", us, frac=gbs(by, us), from_32bit_us=round(us32, 2),
+                from_32bit_frac=gbs(by + 2 * T * W, us32), rms_us=round(us2, 2), rms_frac=gbs(by, us2))
+            # the memory: 16 heads of 64 x 128, beside retention with heads of 64 x 128 and Mamba-2 with 32 heads of 128 x 64
+            Hm, d, dv, cap = 16, 64, 128, 15.0
+            n_in = 2 * Hm * (d + dv) + 2 * Hm
+            projs = [torch.randn(T, n_in, device=dev) for _ in range(L)]
+            ib, fb = torch.zeros(Hm, device=dev), torch.full((Hm,), 4.0, device=dev)
+            sts = [torch.randn(R_, Hm, dv + 1, d, device=dev) * 0.1 for _ in range(L)]
+            ms_ = [torch.rand(R_, Hm, device=dev) for _ in range(L)]
+            nwm = torch.ones(Hm * dv, device=dev)
+            rst = [torch.randn(R_, Hm, dv, d, device=dev) * 0.1 for _ in range(L)]
+            dec = torch.full((Hm,), 0.99, device=dev)
+            g_off = Hm * (2 * d + dv)
+            ret = lambda p, st: ops.state_scan(p[:, :Hm * d], p[:, Hm * d:2 * Hm * d], p[:, 2 * Hm * d:g_off], st, batch, Hm, d, dv,
+                                               decay=dec)
+            usr = timed(lambda: [ret(p, st) for p, st in zip(projs, rst)])
+            by_r = T * Hm * (2 * d + 2 * dv) * 4 + R_ * Hm * dv * d * 8
+            if T == R_:
+                us1 = timed(lambda: [ops.mlstm_step(p, ib, fb, cap, st, m_, batch, Hm, d, dv) for p, st, m_ in zip(projs, sts, ms_)])
+
+                def step(p, st, m_):
+                    o = ops.mlstm_step(p, ib, fb, cap, st, m_, batch, Hm, d, dv)
+                    return ops.mlstm_out(o, p, nwm, 1e-6, d ** -0.5, None, ib, fb, cap, m_, batch, Hm, d, dv, torch.bfloat16)
+                us = timed(lambda: [step(p, st, m_) for p, st, m_ in zip(projs, sts, ms_)])
+                usr2 = timed(lambda: [ops.head_norm_gate(ret(p, st), p[:, g_off:g_off + Hm * dv], nwm, 1e-6, torch.bfloat16)
+                                      for p, st in zip(projs, rst)])
+                by = T * n_in * 4 + R_ * Hm * ((dv + 1) * d + 1) * 8
+                out(f"memory between its products, single tokens, {T} requests", us, frac=gbs(by + T * Hm * dv * 2, us),
+                    step_us=round(us1, 2), step_frac=gbs(by, us1), retention_us=round(usr2, 2),
+                    retention_frac=gbs(by_r + T * Hm * dv * (4 + 2 - 4), usr2), retention_scan_us=round(usr, 2),
+                    retention_scan_frac=gbs(by_r, usr))
+            else:
+                us = timed(lambda: [ops.mlstm_scan(p, ib, fb, cap, st, m_, batch, Hm, d, dv, chunked=True) for p, st, m_ in zip(projs, sts, ms_)])
+                ust = timed(lambda: [ops.mlstm_scan(p, ib, fb, cap, st, m_, batch, Hm, d, dv, chunked=False) for p, st, m_ in zip(projs, sts, ms_)])
+                Hs, N, sv, Gs = 32, 128, 64, 2
+                xbc = [torch.randn(T, Hs * sv + 2 * Gs * N, device=dev) * 0.3 for _ in range(L)]
+                dt, A, D = torch.rand(T, Hs, device=dev) * 0.1, torch.zeros(Hs, device=dev), torch.ones(Hs, device=dev)
+                sss = [torch.randn(1, Hs, sv, N, device=dev) * 0.1 for _ in range(L)]
+                us2 = timed(lambda: [ops.ssd_chunk_scan(x, dt, A, D, st, batch, Hs, Gs, N, sv) for x, st in zip(xbc, sss)])
+                by = T * Hm * (2 * d + 2 * dv + 3) * 4
+                # fused multiply-adds of the chunked form per token: state sums and read-outs 2 d dv, dot products and their sums 64 (d + dv) / 2
+                fma = lambda h, a, b, g: h * (2 * a * b + 32 * b) + g * 32 * a
+                out(f"gates and recurrence of the memory H{Hm} {d} x {dv} T{T}", us, frac=gbs(by, us),
+                    TFLOPs=round(2 * T * fma(Hm, d, dv, Hm) / us / 1e6, 1), tokens_us=round(ust, 2), ssd_us=round(us2, 2),
+                    ssd_frac=gbs(T * (2 * Hs * sv + 2 * Gs * N) * 4, us2), ssd_TFLOPs=round(2 * T * fma(Hs, N, sv, Gs) / us2 / 1e6, 1),
+                    retention_us=round(usr, 2), retention_frac=gbs(by_r, usr))
+                os_ = [torch.randn(T, Hm, dv + 1, device=dev) for _ in range(L)]
+                oh = [torch.randn(T, Hm, dv, device=dev) for _ in range(L)]
+                mr = torch.rand(T, Hm, device=dev)
+                us = timed(lambda: [ops.mlstm_out(o, p, nwm, 1e-6, d ** -0.5, mr, ib, fb, cap, ms_[0], batch, Hm, d, dv, torch.bfloat16)
+                                    for o, p in zip(os_, projs)])
+                us2 = timed(lambda: [ops.head_norm_gate(o, p[:, g_off:g_off + Hm * dv], nwm, 1e-6, torch.bfloat16) for o, p in zip(oh, projs)])
+                out(f"memory's output: quotient, heads' norm, gate T{T}", us, frac=gbs(T * Hm * dv * 10, us), heads_us=round(us2, 2),
+                    heads_frac=gbs(T * Hm * dv * 10, us2))
+            # the gate on the heads' outputs
+            xs = [torch.randn(T, W, device=dev).to(torch.bfloat16) for _ in range(L)]
+            us = timed(lambda: [ops.sigmoid_gate_(x, y, 128) for x, y in zip(xs, ys)])
+            us2 = timed(lambda: [ops.activation(x, "silu") for x in xs])
+            out(f"sigmoid gate on the heads' outputs W{W} T{T}", us, frac=gbs(T * W * 6, us), silu_us=round(us2, 2), silu_frac=gbs(T * W * 4, us2))
+            # router, experts, sum
+            E, top, F = 32, 4, 1536
+            router, corr, gate = torch.randn(E, W, device=dev) * 0.02, torch.zeros(E, device=dev), torch.randn(W, device=dev) * 0.02
+            us = timed(lambda: [ops.moe_route(x, router, None, top, False, groups=(4, 2), scale=2.5, gate_row=gate) for x in xs])
+            us2 = timed(lambda: [ops.moe_route(x, router, corr, top) for x in xs])
+            out(f"router over {E} with groups and a gate T{T}", us, frac=gbs(T * W * 2 + E * W * 4, us), plain_us=round(us2, 2),
+                plain_frac=gbs(T * W * 2 + E * W * 4, us2))
+            ids = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(T)]).to(torch.int32).contiguous()
+            wu = [(torch.randn(E, F, W, device=dev) / W ** 0.5).to(torch.bfloat16) for _ in range(L)]
+            wg = [(torch.randn(E, 2 * F * 2 // 3, W, device=dev) / W ** 0.5).to(torch.bfloat16) for _ in range(L)]
+            tr = ops.moe_tile_rows(torch.bfloat16, T * top, E, W, F)
+            sp, pp, tiles = ops.moe_align(ids, E, tr)
+            us = timed(lambda: [ops.moe_grouped_gemm(xs[0], sp, top, w, tiles, T * top, False, tr, plain_act="gelu") for w in wu])
+            us2 = timed(lambda: [ops.moe_grouped_gemm(xs[0], sp, top, w, tiles, T * top, True, tr) for w in wg])
+            touched = int(torch.unique(ids).numel())
+            by, by2 = touched * F * W * 2, touched * (2 * F * 2 // 3) * W * 2
+            fl, fl2 = 2 * T * top * F * W, 2 * T * top * (2 * F * 2 // 3) * W
+            out(f"experts' first product with gelu {E} x {F} T{T}", us, frac_hbm=gbs(by, us), frac_flops=tfl(fl, us), gated_us=round(us2, 2),
+                gated_frac_hbm=gbs(by2, us2), gated_frac_flops=tfl(fl2, us2))
+            del wu, wg
+            wts, sg = torch.rand(T, top, device=dev), torch.rand(T, device=dev)
+            yy = [torch.randn(T * top, W, device=dev).to(torch.bfloat16) for _ in range(L)]
+            us = timed(lambda: [ops.moe_combine(x, y, s_, ids, wts, pp, E, shared_weight=sg, all_experts=True) for x, y, s_ in zip(xs, yy, ys)])
+            us2 = timed(lambda: [ops.moe_combine(x, y, s_, ids, wts, pp, E) for x, y, s_ in zip(xs, yy, ys)])
+            by = T * W * (top * 2 + 2 + 4)
+            out(f"experts' sum with a gated shared one W{W} T{T}", us, frac=gbs(by, us), plain_us=round(us2, 2), plain_frac=gbs(by + T * W * 2, us2))
+            del yy
+            # a latent's rows: 16 heads of 128 + 64 over 512
+            Hl, dn, dr, R = 16, 128, 64, 512
+            pr = [torch.randn(T, Hl * (dn + dr) + R + dr, device=dev).to(torch.bfloat16) for _ in range(L)]
+            caches = [torch.zeros(-(-T // page), page, R + dr, dtype=torch.bfloat16, device=dev) for _ in range(L)]
+            qa = torch.empty(T, Hl, R + dr, dtype=torch.bfloat16, device=dev)
+            freq, nr = rotary_frequencies(dr, 10000.0).to(dev), torch.ones(R, device=dev)
+            slots = torch.arange(T, dtype=torch.int32, device=dev)
+            rope = lambda **k: timed(lambda: [ops.latent_rope_cache(p, Hl * (dn + dr), qa, c, nr, 1e-6, freq, dr, batch.positions, slots,
+                                                                    Hl, dn, dr, R, **k) for p, c in zip(pr, caches)])
+            us, us2 = rope(interleaved=True, mult=1.2), rope()
+            by = T * (Hl * dr * 4 + (R + dr) * 4)
+            out(f"latent rows and rotations H{Hl} {dn}+{dr} of {R} T{T}", us, frac=gbs(by, us), plain_us=round(us2, 2), plain_frac=gbs(by, us2))
+        # attention at context 4,096: chunks of 768 (the open one holds 256 keys at the end) beside a window of as many
+        # keys on average; a latent's window of 512 beside the whole context
+        Hh, G, dd, size = 16, 2, 128, 768
+        for T, B in ((64, 64), (4096, 1)):
+            ctx = 4096
+            blocks = -(-ctx // page)
+            kvs = [torch.randn(B * blocks, 2, G, page, dd, device=dev).to(torch.bfloat16) for _ in range(L)]
+            bt = torch.arange(B * blocks, dtype=torch.int32, device=dev).view(B, blocks).contiguous()
+            q = (torch.randn(T, Hh * dd, device=dev) * dd ** -0.5).to(torch.bfloat16)
+            req = (torch.arange(T, device=dev) // (T // B)).to(torch.int32)
+            pos = (torch.arange(T, device=dev) % (T // B) + (ctx - T // B)).to(torch.int32)
+            o = torch.empty(T, Hh * dd, dtype=torch.bfloat16, device=dev)
+            t64 = torch.tensor([(k, min(64, T - k), 0) for k in range(0, T, 64)], dtype=torch.int32, device=dev)
+            win = 256 if B > 1 else size // 2
+            res = {}
+            for form, more, w_ in (("chunk", dict(chunk=size), 0), ("window", {}, win)):
+                if B > 1:
+                    splits = ops.decode_splits(T, G * (-(-(Hh // G) // 8)), size if form == "chunk" else win)
+                    res[form] = timed(lambda: [ops.decode_attention(q, Hh * dd, o, kv, bt, None, T, req, pos, Hh, G, dd, w_, 1.0, splits, **more)
+                                               for kv in kvs])
+                else:
+                    res[form] = timed(lambda: [ops.prefill_attention(q, Hh * dd, o, kv, bt, t64, pos, Hh, G, dd, w_, 1.0, **more) for kv in kvs])
+            see = dict(chunk=lambda p: p % size + 1, window=lambda p: min(p + 1, win))
+            seen = {f: sum(see[f](int(p)) for p in pos.tolist()) for f in res}
+            info = {}
+            for f, us in res.items():
+                info[f + "_us"] = round(us, 2)
+                info[f + "_frac"] = gbs(seen[f] * G * 2 * dd * 2, us) if B > 1 else tfl(Hh * 4 * dd * seen[f], us)
+            out(f"attention in chunks of {size}, H{Hh} G{G} d{dd}, {B} requests x {T // B} tokens", res["chunk"], **info)
+            del kvs
+            Hl, R, dr, dn, dv, win = 16, 512, 64, 128, 128, 512
+            D = R + dr
+            caches = [torch.randn(B * blocks, page, D, device=dev).to(torch.bfloat16) for _ in range(L)]
+            if B > 1:
+                qa = (torch.randn(T, Hl, D, device=dev) * D ** -0.5).to(torch.bfloat16)
+                ol = torch.empty(T, Hl, R, dtype=torch.bfloat16, device=dev)
+                lat = lambda w_: timed(lambda: [ops.latent_attention_mma(qa, ol, c, bt, None, None, T, req, pos, R, w_, 1.0,
+                                                                         ops.latent_decode_splits(T, 1, w_ or ctx)) for c in caches])
+                us, us2 = lat(win), lat(0)
+                out(f"latent attention window {win}, H{Hl} of {R}+{dr}, {B} requests", us, frac=gbs(B * win * D * 2, us), whole_us=round(us2, 2),
+                    whole_frac=gbs(B * ctx * D * 2, us2))
+            else:
+                uk, uv = ((torch.randn(Hl * n, R, device=dev) / R ** 0.5).to(torch.bfloat16) for n in (dn, dv))
+                qx = (torch.randn(T, Hl * (dn + dr), device=dev) * 0.05).to(torch.bfloat16)
+                ox = torch.zeros(T, Hl * (dn + dr), dtype=torch.bfloat16, device=dev)
+                cu, cl = torch.tensor([0, T], dtype=torch.int32, device=dev), torch.tensor([ctx], dtype=torch.int32, device=dev)
+                use = timed(lambda: [ops.latent_expand_context(c, bt, cu, cl, uk, uv, Hl, dn, dr, dv, R) for c in caches])
+                kv, kt = ops.latent_expand_context(caches[0], bt, cu, cl, uk, uv, Hl, dn, dr, dv, R)
+                att = lambda w_: timed(lambda: [ops.prefill_attention(qx, Hl * (dn + dr), ox, kv, kt, t64, pos, Hl, Hl, dn + dr, w_, 1.0)
+                                                for _ in range(L)])
+                us, us2 = att(win), att(0)
+                pairs = lambda w_: sum(min(int(p) + 1, w_ or ctx) for p in pos.tolist())
+                out(f"latent attention window {win}, H{Hl} expanded {dn}+{dr}, {T} tokens", us, frac=tfl(Hl * 2 * (dn + dr + dv) * pairs(win), us),
+                    whole_us=round(us2, 2), whole_frac=tfl(Hl * 2 * (dn + dr + dv) * pairs(0), us2), expand_us=round(use, 2),
+                    expand_frac_flops=tfl(2 * ctx * R * Hl * (dn + dv), use))
     if on("moe"):
         # the routed experts' two grouped products (32 experts of 1,024 at width 2,048, 4 choices) beside the dense
         # model's gate|up and down products of equal work: decode by bytes of weights read, prompts by FLOP/s
@@ -1736,16 +2056,18 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the named configuration (0: all)")
     ap.add_argument("--mode", default="all", choices=["all", "decode", "prefill", "kernels", "dizatar", "rupulix", "mepatar", "kasarax",
-                                                           "sagizen"],
+                                                           "sagizen", "bunudra"],
                     help="all: the contract's line; decode / prefill: one short measurement (for profiling); "
                          "kernels: the hot kernels one by one; dizatar / rupulix: prefill and decode of the Dizatar / Rupulix design at "
                          "layer sizes of real models beside the dense model of equal width; mepatar: the same for "
                          "the Mepatar design beside Rupulix; kasarax: the same for the Kasarax design beside Mepatar; "
-                         "sagizen: the same for the Sagizen design beside Mepatar and Kasarax")
-    ap.add_argument("--sizes", default="", help="--mode dizatar / rupulix / mepatar / kasarax / sagizen: comma-separated subset of w1024, w2048")
+                         "sagizen: the same for the Sagizen design beside Mepatar and Kasarax; "
+                         "bunudra: the same for the Bunudra design beside Dizatar and Mepatar")
+    ap.add_argument("--models", default="", help="--mode bunudra: comma-separated subset of bunudra, dizatar, mepatar")
+    ap.add_argument("--sizes", default="", help="--mode dizatar / rupulix / mepatar / kasarax / sagizen / bunudra: comma-separated subset of w1024, w2048")
     ap.add_argument("--cases", default="", help="--mode kernels: comma-separated subset of sampling, decode_gemm, "
                     "decode_gemm_mid, decode_attention, prefill_gemm, prefill_attention, primitives, latent_attention, moe, "
-                    "talking_attention, rupulix_rows, mepatar_rows, kasarax_rows, sagizen_rows")
+                    "talking_attention, rupulix_rows, mepatar_rows, kasarax_rows, sagizen_rows, bunudra_rows")
     ap.add_argument("--batch", type=int, default=8, help="--mode decode: requests in the batch")
     ap.add_argument("--tokens", type=int, default=PREFILL_TOKENS, help="--mode prefill: prompt length")
     ap.add_argument("--context", type=int, default=CONTEXT, help="--mode decode: tokens each request holds")
@@ -1772,6 +2094,8 @@ def main():
         return run_kasarax(args)
     if args.mode == "sagizen":
         return run_sagizen(args)
+    if args.mode == "bunudra":
+        return run_bunudra(args)
     return run_ours(args)
 
 
