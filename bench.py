@@ -1917,8 +1917,9 @@ def run_kernels(args):
             # router, experts, sum
             E, top, F = 32, 4, 1536
             router, corr, gate = torch.randn(E, W, device=dev) * 0.02, torch.zeros(E, device=dev), torch.randn(W, device=dev) * 0.02
-            us = timed(lambda: [ops.moe_route(x, router, None, top, False, groups=(4, 2), scale=2.5, gate_row=gate) for x in xs])
-            us2 = timed(lambda: [ops.moe_route(x, router, corr, top) for x in xs])
+            half = ops.pad_rows(torch.cat([router, gate[None]]).to(torch.bfloat16))
+            us = timed(lambda: [ops.moe_route(x, router, None, top, False, groups=(4, 2), scale=2.5, gate_row=gate, half_rows=half) for x in xs])
+            us2 = timed(lambda: [ops.moe_route(x, router, corr, top) for x in xs])        # every row by the kernel itself
             out(f"router over {E} with groups and a gate T{T}", us, frac=gbs(T * W * 2 + E * W * 4, us), plain_us=round(us2, 2),
                 plain_frac=gbs(T * W * 2 + E * W * 4, us2))
             ids = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(T)]).to(torch.int32).contiguous()

@@ -224,11 +224,14 @@ extern "C" int rg_latent_attention_general(
 // dv to d), which the dense model's flash kernel reads.  The temporary pages are numbered request by request:
 // page j of the step's request r is page r * max_blocks + j.  Requests that bring one token are skipped.
 
+// Both kernels move 16 bytes at a time (V numbers) where every part of a row starts on 16-byte boundaries.
+
 // lat [requests * max_blocks * page_size, R]: row (r * max_blocks + j) * page_size + o = latent of r's token j * page_size + o
-template <typename A>
+template <typename A, int V>
 __global__ void latent_gather_kernel(const A* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
                                      const int* __restrict__ cu_seqlens, const int* __restrict__ context_lens,
                                      A* __restrict__ lat, int page_size, int R, int D) {
+    struct __align__(sizeof(A) * V) Piece { A x[V]; };
     pdl_wait();
     pdl_trigger();
     const int j = blockIdx.x, r = blockIdx.y;
@@ -240,9 +243,10 @@ __global__ void latent_gather_kernel(const A* __restrict__ cache, const int* __r
     const int n = min(page_size, ctx - j * page_size);
     const A* src = cache + (size_t)page * page_size * D;
     A* dst = lat + ((size_t)r * max_blocks + j) * page_size * R;
-    for (int i = threadIdx.x; i < n * R; i += blockDim.x) {
-        const int o = i / R, c = i - o * R;
-        dst[(size_t)o * R + c] = src[(size_t)o * D + c];
+    const int per = R / V;
+    for (int i = blockIdx.z * blockDim.x + threadIdx.x; i < n * per; i += gridDim.z * blockDim.x) {
+        const int o = i / per, c = (i - o * per) * V;
+        *reinterpret_cast<Piece*>(dst + (size_t)o * R + c) = *reinterpret_cast<const Piece*>(src + (size_t)o * D + c);
     }
 }
 
@@ -250,47 +254,57 @@ extern "C" int rg_latent_gather(const void* cache, const int* block_table, int m
                                 const int* context_lens, void* lat, int dtype, int requests, int page_size, int R, int D,
                                 void* stream) {
     if (requests <= 0 || max_blocks <= 0) return 0;
+    if (dtype != RG_DTYPE_BF16 && dtype != RG_DTYPE_F32) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(max_blocks, requests);
-    if (dtype == RG_DTYPE_BF16)
-        return rg_launch(latent_gather_kernel<bf16>, grid, dim3(256), 0, s, 1, (const bf16*)cache, block_table, max_blocks,
-                         cu_seqlens, context_lens, (bf16*)lat, page_size, R, D);
-    if (dtype == RG_DTYPE_F32)
-        return rg_launch(latent_gather_kernel<float>, grid, dim3(256), 0, s, 1, (const float*)cache, block_table,
-                         max_blocks, cu_seqlens, context_lens, (float*)lat, page_size, R, D);
-    return RG_ERR_UNSUPPORTED;
+    const int v = dtype == RG_DTYPE_BF16 ? 8 : 4;
+    const bool vec = R % v == 0 && D % v == 0 && (((uintptr_t)cache | (uintptr_t)lat) & 15) == 0;
+    const long long pieces = (long long)page_size * R / (vec ? v : 1);
+    dim3 grid(max_blocks, requests, pieces > 4096 ? 8 : (unsigned)((pieces + 511) / 512));
+#define LAT_GATHER(A, V) return rg_launch(latent_gather_kernel<A, V>, grid, dim3(256), 0, s, 1, (const A*)cache, block_table, \
+        max_blocks, cu_seqlens, context_lens, (A*)lat, page_size, R, D)
+    if (dtype == RG_DTYPE_BF16) { if (vec) LAT_GATHER(bf16, 8); LAT_GATHER(bf16, 1); }
+    if (vec) LAT_GATHER(float, 4);
+    LAT_GATHER(float, 1);
+#undef LAT_GATHER
 }
 
 // kn [N, H * dn], vv [N, H * dv] (rows as in lat), the rotated key parts from the cache rows' last dr numbers
-// -> kv [requests * max_blocks, 2, H, page_size, d]
-template <typename A>
+// -> kv [requests * max_blocks, 2, H, page_size, d].  One block per temporary page and head.
+template <typename A, int V>
 __global__ void latent_pack_kv_kernel(const A* __restrict__ kn, const A* __restrict__ vv, const A* __restrict__ cache,
                                       const int* __restrict__ block_table, int max_blocks,
                                       const int* __restrict__ cu_seqlens, const int* __restrict__ context_lens,
                                       A* __restrict__ kv, int page_size, int H, int dn, int dr, int dv, int R) {
+    struct __align__(sizeof(A) * V) Piece { A x[V]; };
     pdl_wait();
     pdl_trigger();
-    const int j = blockIdx.x, r = blockIdx.y;
+    const int j = blockIdx.x, r = blockIdx.y, h = blockIdx.z;
     if (cu_seqlens[r + 1] - cu_seqlens[r] < 2) return;
     const int ctx = context_lens[r];
     if (j * page_size >= ctx) return;
     const int page = block_table[(size_t)r * max_blocks + j];
-    const int n = min(page_size, ctx - j * page_size);
-    const int d = dn + dr, D = R + dr;
+    // a page that a window has passed: masked, but read beside the edge, so all of it is zeros
+    const int n = page < 0 ? page_size : min(page_size, ctx - j * page_size);
+    const int d = dn + dr, D = R + dr, per = d / V;
     const size_t tp = (size_t)r * max_blocks + j;                  // the temporary page
-    A* kdst = kv + tp * 2 * H * page_size * d;
-    if (page < 0) {                                                // a window has passed it: masked, but read beside the edge
-        for (int i = threadIdx.x; i < 2 * H * page_size * d; i += blockDim.x) kdst[i] = from_f32<A>(0.f);
-        return;
-    }
+    A* kdst = kv + (tp * 2 * H + h) * page_size * d;
     A* vdst = kdst + (size_t)H * page_size * d;
-    const size_t row0 = tp * page_size;
-    const A* krot = cache + (size_t)page * page_size * D + R;
-    for (int i = threadIdx.x; i < H * n * d; i += blockDim.x) {
-        const int h = i / (n * d), rem = i - h * n * d, o = rem / d, c = rem - o * d;
-        kdst[((size_t)h * page_size + o) * d + c] = c < dn ? kn[(row0 + o) * H * dn + (size_t)h * dn + c]
-                                                           : krot[(size_t)o * D + c - dn];
-        vdst[((size_t)h * page_size + o) * d + c] = c < dv ? vv[(row0 + o) * H * dv + (size_t)h * dv + c] : from_f32<A>(0.f);
+    const A* krow = kn + (tp * page_size * H + h) * dn;
+    const A* vrow = vv + (tp * page_size * H + h) * dv;
+    const A* krot = cache + (size_t)max(page, 0) * page_size * D + R;
+    Piece zero;
+#pragma unroll
+    for (int e = 0; e < V; ++e) zero.x[e] = from_f32<A>(0.f);
+    for (int i = threadIdx.x; i < n * per; i += blockDim.x) {
+        const int o = i / per, c = (i - o * per) * V;
+        Piece k = zero, v = zero;
+        if (page >= 0) {
+            k = c < dn ? *reinterpret_cast<const Piece*>(krow + (size_t)o * H * dn + c)
+                       : *reinterpret_cast<const Piece*>(krot + (size_t)o * D + c - dn);
+            if (c < dv) v = *reinterpret_cast<const Piece*>(vrow + (size_t)o * H * dv + c);
+        }
+        *reinterpret_cast<Piece*>(kdst + (size_t)o * d + c) = k;
+        *reinterpret_cast<Piece*>(vdst + (size_t)o * d + c) = v;
     }
 }
 
@@ -298,16 +312,16 @@ extern "C" int rg_latent_pack_kv(const void* kn, const void* vv, const void* cac
                                  int max_blocks, const int* cu_seqlens, const int* context_lens, void* kv, int dtype,
                                  int requests, int page_size, int H, int dn, int dr, int dv, int R, void* stream) {
     if (requests <= 0 || max_blocks <= 0) return 0;
-    if (dv > dn + dr) return RG_ERR_UNSUPPORTED;
+    if (dv > dn + dr || H < 1 || H > 65535 || (dtype != RG_DTYPE_BF16 && dtype != RG_DTYPE_F32)) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    dim3 grid(max_blocks, requests);
-    if (dtype == RG_DTYPE_BF16)
-        return rg_launch(latent_pack_kv_kernel<bf16>, grid, dim3(256), 0, s, 1, (const bf16*)kn, (const bf16*)vv,
-                         (const bf16*)cache, block_table, max_blocks, cu_seqlens, context_lens, (bf16*)kv, page_size, H, dn,
-                         dr, dv, R);
-    if (dtype == RG_DTYPE_F32)
-        return rg_launch(latent_pack_kv_kernel<float>, grid, dim3(256), 0, s, 1, (const float*)kn, (const float*)vv,
-                         (const float*)cache, block_table, max_blocks, cu_seqlens, context_lens, (float*)kv, page_size, H,
-                         dn, dr, dv, R);
-    return RG_ERR_UNSUPPORTED;
+    dim3 grid(max_blocks, requests, H);
+    const int v = dtype == RG_DTYPE_BF16 ? 8 : 4;
+    const bool vec = dn % v == 0 && dr % v == 0 && dv % v == 0 && R % v == 0
+                     && (((uintptr_t)kn | (uintptr_t)vv | (uintptr_t)cache | (uintptr_t)kv) & 15) == 0;
+#define LAT_PACK(A, V) return rg_launch(latent_pack_kv_kernel<A, V>, grid, dim3(128), 0, s, 1, (const A*)kn, (const A*)vv, \
+        (const A*)cache, block_table, max_blocks, cu_seqlens, context_lens, (A*)kv, page_size, H, dn, dr, dv, R)
+    if (dtype == RG_DTYPE_BF16) { if (vec) LAT_PACK(bf16, 8); LAT_PACK(bf16, 1); }
+    if (vec) LAT_PACK(float, 4);
+    LAT_PACK(float, 1);
+#undef LAT_PACK
 }

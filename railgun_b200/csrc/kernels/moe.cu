@@ -12,20 +12,23 @@
 // the products run over a list of row tiles that `moe_align` writes (at most pairs / tile + E of them; the
 // launch covers that bound and unused tiles return at once), which keeps a step capturable in a CUDA graph.
 //
-//   moe_route          one block per four tokens: its warps (up to 32) share the router's rows, then take a token each
+//   moe_route          one block per 1 to 4 tokens (more the more tokens there are: a router row is read once for all
+//                      of a block's): its warps (up to 32) share the router's rows two by two, then take a token each;
+//                      or, for many tokens, from logits that a matrix product has worked out, a warp per token
 //   moe_align          one block: counts per expert, segment starts, the pairs in expert order, the tile list
 //   moe_grouped_gemm   32-bit arithmetic on CUDA cores, any sizes and both storage types (the true 32-bit path)
 //   moe_combine        one block per token, 32-bit sum in the order of the choices
 #include "common.cuh"
 
-#define ROUTE_TOKENS 4        // tokens per block: a router row is read once for all of them
+#define ROUTE_ROWS 2          // router rows a warp takes at a time: a token's numbers are read once for both
 
-template <typename A>
-__global__ void moe_route_kernel(const A* __restrict__ x, const float* __restrict__ router,
+template <typename A, int ROUTE_TOKENS>
+__global__ void __launch_bounds__(1024)
+moe_route_kernel(const A* __restrict__ x, const float* __restrict__ router,
                                  const float* __restrict__ correction, int* __restrict__ ids,
                                  float* __restrict__ weights, int T, int W, int N, int top, int renormalize,
                                  int scoring, int groups, int keep, float scale, const float* __restrict__ gate_row,
-                                 float* __restrict__ gate) {
+                                 float* __restrict__ gate, const float* __restrict__ logits, int logits_ld) {
     extern __shared__ float sm[];                 // per token of the block: N scores, N choice scores, groups' bests, a gate
     const int stride = 2 * N + groups + 1;
     // gate_row: one more row of the router whose logit's sigmoid is left in gate[t] (a shared expert's weight)
@@ -39,40 +42,64 @@ __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restric
     // every lane adds its own elements in index order (four at a time where rows start on 16-byte boundaries),
     // then the lanes are added up: a token's logits do not depend on what else is in the step
     const bool vec = (W & 3) == 0 && sizeof(A) == 2;
-    for (int n = warp; n < rows; n += nwarps) {
-        const float* wr = n < N ? router + (size_t)n * W : gate_row;
-        float dot[ROUTE_TOKENS];
+    if (logits) {
+        for (int i = threadIdx.x; i < nt * rows; i += blockDim.x) {
+            const int j = i / rows, n = i - j * rows;
+            base[(size_t)j * stride + (n < N ? n : 2 * N + groups)] = logits[(size_t)(t0 + j) * logits_ld + n];
+        }
+    }
+    for (int n0 = logits ? rows : warp * ROUTE_ROWS; n0 < rows; n0 += nwarps * ROUTE_ROWS) {
+        const float* wr[ROUTE_ROWS];
+        float dot[ROUTE_ROWS][ROUTE_TOKENS];
 #pragma unroll
-        for (int j = 0; j < ROUTE_TOKENS; ++j) dot[j] = 0.f;
+        for (int e = 0; e < ROUTE_ROWS; ++e) {
+            const int n = min(n0 + e, rows - 1);
+            wr[e] = n < N ? router + (size_t)n * W : gate_row;
+#pragma unroll
+            for (int j = 0; j < ROUTE_TOKENS; ++j) dot[e][j] = 0.f;
+        }
         if (vec) {
-#pragma unroll 4
+#pragma unroll (ROUTE_TOKENS <= 2 ? 4 : 1)
             for (int i = lane * 4; i < W; i += 128) {
-                const float4 r = *reinterpret_cast<const float4*>(wr + i);
+                float4 r[ROUTE_ROWS];
+#pragma unroll
+                for (int e = 0; e < ROUTE_ROWS; ++e) r[e] = *reinterpret_cast<const float4*>(wr[e] + i);
 #pragma unroll
                 for (int j = 0; j < ROUTE_TOKENS; ++j) {
                     if (j < nt) {
                         const uint2 raw = *reinterpret_cast<const uint2*>(x + (size_t)(t0 + j) * W + i);
-                        const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&raw.x);
-                        const __nv_bfloat162 hi = *reinterpret_cast<const __nv_bfloat162*>(&raw.y);
-                        dot[j] += r.x * __low2float(lo);
-                        dot[j] += r.y * __high2float(lo);
-                        dot[j] += r.z * __low2float(hi);
-                        dot[j] += r.w * __high2float(hi);
+                        const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+                        const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+#pragma unroll
+                        for (int e = 0; e < ROUTE_ROWS; ++e) {
+                            dot[e][j] += r[e].x * lo.x;
+                            dot[e][j] += r[e].y * lo.y;
+                            dot[e][j] += r[e].z * hi.x;
+                            dot[e][j] += r[e].w * hi.y;
+                        }
                     }
                 }
             }
         } else {
             for (int i = lane; i < W; i += 32) {
-                const float r = wr[i];
 #pragma unroll
-                for (int j = 0; j < ROUTE_TOKENS; ++j)
-                    if (j < nt) dot[j] += r * to_f32(x[(size_t)(t0 + j) * W + i]);
+                for (int j = 0; j < ROUTE_TOKENS; ++j) {
+                    if (j < nt) {
+                        const float v = to_f32(x[(size_t)(t0 + j) * W + i]);
+#pragma unroll
+                        for (int e = 0; e < ROUTE_ROWS; ++e) dot[e][j] += wr[e][i] * v;
+                    }
+                }
             }
         }
 #pragma unroll
-        for (int j = 0; j < ROUTE_TOKENS; ++j) {
-            const float d = warp_sum(dot[j]);
-            if (lane == 0) base[(size_t)j * stride + (n < N ? n : 2 * N + groups)] = d;
+        for (int e = 0; e < ROUTE_ROWS; ++e) {
+            const int n = n0 + e;
+#pragma unroll
+            for (int j = 0; j < ROUTE_TOKENS; ++j) {
+                const float d = warp_sum(dot[e][j]);
+                if (lane == 0 && n < rows) base[(size_t)j * stride + (n < N ? n : 2 * N + groups)] = d;
+            }
         }
     }
     __syncthreads();
@@ -150,24 +177,34 @@ __global__ void moe_route_kernel(const A* __restrict__ x, const float* __restric
     }
 }
 
+// logits [T, logits_ld] or null: the router's (and behind them the gate row's) products, already worked out.
 extern "C" int rg_moe_route(const void* x, int dtype, const float* router, const float* correction, int* ids,
                             float* weights, int T, int W, int N, int top, int renormalize, int scoring, int groups, int keep,
-                            float scale, const float* gate_row, float* gate, void* stream) {
+                            float scale, const float* gate_row, float* gate, const float* logits, int logits_ld,
+                            void* stream) {
     if (T <= 0) return 0;
-    if (top < 1 || top > N || scoring < 0 || scoring > 1 || groups < 0 || (gate_row && !gate)) return RG_ERR_UNSUPPORTED;
+    if (top < 1 || top > N || scoring < 0 || scoring > 1 || groups < 0 || (gate_row && !gate)
+        || (logits && logits_ld < N + (gate_row ? 1 : 0))) return RG_ERR_UNSUPPORTED;
     if (groups > 0 && (N % groups || keep < 1 || keep > groups || top > keep * (N / groups))) return RG_ERR_UNSUPPORTED;
-    const size_t smem = (size_t)ROUTE_TOKENS * (2 * N + groups + 1) * sizeof(float);
+    const size_t per_token = (size_t)(2 * N + groups + 1) * sizeof(float);
+    int tokens = logits ? 8 : 1;                                   // a block's; without logits while there are blocks for every SM
+    while (!logits && tokens < 4 && T >= 148 * tokens) tokens *= 2;
+    while (tokens > 1 && per_token * tokens > 48 * 1024) tokens /= 2;
+    const size_t smem = per_token * tokens;
     if (smem > 48 * 1024) return RG_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    const int rows = N + (gate_row ? 1 : 0);
-    const int warps = rows < 4 ? 4 : (rows > 32 ? 32 : rows);      // a warp per router row, up to 32
-    dim3 grid((T + ROUTE_TOKENS - 1) / ROUTE_TOKENS), block(warps * 32);
-    if (dtype == RG_DTYPE_BF16)
-        return rg_launch(moe_route_kernel<bf16>, grid, block, smem, s, 1, (const bf16*)x, router, correction, ids,
-                         weights, T, W, N, top, renormalize, scoring, groups, keep, scale, gate_row, gate);
-    if (dtype == RG_DTYPE_F32)
-        return rg_launch(moe_route_kernel<float>, grid, block, smem, s, 1, (const float*)x, router, correction, ids,
-                         weights, T, W, N, top, renormalize, scoring, groups, keep, scale, gate_row, gate);
+    const int pairs = (N + (gate_row ? 1 : 0) + ROUTE_ROWS - 1) / ROUTE_ROWS;
+    int warps = pairs > 32 ? 32 : pairs;                           // a warp per two rows, and no fewer than take a token each
+    if (warps < 4 || logits) warps = logits ? 8 : 4;
+    dim3 grid((T + tokens - 1) / tokens), block(warps * 32);
+#define RG_ROUTE(A, N_) return rg_launch(moe_route_kernel<A, N_>, grid, block, smem, s, 1, (const A*)x, router, correction, ids, \
+        weights, T, W, N, top, renormalize, scoring, groups, keep, scale, gate_row, gate, logits, logits_ld)
+#define RG_ROUTE_TOKENS(A) switch (tokens) { case 1: RG_ROUTE(A, 1); case 2: RG_ROUTE(A, 2); case 4: RG_ROUTE(A, 4); \
+        default: RG_ROUTE(A, 8); }
+    if (dtype == RG_DTYPE_BF16) RG_ROUTE_TOKENS(bf16)
+    if (dtype == RG_DTYPE_F32) RG_ROUTE_TOKENS(float)
+#undef RG_ROUTE_TOKENS
+#undef RG_ROUTE
     return RG_ERR_UNSUPPORTED;
 }
 

@@ -526,11 +526,13 @@ def latent_attention_mma(qa: torch.Tensor, out: torch.Tensor, cache: torch.Tenso
 MOE_TILE_ROWS = 32
 
 
+ROUTE_PRODUCT_MIN_ROWS = 128
 MOE_SCORINGS = {"softmax": 0, "sigmoid": 1}
 
 
 def moe_route(x: torch.Tensor, router: torch.Tensor, correction, top: int, renormalize: bool = True,
-              scoring: str = "softmax", groups=None, scale: float = 1.0, gate_row: torch.Tensor | None = None):
+              scoring: str = "softmax", groups=None, scale: float = 1.0, gate_row: torch.Tensor | None = None,
+              half_rows: torch.Tensor | None = None):
     """Router of a mixture of experts: softmax of the 32-bit logits ``router`` x
     over all N outputs (``scoring`` "sigmoid": the sigmoid of each logit
     instead); the ``top`` outputs with the largest score + correction
@@ -538,8 +540,10 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction, top: int, renor
     their sum, or with ``renormalize`` False the scores themselves, times
     ``scale``.  ``groups`` = (count, keep): the outputs form that many equal
     groups of neighbours and only those of the ``keep`` groups with the largest
-    best score can be chosen.  Returns (ids int32 [T, top], weights float32
-    [T, top]); with ``gate_row`` (float32 [W]) also sigmoid(gate_row . x),
+    best score can be chosen.  ``half_rows``: the router's rows (and the gate's
+    behind them) in bfloat16, given only if they are the same numbers: many rows of
+    ``x`` then get their logits from one product with 32-bit sums and output.
+    Returns (ids int32 [T, top], weights float32 [T, top]); with ``gate_row`` (float32 [W]) also sigmoid(gate_row . x),
     float32 [T]."""
     _check(x, "x")
     _check(router, "router", torch.float32)
@@ -560,12 +564,18 @@ def moe_route(x: torch.Tensor, router: torch.Tensor, correction, top: int, renor
         if gate_row.numel() != W:
             raise KernelError(f"moe_route: a gate row of {gate_row.numel()} numbers for rows of {W}")
         gate = torch.empty(T, dtype=torch.float32, device=x.device)
+    logits = None
+    if half_rows is not None and x.dtype == torch.bfloat16 and T >= ROUTE_PRODUCT_MIN_ROWS:
+        if half_rows.shape[0] < N + int(gate_row is not None) or half_rows.shape[1] != W:
+            raise KernelError(f"moe_route: {tuple(half_rows.shape)} rows in bfloat16 for {N} outputs of rows of {W}")
+        logits = linear(x, half_rows, out_dtype=torch.float32)
     ids = torch.empty((T, top), dtype=torch.int32, device=x.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=x.device)
     _ok(_fn("moe", "rg_moe_route")(_ptr(x), c_int(_dtype_code(x)), _ptr(router), _ptr(correction), _ptr(ids),
                                    _ptr(weights), c_int(T), c_int(W), c_int(N), c_int(top), c_int(1 if renormalize else 0),
                                    c_int(MOE_SCORINGS[scoring]), c_int(count), c_int(keep), c_float(scale),
-                                   _ptr(gate_row), _ptr(gate), _stream()), "moe_route")
+                                   _ptr(gate_row), _ptr(gate), _ptr(logits),
+                                   c_int(logits.stride(0) if logits is not None else 0), _stream()), "moe_route")
     return (ids, weights) if gate_row is None else (ids, weights, gate)
 
 

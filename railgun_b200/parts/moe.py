@@ -122,11 +122,19 @@ class RoutedExperts(FeedForward):
             self.shared = self._shared_kind(p)(self._shared_params(p), prefix, env, tensors)
             if p.get("shared_gate"):
                 self.shared_gate = tensors.get(b + "shared.sg", torch.float32).reshape(-1).contiguous()
+        # prompts: the logits as one product, where bfloat16 holds the router's numbers as they are (the sums are 32-bit)
+        self.router_half = None
+        if env.dtype == torch.bfloat16:
+            rows = self.router if self.shared_gate is None else torch.cat([self.router, self.shared_gate[None]], dim=0)
+            half = rows.to(torch.bfloat16)
+            if torch.equal(half.float(), rows):
+                self.router_half = ops.pad_rows(half)
 
     def forward(self, x, batch):
         T = x.shape[0]
         ids, weights, *gate = ops.moe_route(x, self.router, self.correction, self.top, self.renormalize, self.scoring,
-                                            groups=self.groups, scale=self.weight_scale, gate_row=self.shared_gate)
+                                            groups=self.groups, scale=self.weight_scale, gate_row=self.shared_gate,
+                                            half_rows=self.router_half)
         y = pair_pos = None
         if self.E:
             places = T * self.top

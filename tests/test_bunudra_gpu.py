@@ -253,6 +253,17 @@ def test_router_with_groups_alone(N, top, W, groups, dtype):
     assert np.allclose(g.cpu().numpy(), P.sigmoid(x.double().numpy() @ gate.double().numpy()), atol=2e-6)
     two = ops.moe_route(dev(x), dev(router), None, top, False, groups=groups)              # without a gate: two results
     assert len(two) == 2 and torch.equal(two[0], ids)
+    if dtype == "bfloat16" and W % 8 == 0:
+        # many rows: the logits as one product, where bfloat16 holds the router's numbers
+        half = torch.cat([router, gate[None]]).to(torch.bfloat16)
+        many = dev(x).repeat(5, 1)
+        a = ops.moe_route(many, dev(half[:N].float()), None, top, False, groups=groups, scale=1.7, gate_row=dev(half[N].float()))
+        b = ops.moe_route(many, dev(half[:N].float()), None, top, False, groups=groups, scale=1.7, gate_row=dev(half[N].float()),
+                          half_rows=ops.pad_rows(dev(half)))
+        zh = x.double().numpy() @ half[:N].double().numpy().T
+        ok = torch.tensor([P.routing_margin(z, top, gd) > 1e-4 and np.diff(np.sort(z)).min() > 1e-4 for z in zh] * 5)
+        assert int(ok.sum()) > 150 and torch.equal(a[0].cpu()[ok], b[0].cpu()[ok])
+        assert torch.allclose(a[1].cpu()[ok], b[1].cpu()[ok], rtol=3e-5) and torch.allclose(a[2], b[2], atol=3e-6)
 
 
 def experts_part(W, m, t, dtype):
