@@ -148,8 +148,11 @@ struct TileGather {
 // EXACT: the head size is DMAX itself, known at compile time (loops unroll without guards and shared-memory
 // addresses fold into the instructions); otherwise any multiple of 16 up to DMAX, passed at run time.
 // POOL: the pooled entries' tiles come first, like the kept first tokens' tiles (`keep` is 0 then).
+// At head size 192 two blocks fit an SM if q has no place of its own in shared memory.
+__host__ __device__ constexpr bool prefill_q_borrows(int dmax) { return dmax == 192; }
+
 template <int DMAX, bool EXACT, bool POOL>
-__global__ void __launch_bounds__(NTHREADS, DMAX <= 64 ? 4 : (DMAX <= 128 ? 2 : 1))
+__global__ void __launch_bounds__(NTHREADS, DMAX <= 64 ? 4 : (DMAX <= 192 ? 2 : 1))
 prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restrict__ out,
                          const bf16* __restrict__ kv_cache, const int* __restrict__ block_table, int max_blocks,
                          const int* __restrict__ tiles, const int* __restrict__ positions, int nh, int nkv, int d_arg,
@@ -160,12 +163,14 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const int d = EXACT ? DMAX : d_arg;
     constexpr int KD = DMAX / 16;          // k-steps over the head dimension
     constexpr int ND = DMAX / 8;           // n-tiles of the output
-    constexpr bool Q_IN_REGS = DMAX <= 128;
+    constexpr bool Q_IN_REGS = DMAX <= 192;
+    constexpr bool Q_BORROWS = prefill_q_borrows(DMAX);   // q waits in the second stage's place until it is in registers
     extern __shared__ __align__(16) unsigned char smem_raw[];
     const int stride = d + PAD;
-    bf16* sQ = reinterpret_cast<bf16*>(smem_raw);                 // [64][stride]
-    bf16* sKV = sQ + 64 * stride;                                 // 2 stages x (K [BN][stride], V [BN][stride])
     const int stage_elems = 2 * BN * stride;
+    bf16* first = reinterpret_cast<bf16*>(smem_raw);
+    bf16* sKV = Q_BORROWS ? first : first + 64 * stride;          // 2 stages x (K [BN][stride], V [BN][stride])
+    bf16* sQ = Q_BORROWS ? sKV + stage_elems : first;             // [64][stride]
 
     pdl_wait();
     pdl_trigger();
@@ -230,6 +235,15 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
     const int b_key = (lane & 7) + (lane >> 4) * 8, b_dim = ((lane >> 3) & 1) * 8;          // K as B operand
     const int v_key = (lane & 7) + ((lane >> 3) & 1) * 8, v_dim = (lane >> 4) * 8;          // V as B operand (.trans)
 
+    if (Q_BORROWS) {
+        cp_async_wait<0>();
+        __syncthreads();
+#pragma unroll
+        for (int kd = 0; kd < KD; ++kd)
+            if (kd < d16) ldmatrix_x4(qf[Q_IN_REGS ? kd : 0], sQ + a_row * stride + kd * 16 + a_col);
+        __syncthreads();
+    }
+
     for (int vt = v0; vt <= kt1; ++vt) {
         const int kt = phys(vt);
         const int stage = (vt - v0) & 1;
@@ -246,7 +260,7 @@ prefill_attention_kernel(const bf16* __restrict__ q, int q_stride, bf16* __restr
             cp_async_wait<0>();
         }
         __syncthreads();
-        if (Q_IN_REGS && vt == v0) {
+        if (Q_IN_REGS && !Q_BORROWS && vt == v0) {
 #pragma unroll
             for (int kd = 0; kd < KD; ++kd)
                 if (kd < d16) ldmatrix_x4(qf[kd], sQ + a_row * stride + kd * 16 + a_col);
@@ -801,7 +815,7 @@ __global__ void decode_reduce_kernel(const float* __restrict__ part_o, const flo
     }
 }
 
-static size_t prefill_smem(int d) { return (size_t)(64 + 2 * 2 * BN) * (d + PAD) * sizeof(bf16); }
+static size_t prefill_smem(int d) { return (size_t)((prefill_q_borrows(d) ? 0 : 64) + 2 * 2 * BN) * (d + PAD) * sizeof(bf16); }
 static size_t decode_smem(int d) {
     // stages (+ a separate Q tile for the largest head-size class); the end-of-kernel combine reuses them
     const size_t stages = (size_t)((d > 128 ? 16 : 0) + DEC_STAGES * 2 * BN) * (d + PAD) * sizeof(bf16);
@@ -846,7 +860,7 @@ extern "C" int rg_prefill_attention_sink(const void* q, int q_stride, void* out,
         (bf16*)out, (const bf16*)kv_cache, block_table, max_blocks, tiles, positions, nh, nkv, d, page_size, page_shift, \
         window, window > 0 ? keep_first : 0, scale_log2, sink, (const bf16*)gate, gate_ld, (const bf16*)pool_kv, \
         pool_table, pool_blocks, pool, out_ld, out_scale); }
-    if (d == 64) RG_PREFILL(64, true) else if (d == 128) RG_PREFILL(128, true)
+    if (d == 64) RG_PREFILL(64, true) else if (d == 128) RG_PREFILL(128, true) else if (d == 192) RG_PREFILL(192, true)
     else if (d < 64) RG_PREFILL(64, false) else if (d < 128) RG_PREFILL(128, false) else RG_PREFILL(256, false)
 #undef RG_PREFILL_
 #undef RG_PREFILL

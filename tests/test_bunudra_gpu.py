@@ -383,7 +383,7 @@ def chunk_row(q, k, v, pos, size):
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,G,d,dv,page,size", [(4, 2, 16, 8, 8, 40), (6, 2, 112, 80, 16, 64), (3, 3, 24, 40, 16, 1), (2, 1, 16, 16, 4, 100),
                                                 (8, 8, 32, 32, 32, 65), (5, 1, 12, 20, 6, 63), (16, 2, 128, 128, 16, 128),
-                                                (12, 1, 64, 32, 16, 7), (2, 1, 256, 64, 16, 150), (4, 4, 64, 64, 64, 5000)])
+                                                (12, 1, 64, 32, 16, 7), (2, 1, 256, 64, 16, 150), (4, 4, 64, 64, 64, 5000), (6, 3, 180, 130, 16, 70)])
 def test_attention_in_chunks_alone(H, G, d, dv, page, size, dtype):
     """A query points at one loud key: its chunk's first one, the last of the chunk before it, the first of that chunk,
     its own, the sequence's first.  It is a single token and inside a portion that crosses the chunk's edge; in bfloat16
