@@ -1,14 +1,14 @@
 // The matrix memory of xLSTM (Beck et al., "xLSTM: Extended Long Short-Term Memory") around its scan:
 //
-//   i = cap tanh((z_i + b_i) / cap),   f = log sigmoid(cap tanh((z_f + b_f) / cap))      per head
-//   m_t = max(f + m_(t-1), i)                                                            m = 0 before the first token
-//   S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k v^T,   n_t likewise with k alone
-//   o   = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6)
+//   a = c(z_in), b = log sigmoid(c(z_forget)),  c(z) = cap tanh(z / cap)               per head
+//   m' = max(m + b, a)                                                                 m = 0 where a sequence begins
+//   [S | n] <- e^(m + b - m') [S | n] + e^(a - m') k [v | 1]^T
+//   [y | y_n] = q^T [S | n],  out = y / (max(|y_n|, e^(-m')) + 1e-6)
 //
 // n is one more column of S: the column of a value that is always 1.  The state of a request is S transposed with n
 // behind it, [H, dv + 1, d], and m, [H], all in 32-bit; a request whose start position is 0 begins from zeros whatever
 // its slot holds.
-//   mlstm_gates   portions: i, f and m of every token and head, and from them the factors of the two terms
+//   mlstm_gates   portions: a, b and m of every token and head, and from them the factors of the two terms
 //   mlstm_step    steps of single tokens: gates, S, n and S^T q, n . q in one kernel
 //   mlstm_out     the division, the heads' norm with a weight of all heads' size, the sigmoid gate, one rounding
 // The scan itself of portions is state_scan (state_mixers.cu) or ssd_chunk_scan (ssd_chunk.cu) with a column of ones.
@@ -21,58 +21,72 @@ __device__ __forceinline__ float ml_forget_gate(float z, float cap) {
 }
 
 // raw: rows ld apart, the H raw input gates at i_off, the forget gates at f_off.  keep [T, H] (its logarithm with
-// log_keep), put [T, H], m_out [T, H].  m [slots, H].  One block per (request, head): every thread takes a run of
-// tokens; the runs' composed steps m -> max(a + m, b) are scanned over the block, then every run is gone through again
-// from its own first m.
+// log_keep), put [T, H], m_out [T, H].  m [slots, H].  One block per (request, head), MG_SPAN tokens at a time: the gates'
+// logarithms go into shared memory, every thread takes a run of tokens, the runs' composed steps m -> max(m + A, B) are
+// scanned over the block, then every run is gone through again from its own first m.
 #define MG_THREADS 256
+#define MG_SPAN 4096
 __global__ void __launch_bounds__(MG_THREADS)
 mlstm_gates_kernel(const float* __restrict__ raw, int ld, int i_off, int f_off, const float* __restrict__ ib,
                    const float* __restrict__ fb, float cap, float* __restrict__ m, const int* __restrict__ cu_seqlens,
                    const int* __restrict__ start_pos, const int* __restrict__ slots, float* __restrict__ keep,
                    float* __restrict__ put, float* __restrict__ m_out, int H, int log_keep) {
-    __shared__ float wa[MG_THREADS / 32], wb[MG_THREADS / 32];
+    __shared__ float si[MG_SPAN + MG_SPAN / 32], sf[MG_SPAN + MG_SPAN / 32];   // a place unused after every 32: runs of 16 hit all banks
+    __shared__ float wa[MG_THREADS / 32], wb[MG_THREADS / 32], carry;
     pdl_wait();
     pdl_trigger();
     const int r = blockIdx.x, h = blockIdx.y;
     const int lo = cu_seqlens[r], n = cu_seqlens[r + 1] - lo;
     if (n <= 0) return;
     const int slot = slots[r];
-    const float m0 = slot >= 0 && start_pos[r] > 0 ? m[(size_t)slot * H + h] : 0.f;
     const float bi = ib[h], bf = fb[h];
-    const int run = (n + MG_THREADS - 1) / MG_THREADS;
-    const int t0 = min(n, (int)threadIdx.x * run), t1 = min(n, t0 + run);
-    const float* row = raw + (size_t)lo * ld + h;
-    float a = 0.f, b = -INFINITY;
-    for (int t = t0; t < t1; ++t) {
-        const float i = ml_input_gate(row[(size_t)t * ld + i_off] + bi, cap);
-        const float f = ml_forget_gate(row[(size_t)t * ld + f_off] + bf, cap);
-        a += f;
-        b = fmaxf(b + f, i);
-    }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    auto at = [](int t) { return t + (t >> 5); };
+    if (threadIdx.x == 0) carry = slot >= 0 && start_pos[r] > 0 ? m[(size_t)slot * H + h] : 0.f;
+    for (int s0 = 0; s0 < n; s0 += MG_SPAN) {
+        const int ns = min(MG_SPAN, n - s0);
+        const float* row = raw + (size_t)(lo + s0) * ld + h;
+#pragma unroll 4
+        for (int t = threadIdx.x; t < ns; t += MG_THREADS) {
+            const float zi = row[(size_t)t * ld + i_off], zf = row[(size_t)t * ld + f_off];
+            si[at(t)] = ml_input_gate(zi + bi, cap);
+            sf[at(t)] = ml_forget_gate(zf + bf, cap);
+        }
+        __syncthreads();
+        const int run = (ns + MG_THREADS - 1) / MG_THREADS;
+        const int t0 = min(ns, (int)threadIdx.x * run), t1 = min(ns, t0 + run);
+        float a = 0.f, b = -INFINITY;
+        for (int t = t0; t < t1; ++t) {
+            const float f = sf[at(t)];
+            a += f;
+            b = fmaxf(b + f, si[at(t)]);
+        }
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-        const float ua = __shfl_up_sync(0xffffffffu, a, o), ub = __shfl_up_sync(0xffffffffu, b, o);
-        if (lane >= o) { b = fmaxf(ub + a, b); a += ua; }
+        for (int o = 1; o < 32; o <<= 1) {
+            const float ua = __shfl_up_sync(0xffffffffu, a, o), ub = __shfl_up_sync(0xffffffffu, b, o);
+            if (lane >= o) { b = fmaxf(ub + a, b); a += ua; }
+        }
+        if (lane == 31) { wa[warp] = a; wb[warp] = b; }
+        __syncthreads();
+        float mt = carry;                                  // m before this warp's runs
+        for (int w = 0; w < warp; ++w) mt = fmaxf(wa[w] + mt, wb[w]);
+        const float pa = __shfl_up_sync(0xffffffffu, a, 1), pb = __shfl_up_sync(0xffffffffu, b, 1);
+        if (lane > 0) mt = fmaxf(pa + mt, pb);
+        __syncthreads();                                   // carry has been read
+        for (int t = t0; t < t1; ++t) {
+            const float f = sf[at(t)], i = si[at(t)];
+            const float now = fmaxf(f + mt, i);
+            const float k = f + mt - now;
+            const size_t to = (size_t)(lo + s0 + t) * H + h;
+            keep[to] = log_keep ? k : expf(k);
+            put[to] = expf(i - now);
+            m_out[to] = now;
+            mt = now;
+        }
+        if (t1 == ns && t0 < ns) carry = mt;
+        __syncthreads();
     }
-    if (lane == 31) { wa[warp] = a; wb[warp] = b; }
-    __syncthreads();
-    float mt = m0;                                     // m before this warp's runs
-    for (int w = 0; w < warp; ++w) mt = fmaxf(wa[w] + mt, wb[w]);
-    const float pa = __shfl_up_sync(0xffffffffu, a, 1), pb = __shfl_up_sync(0xffffffffu, b, 1);
-    if (lane > 0) mt = fmaxf(pa + mt, pb);
-    for (int t = t0; t < t1; ++t) {
-        const float i = ml_input_gate(row[(size_t)t * ld + i_off] + bi, cap);
-        const float f = ml_forget_gate(row[(size_t)t * ld + f_off] + bf, cap);
-        const float now = fmaxf(f + mt, i);
-        const float k = f + mt - now;
-        const size_t at = (size_t)(lo + t) * H + h;
-        keep[at] = log_keep ? k : expf(k);
-        put[at] = expf(i - now);
-        m_out[at] = now;
-        mt = now;
-    }
-    if (slot >= 0 && t1 == n && t0 < n) m[(size_t)slot * H + h] = mt;      // read at the start by this block only
+    if (slot >= 0 && threadIdx.x == 0) m[(size_t)slot * H + h] = carry;        // read at the start by this block only
 }
 
 extern "C" int rg_mlstm_gates(const float* raw, int ld, int i_off, int f_off, const float* ib, const float* fb, float cap,

@@ -2,7 +2,8 @@
 
 Layers in the order the configuration lists them.  A layer is a mixer and
 (unless it has none) a feed-forward, each with a layer norm on its OUTPUT
-only (arrangement "postnorm"): x <- x + norm1(mixer(x)), x <- x + norm2(ff(x)).
+only (arrangement "postnorm"): every part reads the 32-bit stream and adds the
+normed result to it.
 
 Mixers: "attention", grouped-query attention ("gqa_attention") with an RMS
 norm per head on q and k and half-layout rotation, in which a query sees its

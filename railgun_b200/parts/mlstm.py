@@ -2,12 +2,15 @@
 Memory"): a matrix per head with an exponential input gate, divided by what a
 normalizer remembers of the keys.
 
-  q = W_q h d^-1/2, k = W_k h [heads, d];  v = W_v h [heads, dv];  per head
-  i = cap tanh((W_i h + b_i) / cap),  f = log sigmoid(cap tanh((W_f h + b_f) / cap))
-  m_t = max(f + m_(t-1), i),  m = 0 before the first token
-  S_t = exp(f + m_(t-1) - m_t) S_(t-1) + exp(i - m_t) k v^T,  n_t likewise with k alone
-  o = S_t^T q / (max(|n_t . q|, exp(-m_t)) + 1e-6)
-  out = W_o (unit_rms(o) per head * weight * sigmoid(W_g h))
+Per head, with the raw numbers of the two gates cut off softly at +-cap (c(z) = cap tanh(z / cap)):
+
+  a = c(z_in),  b = log sigmoid(c(z_forget))         logarithms of what a token brings and of what is kept
+  m' = max(m + b, a)                                 m = 0 where a sequence begins
+  [S | n] <- e^(m + b - m') [S | n] + e^(a - m') k [v | 1]^T
+  [y | y_n] = q^T [S | n],  out = y / (max(|y_n|, e^(-m')) + 1e-6)
+
+so that S and n hold their sums over all tokens divided by e^m and stay in range.  The heads' outputs, each divided by its
+root mean square, are multiplied with a weight of all heads' size and the sigmoid of a gate before the output product.
 
 All first products are one, with 32-bit rows: everything from there to the
 rounding before the output product is 32-bit, and q's factor is applied where

@@ -245,7 +245,7 @@ def experts_ff(h, w, p, m, margins=None):
 
 # ---- the model -------------------------------------------------------------------------------------------
 def layer_forward(x, w, cfg, i, pos, margins=None):
-    """x <- x + norm1(mixer(x)); x <- x + norm2(ff(x))."""
+    """The stream after one layer: each part's output is normed and added."""
     L = cfg["layers"][i]
     eps = cfg["norm"]["eps"]
     p = f"l{i}."

@@ -188,6 +188,32 @@ def test_memory_over_portions(form, H, d, dv, cap):
         assert np.abs(r2[-1, 0] - ref[ask, 0]).max() > 0.01 * np.abs(ref[ask, 0]).max()
 
 
+def test_running_maximum_over_a_long_portion():
+    """m is scanned 4,096 tokens at a time: a portion longer than twice that, beside a short one; rising and falling gates."""
+    from railgun_b200 import ops
+    rng = np.random.default_rng(8)
+    H, d, dv, cap = 2, 4, 3, 10.0
+    lengths, starts, slots = [8200, 5, 4096], [0, 7, 3], [1, 0, 2]
+    T = sum(lengths)
+    rows = memory_rows(rng, T, H, d, dv, cap)
+    at = 2 * H * (d + dv)
+    rows[:, at + H:at + 2 * H] = 5.0 + 5.0 * torch.rand(T, H)                  # keeps nearly everything
+    rows[5000:, at:at + H] -= cap
+    ib, fb = rng.uniform(-1, 1, size=H), rng.uniform(0, 2, size=H)
+    m0 = rng.uniform(0, 2, size=(3, H))
+    state, m = torch.zeros((3, H, dv + 1, d), device=DEV), dev(m0, torch.float32)
+    f32 = lambda a: dev(a, torch.float32)
+    _, m_rows = ops.mlstm_scan(dev(rows), f32(ib), f32(fb), cap, state, m, step_batch(lengths, starts, slots), H, d, dv)
+    _, _, _, _, i, f = memory_parts(rows, H, d, dv, ib, fb, cap)
+    for sl, start, slot in zip(split(lengths), starts, slots):
+        now = m0[slot] if start else np.zeros(H)
+        for t in range(sl.start, sl.stop):
+            now = np.maximum(f[t] + now, i[t])
+            if t % 97 == 0 or t in (sl.start, sl.stop - 1, sl.start + 4095, sl.start + 4096):
+                assert np.abs(m_rows[t].cpu().numpy() - now).max() < 2e-4, t
+        assert np.abs(m[slot].cpu().numpy() - now).max() < 2e-4
+
+
 @pytest.mark.parametrize("H,d,dv,cap", MEMORIES)
 def test_memory_token_by_token(H, d, dv, cap):
     """The fused step: three live requests, one of them new in a dirty slot, and a padding row; state, normalizer and
